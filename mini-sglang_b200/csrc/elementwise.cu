@@ -149,14 +149,15 @@ MSGL_API int msgl_embedding(const int* ids, const void* table, float* out, int T
 }
 
 // ---------------------------------------------------------------------------------------
-// RMSNorm, optionally with the residual sum in front and a row gather:
+// RMSNorm or LayerNorm, optionally with the residual sum in front and a row gather:
 //   v      = (res_in ? res_in[src] : 0) + (x ? float(x[src]) : 0)        src = row_idx ? row_idx[r] : r
 //   res_out[r] = v                                                        (if res_out)
-//   y[r]   = T(v * rsqrt(mean(v^2) + eps) * w)
-// One block per row; the row is kept in shared memory between the two passes when it fits.
+//   y[r]   = T(v * rsqrt(mean(v^2) + eps) * w)                            RMS
+//   y[r]   = T((v - mean(v)) * rsqrt(mean((v - mean(v))^2) + eps) * w)    CENTER: mean taken off, weight, no bias
+// One block per row; the row is kept in shared memory between the passes when it fits.  X: the type of x (T or float).
 // ---------------------------------------------------------------------------------------
-template <typename T>
-__global__ void rmsnorm_kernel(const T* __restrict__ x, const float* res_in, float* res_out,
+template <typename T, typename X, bool CENTER>
+__global__ void rmsnorm_kernel(const X* __restrict__ x, const float* res_in, float* res_out,
                                const int* __restrict__ row_idx, const void* __restrict__ w, int w_is_f32,
                                float eps, T* __restrict__ y, int H, int cache_row) {
     extern __shared__ float srow[];
@@ -164,31 +165,33 @@ __global__ void rmsnorm_kernel(const T* __restrict__ x, const float* res_in, flo
     const int r = blockIdx.x;
     const size_t src = (size_t)(row_idx ? row_idx[r] : r) * H;
     const size_t dst = (size_t)r * H;
-    float ss = 0.f;
+    float ss = 0.f, sm = 0.f;
     for (int i = threadIdx.x; i < H; i += blockDim.x) {
         float v = 0.f;
         if (res_in) v = res_in[src + i];
-        if (x) v += to_f32<T>(x[src + i]);
+        if (x) v += to_f32<X>(x[src + i]);
         if (res_out) res_out[dst + i] = v;
         if (cache_row) srow[i] = v;
-        ss += v * v;
+        if (CENTER) sm += v; else ss += v * v;
+    }
+    auto value = [&](int i) -> float {
+        if (cache_row) return srow[i];
+        // row too long for shared memory: recompute from the inputs
+        if (res_out) return res_out[dst + i];
+        float v = 0.f;
+        if (res_in) v = res_in[src + i];
+        if (x) v += to_f32<X>(x[src + i]);
+        return v;
+    };
+    float mean = 0.f;
+    if (CENTER) {
+        mean = block_sum(sm, red) / (float)H;
+        for (int i = threadIdx.x; i < H; i += blockDim.x) { const float c = value(i) - mean; ss += c * c; }
     }
     const float total = block_sum(ss, red);
     const float inv = rsqrtf(total / (float)H + eps);
-    for (int i = threadIdx.x; i < H; i += blockDim.x) {
-        float v;
-        if (cache_row) {
-            v = srow[i];
-        } else {  // row too long for shared memory: recompute from the inputs
-            v = 0.f;
-            if (res_out) v = res_out[dst + i];
-            else {
-                if (res_in) v = res_in[src + i];
-                if (x) v += to_f32<T>(x[src + i]);
-            }
-        }
-        y[dst + i] = from_f32<T>(v * inv * load_weight(w, i, w_is_f32));
-    }
+    for (int i = threadIdx.x; i < H; i += blockDim.x)
+        y[dst + i] = from_f32<T>((value(i) - mean) * inv * load_weight(w, i, w_is_f32));
 }
 
 // Vectorised variant: 8 elements per thread and pass, the whole row held in registers between the
@@ -221,8 +224,8 @@ template <> struct Vec8<__nv_bfloat16> {
     }
 };
 
-template <typename T, int VPT>
-__global__ void rmsnorm_vec_kernel(const T* __restrict__ x, const float* res_in, float* res_out,
+template <typename T, typename X, bool CENTER, int VPT>
+__global__ void rmsnorm_vec_kernel(const X* __restrict__ x, const float* res_in, float* res_out,
                                    const int* __restrict__ row_idx, const void* __restrict__ w, int w_is_f32,
                                    float eps, T* __restrict__ y, int H) {
     __shared__ float red[32];
@@ -245,7 +248,7 @@ __global__ void rmsnorm_vec_kernel(const T* __restrict__ x, const float* res_in,
     pdl_after_wait();
     pdl_small();
     float v[VPT][8];
-    float ss = 0.f;
+    float ss = 0.f, sm = 0.f;
 #pragma unroll
     for (int j = 0; j < VPT; ++j) {
         const int i = (threadIdx.x + j * blockDim.x) << 3;
@@ -257,13 +260,24 @@ __global__ void rmsnorm_vec_kernel(const T* __restrict__ x, const float* res_in,
             }
             if (x) {
                 float xv[8];
-                Vec8<T>::load(x + src + i, xv);
+                Vec8<X>::load(x + src + i, xv);
 #pragma unroll
                 for (int k = 0; k < 8; ++k) v[j][k] += xv[k];
             }
             if (res_out) Vec8<float>::store(res_out + dst + i, v[j]);
 #pragma unroll
-            for (int k = 0; k < 8; ++k) ss += v[j][k] * v[j][k];
+            for (int k = 0; k < 8; ++k) { if (CENTER) sm += v[j][k]; else ss += v[j][k] * v[j][k]; }
+        }
+    }
+    if (CENTER) {
+        const float mean = block_sum(sm, red) / (float)H;
+#pragma unroll
+        for (int j = 0; j < VPT; ++j) {
+            const int i = (threadIdx.x + j * blockDim.x) << 3;
+            if ((i >> 3) < nvec) {
+#pragma unroll
+                for (int k = 0; k < 8; ++k) { v[j][k] -= mean; ss += v[j][k] * v[j][k]; }
+            }
         }
     }
     const float total = block_sum(ss, red);
@@ -280,45 +294,44 @@ __global__ void rmsnorm_vec_kernel(const T* __restrict__ x, const float* res_in,
     }
 }
 
-template <typename T>
-static bool launch_rmsnorm_vec(const void* x, const float* res_in, float* res_out, const int* row_idx, const void* w,
-                               int w_is_f32, float eps, void* y, int rows, int H, cudaStream_t stream) {
+template <typename T, typename X, bool CENTER>
+static int launch_norm(const void* x, const float* res_in, float* res_out, const int* row_idx, const void* w, int w_is_f32,
+                       float eps, void* y, int rows, int H, cudaStream_t stream) {
     const uintptr_t all = (uintptr_t)x | (uintptr_t)res_in | (uintptr_t)res_out | (uintptr_t)w | (uintptr_t)y;
-    if ((H & 7) || (all & 15)) return false;
-    const int nvec = H >> 3;
-    int threads = ((nvec + 31) / 32) * 32;
-    int vpt = 1;
-    while (threads > 512) { vpt *= 2; threads = (((nvec + vpt - 1) / vpt + 31) / 32) * 32; }
-    if (vpt > 4) return false;
-    const T* xp = (const T*)x;
+    const X* xp = (const X*)x;
     T* yp = (T*)y;
-    if (vpt == 1) msgl_launch_pdl(rmsnorm_vec_kernel<T, 1>, dim3(rows), dim3(threads), 0, stream, xp, res_in, res_out, row_idx, w, w_is_f32, eps, yp, H);
-    else if (vpt == 2) msgl_launch_pdl(rmsnorm_vec_kernel<T, 2>, dim3(rows), dim3(threads), 0, stream, xp, res_in, res_out, row_idx, w, w_is_f32, eps, yp, H);
-    else msgl_launch_pdl(rmsnorm_vec_kernel<T, 4>, dim3(rows), dim3(threads), 0, stream, xp, res_in, res_out, row_idx, w, w_is_f32, eps, yp, H);
-    return true;
-}
-
-MSGL_API int msgl_rmsnorm(const void* x, const float* res_in, float* res_out, const int* row_idx,
-                          const void* w, int w_is_f32, float eps, void* y, int rows, int H,
-                          int dtype, cudaStream_t stream) {
-    if (rows <= 0) return MSGL_OK;
-    if (H <= 0) return MSGL_ERR_SIZE;
-    if (dtype == MSGL_F32 && launch_rmsnorm_vec<float>(x, res_in, res_out, row_idx, w, w_is_f32, eps, y, rows, H, stream))
-        return msgl_check_launch();
-    if (dtype == MSGL_BF16 && launch_rmsnorm_vec<__nv_bfloat16>(x, res_in, res_out, row_idx, w, w_is_f32, eps, y, rows, H, stream))
-        return msgl_check_launch();
+    if (!((H & 7) || (all & 15))) {
+        const int nvec = H >> 3;
+        int threads = ((nvec + 31) / 32) * 32;
+        int vpt = 1;
+        while (threads > 512) { vpt *= 2; threads = (((nvec + vpt - 1) / vpt + 31) / 32) * 32; }
+        if (vpt <= 4) {
+            if (vpt == 1) msgl_launch_pdl(rmsnorm_vec_kernel<T, X, CENTER, 1>, dim3(rows), dim3(threads), 0, stream, xp, res_in, res_out, row_idx, w, w_is_f32, eps, yp, H);
+            else if (vpt == 2) msgl_launch_pdl(rmsnorm_vec_kernel<T, X, CENTER, 2>, dim3(rows), dim3(threads), 0, stream, xp, res_in, res_out, row_idx, w, w_is_f32, eps, yp, H);
+            else msgl_launch_pdl(rmsnorm_vec_kernel<T, X, CENTER, 4>, dim3(rows), dim3(threads), 0, stream, xp, res_in, res_out, row_idx, w, w_is_f32, eps, yp, H);
+            return msgl_check_launch();
+        }
+    }
     const int threads = H >= 2048 ? 512 : (H >= 512 ? 256 : 128);
     const int cache_row = (size_t)H * 4 <= 40 * 1024;
     const size_t smem = cache_row ? (size_t)H * 4 : 0;
-    if (dtype == MSGL_F32)
-        rmsnorm_kernel<float><<<rows, threads, smem, stream>>>((const float*)x, res_in, res_out, row_idx, w, w_is_f32,
-                                                               eps, (float*)y, H, cache_row);
-    else if (dtype == MSGL_BF16)
-        rmsnorm_kernel<__nv_bfloat16><<<rows, threads, smem, stream>>>((const __nv_bfloat16*)x, res_in, res_out, row_idx,
-                                                                       w, w_is_f32, eps, (__nv_bfloat16*)y, H, cache_row);
-    else
-        return MSGL_ERR_DTYPE;
+    rmsnorm_kernel<T, X, CENTER><<<rows, threads, smem, stream>>>(xp, res_in, res_out, row_idx, w, w_is_f32, eps, yp, H, cache_row);
     return msgl_check_launch();
+}
+
+// x_is_f32: x is float32 whatever the output type; center: LayerNorm (mean taken off), else RMSNorm
+MSGL_API int msgl_rmsnorm(const void* x, int x_is_f32, const float* res_in, float* res_out, const int* row_idx,
+                          const void* w, int w_is_f32, float eps, int center, void* y, int rows, int H,
+                          int dtype, cudaStream_t stream) {
+    if (rows <= 0) return MSGL_OK;
+    if (H <= 0) return MSGL_ERR_SIZE;
+#define NORM(T, X)                                                                                                          \
+    (center ? launch_norm<T, X, true>(x, res_in, res_out, row_idx, w, w_is_f32, eps, y, rows, H, stream)                     \
+            : launch_norm<T, X, false>(x, res_in, res_out, row_idx, w, w_is_f32, eps, y, rows, H, stream))
+    if (dtype == MSGL_F32) return NORM(float, float);
+    if (dtype == MSGL_BF16) return x_is_f32 ? NORM(__nv_bfloat16, float) : NORM(__nv_bfloat16, __nv_bfloat16);
+#undef NORM
+    return MSGL_ERR_DTYPE;
 }
 
 // ---------------------------------------------------------------------------------------

@@ -11,7 +11,7 @@
 //                               float32 per request; walks a request's tokens in order (decode and short portions)
 //   decay_chunk_*_kernel        the same for long portions: chunks of a request in parallel, their sums scanned in order
 //   rms_gate_kernel             RMS norm over a row, times sigmoid(gate), times a constant
-//   gated_act_kernel            act(gate) * up with act = silu or tanh-gelu
+//   gated_act_kernel            act(gate) * up with act = silu, tanh-gelu, sigmoid, relu or relu^2
 //   head_gate_kernel            a head's output times the sigmoid of the head's gate, into packed rows
 //   scaled_embedding_kernel     res = float(E[ids]) * c, the start of the float32 stream of a model that scales its embedding
 //   postnorm_residual_kernel    res += c * rmsnorm(a) * w (a sublayer's output normed before it is added), and the next
@@ -942,8 +942,18 @@ MSGL_API int msgl_rms_gate(const float* x, int N, const float* w, float eps, con
 }
 
 // ---------------------------------------------------------------------------------------
-// out = act(gate) * up; act 0 = silu, 1 = gelu (tanh form), 2 = sigmoid
+// out = act(gate) * up; act 0 = silu, 1 = gelu (tanh form), 2 = sigmoid, 3 = the square of relu, 4 = relu
 // ---------------------------------------------------------------------------------------
+__device__ __forceinline__ float gate_act_of(int act, float z) {
+    switch (act) {
+        case 1: return gelu_tanhf_(z);
+        case 2: return sigmoidf_(z);
+        case 3: { const float r = fmaxf(z, 0.f); return r * r; }
+        case 4: return fmaxf(z, 0.f);
+        default: return siluf_(z);
+    }
+}
+
 template <typename T, int V>
 __global__ void gated_act_kernel(const void* in_, long long in_stride, int gate_off, int up_off, void* out_, long long out_stride,
                                  int out_off, int I, int act) {
@@ -951,31 +961,35 @@ __global__ void gated_act_kernel(const void* in_, long long in_stride, int gate_
     const T* in = reinterpret_cast<const T*>(in_) + t * in_stride;
     T* out = reinterpret_cast<T*>(out_) + t * out_stride + out_off;
     for (int i = (blockIdx.y * blockDim.x + threadIdx.x) * V; i < I; i += gridDim.y * blockDim.x * V) {
-        float g[2], u[2], o[2];
-        ld_v<V>(in + gate_off + i, g);
-        ld_v<V>(in + up_off + i, u);
-        o[0] = (act == 1 ? gelu_tanhf_(g[0]) : (act == 2 ? sigmoidf_(g[0]) : siluf_(g[0]))) * u[0];
-        o[1] = V == 2 ? (act == 1 ? gelu_tanhf_(g[1]) : (act == 2 ? sigmoidf_(g[1]) : siluf_(g[1]))) * u[1] : 0.f;
-        st_v<V>(out + i, o);
+        float g[V], u[V], o[V];
+        ld_w<V>(in + gate_off + i, g);
+        ld_w<V>(in + up_off + i, u);
+#pragma unroll
+        for (int k = 0; k < V; ++k) o[k] = gate_act_of(act, g[k]) * u[k];
+        st_w<V>(out + i, o);
     }
 }
 
 MSGL_API int msgl_gated_act(const void* in, long long in_stride, int gate_off, int up_off, void* out, long long out_stride,
                             int out_off, int I, int act, int T, int dtype, cudaStream_t stream) {
     if (T <= 0 || I <= 0) return MSGL_OK;
-    if (act < 0 || act > 2) return MSGL_ERR_SIZE;
+    if (act < 0 || act > 4) return MSGL_ERR_SIZE;
     if (dtype != MSGL_F32 && dtype != MSGL_BF16) return MSGL_ERR_DTYPE;
     const size_t item = dtype == MSGL_F32 ? 4 : 2;
+    const bool v8 = multiple_of(8, I, in_stride, gate_off, up_off, out_stride, out_off) && aligned_to(in, 16) && aligned_to(out, 16);
     const bool v2 = even_all(I, in_stride, gate_off, up_off, out_stride, out_off) && aligned_to(in, 2 * item) && aligned_to(out, 2 * item);
-    const int per = v2 ? 2 : 1;
-    const dim3 grid(T, max(1, min((I + 256 * per - 1) / (256 * per), 64)));
-    if (dtype == MSGL_F32) {
-        if (v2) gated_act_kernel<float, 2><<<grid, 256, 0, stream>>>(in, in_stride, gate_off, up_off, out, out_stride, out_off, I, act);
-        else gated_act_kernel<float, 1><<<grid, 256, 0, stream>>>(in, in_stride, gate_off, up_off, out, out_stride, out_off, I, act);
-    } else {
-        if (v2) gated_act_kernel<__nv_bfloat16, 2><<<grid, 256, 0, stream>>>(in, in_stride, gate_off, up_off, out, out_stride, out_off, I, act);
-        else gated_act_kernel<__nv_bfloat16, 1><<<grid, 256, 0, stream>>>(in, in_stride, gate_off, up_off, out, out_stride, out_off, I, act);
-    }
+    const int per = v8 ? 8 : (v2 ? 2 : 1);
+    const int threads = I >= 256 * per ? 256 : max(32, (I / per + 31) / 32 * 32);
+    const dim3 grid(T, max(1, min((I + threads * per - 1) / (threads * per), 64)));
+#define GATED_ACT(T_)                                                                                                        \
+    do {                                                                                                                     \
+        if (v8) gated_act_kernel<T_, 8><<<grid, threads, 0, stream>>>(in, in_stride, gate_off, up_off, out, out_stride, out_off, I, act);       \
+        else if (v2) gated_act_kernel<T_, 2><<<grid, threads, 0, stream>>>(in, in_stride, gate_off, up_off, out, out_stride, out_off, I, act);  \
+        else gated_act_kernel<T_, 1><<<grid, threads, 0, stream>>>(in, in_stride, gate_off, up_off, out, out_stride, out_off, I, act);          \
+    } while (0)
+    if (dtype == MSGL_F32) GATED_ACT(float);
+    else GATED_ACT(__nv_bfloat16);
+#undef GATED_ACT
     return msgl_check_launch();
 }
 

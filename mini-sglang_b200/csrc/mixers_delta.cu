@@ -4,10 +4,12 @@
 //
 //   scaled_add_norm_kernel     res += x * s (s a float32 vector of the width), then y = rms(res) * w or y = res (or no y)
 //   rotary_angles_kernel       cos | sin of position * frequency for the tokens of a step, in double precision
-//   sink_qkv_prep_kernel       rotation of q and k heads in halves from the step's angles, values blended with another
-//                              layer's, K and V rows (of head sizes of their own) into the paged cache
+//   sink_qkv_prep_kernel       q and k heads RMS-normed, rotated in halves from the step's angles, values blended with another
+//                              layer's or brought to unit root mean square (each where asked), K and V rows (of head sizes of
+//                              their own) into the paged cache; a 16-byte form where nothing is rotated or blended
 //   sink_attention_kernel      causal softmax attention within a window over the paged cache, scores capped by a tanh
-//                              where asked, with exp(sink_h) in the denominator; float32 arithmetic, any head size to 512
+//                              where asked, with exp(sink_h) in the denominator and the output times a sigmoid gate per
+//                              element where given; float32 arithmetic, any head size to 512
 //   sink_attention_mma_kernel  the same for bfloat16 with both products on mma.sync tiles (64 rows a block, float32 scores,
 //                              running maximum and sum), prompts, portions and decoded tokens
 //   sink_merge_kernel          one-token steps cut a request's keys into pieces for blocks of their own: the pieces'
@@ -158,17 +160,38 @@ MSGL_API int msgl_rotary_angles(const int* positions, const double* freq, double
 
 // ---------------------------------------------------------------------------------------
 // q, k, v of a packed projection row [q: n_q * d | k: n_kv * d | v: n_kv * dv]:
-//   q and k heads: the first `rot` elements turn in halves by the token's angles (cs [T][rot] = cos | sin), the rest pass
-//   v heads: v <- (1 - lam) v + lam v_first where another layer's values are given
+//   q and k heads: where weights are given (wq, wk [d], for all heads), x / sqrt(mean(x^2) + eps) * w first; then the first
+//   `rot` elements turn in halves by the token's angles (cs [T][rot] = cos | sin), the rest pass
+//   v heads: v <- (1 - lam) v + lam v_first where another layer's values are given; with v_unit then v / sqrt(mean(v^2) + eps)
 //   q -> q_out [T, n_q, d]; k, v -> the paged caches at token slot out_loc[t] (where given)
 // One warp per (token, head of q, k or v).
 // ---------------------------------------------------------------------------------------
+__device__ __forceinline__ void sk_load16(const float* p, float (&v)[4]) {
+    const float4 a = *reinterpret_cast<const float4*>(p);
+    v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w;
+}
+__device__ __forceinline__ void sk_load16(const __nv_bfloat16* p, float (&v)[8]) {
+    const uint4 a = *reinterpret_cast<const uint4*>(p);
+    const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&a);
+#pragma unroll
+    for (int k = 0; k < 4; ++k) { const float2 f = __bfloat1622float2(h[k]); v[2 * k] = f.x; v[2 * k + 1] = f.y; }
+}
+__device__ __forceinline__ void sk_store16(float* p, const float (&v)[4]) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
+__device__ __forceinline__ void sk_store16(__nv_bfloat16* p, const float (&v)[8]) {
+    uint4 a;
+    __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&a);
+#pragma unroll
+    for (int k = 0; k < 4; ++k) h[k] = __floats2bfloat162_rn(v[2 * k], v[2 * k + 1]);
+    *reinterpret_cast<uint4*>(p) = a;
+}
+
 struct SinkPrepParams {
     const void* proj; long long stride;
     const float* cs; int rot;
     const void* v_first; long long vf_stride; float lam;
     const int* out_loc; void* q_out; void* k_cache; void* v_cache;
     int page_size, n_q, n_kv, d, dv, T;
+    const float* wq; const float* wk; int v_unit; float eps;
 };
 
 template <typename T>
@@ -192,11 +215,19 @@ __global__ void __launch_bounds__(128) sink_qkv_prep_kernel(const SinkPrepParams
             const int loc = p.out_loc[t];
             dst = reinterpret_cast<T*>(p.k_cache) + (((size_t)(loc / p.page_size) * p.n_kv + h) * p.page_size + loc % p.page_size) * p.d;
         }
+        const float* w = is_q ? p.wq : p.wk;
+        float f = 1.f;
+        if (w != nullptr) {
+            float ss = 0.f;
+            for (int e = lane; e < p.d; e += 32) { const float v = to_f32<T>(src[e]); ss = fmaf(v, v, ss); }
+            f = 1.f / sqrtf(warp_sum(ss) / (float)p.d + p.eps);
+        }
+        auto elem = [&](int e) -> float { const float v = to_f32<T>(src[e]); return w != nullptr ? v * f * w[e] : v; };
         for (int e = lane; e < p.d; e += 32) {
-            float v = to_f32<T>(src[e]);
+            float v = elem(e);
             if (cs != nullptr && e < p.rot) {
-                if (e < half) v = v * cs[e] - to_f32<T>(src[e + half]) * cs[half + e];
-                else v = v * cs[e - half] + to_f32<T>(src[e - half]) * cs[e];
+                if (e < half) v = v * cs[e] - elem(e + half) * cs[half + e];
+                else v = v * cs[e - half] + elem(e - half) * cs[e];
             }
             dst[e] = from_f32<T>(v);
         }
@@ -207,25 +238,94 @@ __global__ void __launch_bounds__(128) sink_qkv_prep_kernel(const SinkPrepParams
         const T* vf = p.v_first ? reinterpret_cast<const T*>(p.v_first) + (size_t)t * p.vf_stride + (size_t)h * p.dv : nullptr;
         const int loc = p.out_loc[t];
         T* dst = reinterpret_cast<T*>(p.v_cache) + (((size_t)(loc / p.page_size) * p.n_kv + h) * p.page_size + loc % p.page_size) * p.dv;
-        for (int e = lane; e < p.dv; e += 32) {
-            float v = to_f32<T>(src[e]);
-            if (vf != nullptr) v = (1.f - p.lam) * v + p.lam * to_f32<T>(vf[e]);
-            dst[e] = from_f32<T>(v);
+        auto elem = [&](int e) -> float {
+            const float v = to_f32<T>(src[e]);
+            return vf != nullptr ? (1.f - p.lam) * v + p.lam * to_f32<T>(vf[e]) : v;
+        };
+        float f = 1.f;
+        if (p.v_unit) {
+            float ss = 0.f;
+            for (int e = lane; e < p.dv; e += 32) { const float v = elem(e); ss = fmaf(v, v, ss); }
+            f = 1.f / sqrtf(warp_sum(ss) / (float)p.dv + p.eps);
         }
+        for (int e = lane; e < p.dv; e += 32) dst[e] = from_f32<T>(elem(e) * f);
     }
+}
+
+// The same without rotation or blending, a lane 16 bytes of a head (head sizes that are multiples of the vector and at most
+// 32 vectors): one read of every element, the norms from registers.
+template <typename T>
+__global__ void __launch_bounds__(128) sink_qkv_prep_vec_kernel(const SinkPrepParams p) {
+    constexpr int V = 16 / sizeof(T);
+    const long long w_idx = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+    const int n_slots = p.n_q + 2 * p.n_kv, lane = threadIdx.x & 31;
+    // heads of a size of 16 vectors or less share a warp: `per` heads side by side
+    const int nd = p.d / V, nv = p.dv / V, widest = nd > nv ? nd : nv;
+    const int lanes = widest <= 4 ? 4 : widest <= 8 ? 8 : widest <= 16 ? 16 : 32, per = 32 / lanes;
+    const long long job = w_idx * per + lane / lanes;
+    const int l = lane % lanes;
+    const bool live = job < (long long)p.T * n_slots;
+    const int t = live ? (int)(job / n_slots) : 0, slot = live ? (int)(job - (long long)t * n_slots) : 0;
+    const bool is_v = slot >= p.n_q + p.n_kv, is_q = slot < p.n_q;
+    const int n = is_v ? p.dv : p.d;
+    const T* row = reinterpret_cast<const T*>(p.proj) + (size_t)t * p.stride;
+    const T* src = is_v ? row + (size_t)(p.n_q + p.n_kv) * p.d + (size_t)(slot - p.n_q - p.n_kv) * p.dv : row + (size_t)slot * p.d;
+    const bool mine = live && l * V < n && (is_q || p.k_cache != nullptr);
+    float v[V];
+#pragma unroll
+    for (int k = 0; k < V; ++k) v[k] = 0.f;
+    if (mine) sk_load16(src + l * V, v);
+    float ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < V; ++k) ss = fmaf(v[k], v[k], ss);
+    for (int o = lanes >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    if (!mine) return;
+    const float* w = is_v ? nullptr : (is_q ? p.wq : p.wk);
+    const float f = (is_v ? p.v_unit != 0 : w != nullptr) ? 1.f / sqrtf(ss / (float)n + p.eps) : 1.f;
+    if (w != nullptr) {
+        const float4* w4 = reinterpret_cast<const float4*>(w + l * V);
+#pragma unroll
+        for (int k = 0; k < V / 4; ++k) {
+            const float4 x = w4[k];
+            v[4 * k] *= f * x.x; v[4 * k + 1] *= f * x.y; v[4 * k + 2] *= f * x.z; v[4 * k + 3] *= f * x.w;
+        }
+    } else {
+#pragma unroll
+        for (int k = 0; k < V; ++k) v[k] *= f;
+    }
+    T* dst;
+    if (is_q) {
+        dst = reinterpret_cast<T*>(p.q_out) + ((size_t)t * p.n_q + slot) * p.d;
+    } else {
+        const int loc = p.out_loc[t], h = is_v ? slot - p.n_q - p.n_kv : slot - p.n_q;
+        dst = reinterpret_cast<T*>(is_v ? p.v_cache : p.k_cache) +
+              (((size_t)(loc / p.page_size) * p.n_kv + h) * p.page_size + loc % p.page_size) * n;
+    }
+    sk_store16(dst + l * V, v);
 }
 
 MSGL_API int msgl_sink_qkv_prep(const void* proj, long long stride, const float* cs, int rot, const void* v_first, long long vf_stride,
                                 float lam, const int* out_loc, void* q_out, void* k_cache, void* v_cache, int page_size, int n_q, int n_kv,
-                                int d, int dv, int T_, int dtype, cudaStream_t stream) {
+                                int d, int dv, int T_, int dtype, const float* wq, const float* wk, int v_unit, float eps,
+                                cudaStream_t stream) {
     if (T_ <= 0) return MSGL_OK;
+    if (dtype != MSGL_F32 && dtype != MSGL_BF16) return MSGL_ERR_DTYPE;
     if (d <= 0 || dv <= 0 || n_q <= 0 || n_kv <= 0 || rot < 0 || rot > d || (rot & 1) || page_size < 1 || (rot > 0 && cs == nullptr) ||
         (k_cache != nullptr && (out_loc == nullptr || v_cache == nullptr)))
         return MSGL_ERR_SIZE;
     SinkPrepParams p;
     p.proj = proj; p.stride = stride; p.cs = rot > 0 ? cs : nullptr; p.rot = rot; p.v_first = v_first; p.vf_stride = vf_stride; p.lam = lam;
     p.out_loc = out_loc; p.q_out = q_out; p.k_cache = k_cache; p.v_cache = v_cache; p.page_size = page_size; p.n_q = n_q; p.n_kv = n_kv;
-    p.d = d; p.dv = dv; p.T = T_;
+    p.d = d; p.dv = dv; p.T = T_; p.wq = wq; p.wk = wk; p.v_unit = v_unit; p.eps = eps;
+    const int V = dtype == MSGL_F32 ? 4 : 8;
+    const uintptr_t all = (uintptr_t)proj | (uintptr_t)q_out | (uintptr_t)k_cache | (uintptr_t)v_cache | (uintptr_t)wq | (uintptr_t)wk;
+    if (p.cs == nullptr && v_first == nullptr && d % V == 0 && dv % V == 0 && stride % V == 0 && max(d, dv) <= 32 * V && (all & 15) == 0) {
+        const int widest = max(d, dv) / V, lanes = widest <= 4 ? 4 : widest <= 8 ? 8 : widest <= 16 ? 16 : 32, per = 4 * (32 / lanes);
+        const unsigned blocks = (unsigned)(((long long)T_ * (n_q + 2 * n_kv) + per - 1) / per);
+        if (dtype == MSGL_F32) sink_qkv_prep_vec_kernel<float><<<blocks, 128, 0, stream>>>(p);
+        else sink_qkv_prep_vec_kernel<__nv_bfloat16><<<blocks, 128, 0, stream>>>(p);
+        return msgl_check_launch();
+    }
     const dim3 grid(T_, (n_q + 2 * n_kv + 3) / 4);
     if (dtype == MSGL_F32) sink_qkv_prep_kernel<float><<<grid, 128, 0, stream>>>(p);
     else if (dtype == MSGL_BF16) sink_qkv_prep_kernel<__nv_bfloat16><<<grid, 128, 0, stream>>>(p);
@@ -238,6 +338,7 @@ MSGL_API int msgl_sink_qkv_prep(const void* proj, long long stride, const float*
 //
 //   s(i, j) = q[i, h] . k[j, g] * scale;   s <- cap * tanh(s / cap) (cap > 0);   j <= i and (no window or i - j < window)
 //   o[i, h, :] = sum_j exp(s(i, j)) v[j, g, :] / (sum_j exp(s(i, j)) + exp(sink[h]))
+//   o[i, h, e] <- o[i, h, e] * sigmoid(gate[i, h, e])   (where gates are given: rows of the activation type, one per output element)
 //
 // A block owns a tile of QT tokens x GH query heads of one kv head (SK_ROWS rows, one warp each) and walks the keys in
 // chunks of 32 anchored at multiples of 32, with a running maximum and sum per row.  In the score phase lane l of a row's
@@ -260,6 +361,7 @@ struct SinkAttnParams {
     float* part_o; float* part_ml; int splits, split_keys;      // [splits][T][n_q][dv], [splits][T][n_q][2]
     int T, B, n_q, n_kv, d, dv, page_size, QT, GH, window;
     float scale, softcap;
+    const void* gate; long long gate_stride;      // [T rows][n_q * dv] or null
 };
 
 template <typename T, int DPL>
@@ -395,7 +497,11 @@ __global__ void __launch_bounds__(SK_ROWS * 32) sink_attention_kernel(const Sink
 #pragma unroll
     for (int i = 0; i < DPL; ++i) {
         const int e = lane + 32 * i;
-        if (e < dv) og[e] = from_f32<T>(o[i] * inv);
+        if (e < dv) {
+            float r = o[i] * inv;
+            if (p.gate != nullptr) r *= sigmoidf_(to_f32<T>(reinterpret_cast<const T*>(p.gate)[(size_t)tok * p.gate_stride + (size_t)head * dv + e]));
+            og[e] = from_f32<T>(r);
+        }
     }
 }
 
@@ -403,7 +509,8 @@ __global__ void __launch_bounds__(SK_ROWS * 32) sink_attention_kernel(const Sink
 template <typename T>
 __global__ void __launch_bounds__(128) sink_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                                          const float* __restrict__ sink, T* __restrict__ out, long long out_stride,
-                                                         int T_, int n_q, int dv, int splits) {
+                                                         int T_, int n_q, int dv, int splits, const T* __restrict__ gate,
+                                                         long long gate_stride) {
     const int t = blockIdx.x, head = blockIdx.y;
     const size_t r0 = (size_t)t * n_q + head, step = (size_t)T_ * n_q;
     float M = sink[head];
@@ -417,7 +524,9 @@ __global__ void __launch_bounds__(128) sink_merge_kernel(const float* __restrict
             const float f = expf(part_ml[2 * (r0 + s * step)] - M);
             if (f != 0.f) acc = fmaf(part_o[(r0 + s * step) * dv + e], f, acc);
         }
-        out[(size_t)t * out_stride + (size_t)head * dv + e] = from_f32<T>(acc * inv);
+        acc *= inv;
+        if (gate != nullptr) acc *= sigmoidf_(to_f32<T>(gate[(size_t)t * gate_stride + (size_t)head * dv + e]));
+        out[(size_t)t * out_stride + (size_t)head * dv + e] = from_f32<T>(acc);
     }
 }
 
@@ -425,7 +534,7 @@ MSGL_API int msgl_sink_attention(const void* q, const void* k_cache, const void*
                                  const int* block_table, int bt_stride, int uniform, int n_tiles, const float* sink, void* out,
                                  long long out_stride, float* part_o, float* part_ml, int splits, int split_keys, int T_, int B, int n_q,
                                  int n_kv, int d, int dv, int page_size, int QT, int GH, int window, float scale, float softcap, int dtype,
-                                 cudaStream_t stream) {
+                                 const void* gate, long long gate_stride, cudaStream_t stream) {
     if (n_tiles <= 0) return MSGL_OK;
     if (d <= 0 || dv <= 0 || dv > 32 * SK_MAX_DPL || d > 32 * SK_MAX_DPL || n_kv <= 0 || n_q % n_kv || QT < 1 || GH < 1 ||
         QT * GH > SK_ROWS || page_size < 1 || sink == nullptr || window < 0 || splits < 1 ||
@@ -437,6 +546,7 @@ MSGL_API int msgl_sink_attention(const void* q, const void* k_cache, const void*
     p.bt_stride = bt_stride; p.uniform = uniform; p.sink = sink; p.out = out; p.out_stride = out_stride; p.part_o = part_o;
     p.part_ml = part_ml; p.splits = splits; p.split_keys = split_keys; p.T = T_; p.B = B; p.n_q = n_q; p.n_kv = n_kv; p.d = d; p.dv = dv;
     p.page_size = page_size; p.QT = QT; p.GH = GH; p.window = window; p.scale = scale; p.softcap = softcap;
+    p.gate = gate; p.gate_stride = gate_stride;
     const int G = n_q / n_kv;
     const dim3 grid(n_tiles, n_kv * ((G + GH - 1) / GH), splits);
     const size_t smem = ((size_t)SK_ROWS * d + (size_t)SK_KC * (d + 1) + (size_t)SK_KC * dv) * sizeof(float);
@@ -461,8 +571,8 @@ MSGL_API int msgl_sink_attention(const void* q, const void* k_cache, const void*
     int code = msgl_check_launch();
     if (code != MSGL_OK || splits <= 1) return code;
     const dim3 g2(T_, n_q);
-    if (dtype == MSGL_F32) sink_merge_kernel<float><<<g2, 128, 0, stream>>>(part_o, part_ml, sink, (float*)out, out_stride, T_, n_q, dv, splits);
-    else sink_merge_kernel<__nv_bfloat16><<<g2, 128, 0, stream>>>(part_o, part_ml, sink, (__nv_bfloat16*)out, out_stride, T_, n_q, dv, splits);
+    if (dtype == MSGL_F32) sink_merge_kernel<float><<<g2, 128, 0, stream>>>(part_o, part_ml, sink, (float*)out, out_stride, T_, n_q, dv, splits, (const float*)gate, gate_stride);
+    else sink_merge_kernel<__nv_bfloat16><<<g2, 128, 0, stream>>>(part_o, part_ml, sink, (__nv_bfloat16*)out, out_stride, T_, n_q, dv, splits, (const __nv_bfloat16*)gate, gate_stride);
     return msgl_check_launch();
 }
 
@@ -739,11 +849,18 @@ __global__ void __launch_bounds__(SKM_THREADS) sink_attention_mma_kernel(const S
         const float f = ex2_(m_run[half] - M);
         const float inv = __fdividef(f, l * f + ex2_(sk2 - M));
         __nv_bfloat16* dst = og + tok * p.out_stride + (size_t)head * dv;
+        const __nv_bfloat16* gt = p.gate ? reinterpret_cast<const __nv_bfloat16*>(p.gate) + tok * p.gate_stride + (size_t)head * dv : nullptr;
 #pragma unroll
         for (int nd = 0; nd < NDB; ++nd) {
             const int col = nd * 8 + (lane & 3) * 2;
-            if (col < dv)           // dv is a multiple of 8: a pair lies inside the row or outside it
-                *reinterpret_cast<__nv_bfloat162*>(dst + col) = __floats2bfloat162_rn(o[nd][half * 2] * inv, o[nd][half * 2 + 1] * inv);
+            if (col < dv) {         // dv is a multiple of 8: a pair lies inside the row or outside it
+                float a = o[nd][half * 2] * inv, b = o[nd][half * 2 + 1] * inv;
+                if (gt != nullptr) {
+                    const float2 g = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(gt + col));
+                    a *= sigmoidf_(g.x); b *= sigmoidf_(g.y);
+                }
+                *reinterpret_cast<__nv_bfloat162*>(dst + col) = __floats2bfloat162_rn(a, b);
+            }
         }
     }
 }
@@ -755,10 +872,11 @@ __global__ void __launch_bounds__(SKM_THREADS) sink_attention_mma_kernel(const S
 MSGL_API int msgl_sink_attention_mma(const void* q, const void* k_cache, const void* v_cache, const int* q_start, const int* kv_len,
                                      const int* block_table, int bt_stride, int uniform, int n_tiles, const float* sink, void* out,
                                      long long out_stride, float* part_o, float* part_ml, int splits, int split_keys, int T_, int B, int n_q,
-                                     int n_kv, int d, int dv, int page_size, int window, float scale, float softcap, cudaStream_t stream) {
+                                     int n_kv, int d, int dv, int page_size, int window, float scale, float softcap, const void* gate,
+                                     long long gate_stride, cudaStream_t stream) {
     if (n_tiles <= 0) return MSGL_OK;
     if (d <= 0 || dv <= 0 || d > 128 || dv > 128 || d % 8 || dv % 8 || n_kv <= 0 || n_q % n_kv || page_size < 1 || sink == nullptr ||
-        window < 0 || (out_stride & 1) || ((size_t)out & 3) || splits < 1 ||
+        window < 0 || (out_stride & 1) || ((size_t)out & 3) || (gate_stride & 1) || ((size_t)gate & 3) || splits < 1 ||
         (splits > 1 && (!uniform || part_o == nullptr || part_ml == nullptr || split_keys < SKM_KT || split_keys % SKM_KT || ((size_t)part_o & 7))))
         return MSGL_ERR_SIZE;
     SinkAttnParams p;
@@ -766,6 +884,7 @@ MSGL_API int msgl_sink_attention_mma(const void* q, const void* k_cache, const v
     p.bt_stride = bt_stride; p.uniform = uniform; p.sink = sink; p.out = out; p.out_stride = out_stride; p.part_o = part_o;
     p.part_ml = part_ml; p.splits = splits; p.split_keys = split_keys; p.T = T_; p.B = B; p.n_q = n_q; p.n_kv = n_kv; p.d = d; p.dv = dv;
     p.page_size = page_size; p.QT = 0; p.GH = 0; p.window = window; p.scale = scale; p.softcap = softcap;
+    p.gate = gate; p.gate_stride = gate_stride;
     const int G = n_q / n_kv;
     const dim3 grid(n_tiles, n_kv * (G <= SKM_R ? 1 : (G + SKM_R - 1) / SKM_R), splits);
 #define SKM_LAUNCH(DK, DV)                                                                                                   \
@@ -792,7 +911,7 @@ MSGL_API int msgl_sink_attention_mma(const void* q, const void* k_cache, const v
     int code = msgl_check_launch();
     if (code != MSGL_OK || splits <= 1) return code;
     const dim3 g2(T_, n_q);
-    sink_merge_kernel<__nv_bfloat16><<<g2, 128, 0, stream>>>(part_o, part_ml, sink, (__nv_bfloat16*)out, out_stride, T_, n_q, dv, splits);
+    sink_merge_kernel<__nv_bfloat16><<<g2, 128, 0, stream>>>(part_o, part_ml, sink, (__nv_bfloat16*)out, out_stride, T_, n_q, dv, splits, (const __nv_bfloat16*)gate, gate_stride);
     return msgl_check_launch();
 }
 

@@ -1585,10 +1585,11 @@ MSGL_API int msgl_unary_act(const void* x, long long x_stride, void* out, long l
 // ---------------------------------------------------------------------------------------
 // Router of a mixture of experts: one block per token
 //
-//   z = W h (float32 sums), s = sigmoid(z), choice = s + correction
-//   the experts form `n_groups` equal groups of neighbours; a group's score is the sum of its two largest choice scores; only
-//   experts of the `keep` best groups can be chosen; the `top` largest choice scores among them are chosen (the lower index
-//   wins a tie); weights = the chosen experts' s over their sum (+ 1e-20)
+//   z = W h (float32 sums); s = sigmoid(z) (score 0) or softmax(z) over all experts (score 2); choice = s + correction
+//   the experts form `n_groups` equal groups of neighbours; a group's score is the sum of its two largest choice scores, or the
+//   largest one (group_max); only experts of the `keep` best groups can be chosen; the `top` largest choice scores among them
+//   are chosen (the lower index wins a tie); weights = the chosen experts' s over their sum (+ 1e-20), or as they are (!renorm)
+//   score 1: the logits z themselves are chosen by, weights = softmax over the chosen ones
 //   -> idx int32 [T, top], wts float32 [T, top]
 // ---------------------------------------------------------------------------------------
 #define RT_MAX_EXPERTS 1024
@@ -1596,9 +1597,11 @@ MSGL_API int msgl_unary_act(const void* x, long long x_stride, void* out, long l
 template <typename T>
 __global__ void __launch_bounds__(256) route_kernel(const T* __restrict__ h, long long h_stride, const T* __restrict__ W,
                                                     const float* __restrict__ correction, int H, int E, int n_groups, int keep,
-                                                    int top, int* __restrict__ idx, float* __restrict__ wts, int vec, int softmax,
-                                                    const T* __restrict__ gate_row, float* __restrict__ gate_out) {
-    __shared__ float s_sh[RT_MAX_EXPERTS], c_sh[RT_MAX_EXPERTS], g_sh[RT_MAX_GROUPS];
+                                                    int top, int* __restrict__ idx, float* __restrict__ wts, int vec, int score,
+                                                    int group_max, int renorm, const T* __restrict__ gate_row,
+                                                    float* __restrict__ gate_out) {
+    __shared__ float s_sh[RT_MAX_EXPERTS], c_sh[RT_MAX_EXPERTS], g_sh[RT_MAX_GROUPS], red[32];
+    const bool softmax = score == 1;
     const int t = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5, nw = blockDim.x >> 5;
     const T* hr = h + (size_t)t * h_stride;
     // row E, if there is one, is no expert: the sigmoid of its product with the token is handed out beside the choice
@@ -1622,7 +1625,7 @@ __global__ void __launch_bounds__(256) route_kernel(const T* __restrict__ h, lon
         if (lane == 0) {
             if (e >= E) {
                 gate_out[t] = sigmoidf_(acc);
-            } else if (softmax) {                        // the logits themselves are chosen by and weighted
+            } else if (score) {                          // the logits themselves (1: are chosen by and weighted)
                 s_sh[e] = acc;
                 c_sh[e] = acc;
             } else {
@@ -1633,6 +1636,21 @@ __global__ void __launch_bounds__(256) route_kernel(const T* __restrict__ h, lon
         }
     }
     __syncthreads();
+    if (score == 2) {                                    // softmax over all of them
+        float m = -INFINITY;
+        for (int e = lane; e < E; e += 32) m = fmaxf(m, s_sh[e]);
+        m = warp_max(m);                                 // every warp finds it by itself
+        float part = 0.f;
+        __syncthreads();
+        for (int e = tid; e < E; e += blockDim.x) { const float x = expf(s_sh[e] - m); s_sh[e] = x; part += x; }
+        const float inv = 1.f / block_sum(part, red);
+        for (int e = tid; e < E; e += blockDim.x) {
+            const float s = s_sh[e] * inv;
+            s_sh[e] = s;
+            c_sh[e] = s + (correction ? correction[e] : 0.f);
+        }
+        __syncthreads();
+    }
     const int per = E / n_groups;
     if (keep < n_groups) {
         for (int g = tid; g < n_groups; g += blockDim.x) {
@@ -1641,7 +1659,7 @@ __global__ void __launch_bounds__(256) route_kernel(const T* __restrict__ h, lon
                 const float v = c_sh[g * per + i];
                 if (v > m1) { m2 = m1; m1 = v; } else if (v > m2) m2 = v;
             }
-            g_sh[g] = per >= 2 ? m1 + m2 : m1;
+            g_sh[g] = per >= 2 && !group_max ? m1 + m2 : m1;
         }
         __syncthreads();
         if (tid == 0) {
@@ -1682,18 +1700,18 @@ __global__ void __launch_bounds__(256) route_kernel(const T* __restrict__ h, lon
             const float inv = 1.f / total;
             for (int k = lane; k < top; k += 32) wts[(size_t)t * top + k] = expf(s_sh[idx[(size_t)t * top + k]] - first) * inv;
         } else {
-            const float inv = 1.f / (total + 1e-20f);
+            const float inv = renorm ? 1.f / (total + 1e-20f) : 1.f;
             for (int k = lane; k < top; k += 32) wts[(size_t)t * top + k] = s_sh[idx[(size_t)t * top + k]] * inv;
         }
     }
 }
 
 MSGL_API int msgl_route(const void* h, long long h_stride, const void* W, const float* correction, int H, int E, int n_groups, int keep,
-                        int top, int* idx, float* wts, int T_, int dtype, int softmax, const void* gate_row, float* gate_out,
-                        cudaStream_t stream) {
+                        int top, int* idx, float* wts, int T_, int dtype, int score, int group_max, int renorm, const void* gate_row,
+                        float* gate_out, cudaStream_t stream) {
     if (T_ <= 0) return MSGL_OK;
     if (H <= 0 || E <= 0 || E > RT_MAX_EXPERTS || n_groups < 1 || n_groups > RT_MAX_GROUPS || E % n_groups || keep < 1 || keep > n_groups ||
-        top < 1 || top > keep * (E / n_groups))
+        top < 1 || top > keep * (E / n_groups) || score < 0 || score > 2)
         return MSGL_ERR_SIZE;
     if (dtype != MSGL_F32 && dtype != MSGL_BF16) return MSGL_ERR_DTYPE;
     // whether rows can be read 16 bytes at a time: a matter of the sizes and of the weights' place, the same in every step of a model
@@ -1702,8 +1720,8 @@ MSGL_API int msgl_route(const void* h, long long h_stride, const void* W, const 
                     ((uintptr_t)gate_row % 16) == 0;
     if (gate_row && !gate_out) return MSGL_ERR_SIZE;
     const int threads = E > 4 ? 256 : 128;
-    if (dtype == MSGL_F32) route_kernel<float><<<T_, threads, 0, stream>>>((const float*)h, h_stride, (const float*)W, correction, H, E, n_groups, keep, top, idx, wts, vec, softmax, (const float*)gate_row, gate_out);
-    else route_kernel<__nv_bfloat16><<<T_, threads, 0, stream>>>((const __nv_bfloat16*)h, h_stride, (const __nv_bfloat16*)W, correction, H, E, n_groups, keep, top, idx, wts, vec, softmax, (const __nv_bfloat16*)gate_row, gate_out);
+    if (dtype == MSGL_F32) route_kernel<float><<<T_, threads, 0, stream>>>((const float*)h, h_stride, (const float*)W, correction, H, E, n_groups, keep, top, idx, wts, vec, score, group_max, renorm, (const float*)gate_row, gate_out);
+    else route_kernel<__nv_bfloat16><<<T_, threads, 0, stream>>>((const __nv_bfloat16*)h, h_stride, (const __nv_bfloat16*)W, correction, H, E, n_groups, keep, top, idx, wts, vec, score, group_max, renorm, (const __nv_bfloat16*)gate_row, gate_out);
     return msgl_check_launch();
 }
 
@@ -1778,12 +1796,98 @@ MSGL_API int msgl_experts_few(const void* h, long long h_stride, const void* Wgu
 }
 
 // ---------------------------------------------------------------------------------------
+// The same for experts without a gate, act_(t, k) = act(Wu[e] h_t), Wu [E][F][H], where a router output e >= E stands for the
+// input itself: it adds wts[t, k] * h_t.  A lane takes 16 bytes of a row at a time where the sizes allow it.
+//   out[t, c] = sum_k wts[t, k] * (e_k < E ? Wd[e_k][c] . act_(t, k) : h[t, c]) + extra[t, c]
+// ---------------------------------------------------------------------------------------
+template <typename T, bool VEC>
+__device__ __forceinline__ float lane_dot(const T* __restrict__ a, const T* __restrict__ b, int n, int lane) {
+    float acc = 0.f;
+    if (VEC) {
+        constexpr int V = VecOf<T>::N;
+#pragma unroll 4
+        for (int i = lane * V; i < n; i += 32 * V) {
+            float x[V], y[V];
+            VecOf<T>::load(a + i, x);
+            VecOf<T>::load(b + i, y);
+#pragma unroll
+            for (int k = 0; k < V; ++k) acc = fmaf(x[k], y[k], acc);
+        }
+    } else {
+        for (int i = lane; i < n; i += 32) acc = fmaf(to_f32<T>(a[i]), to_f32<T>(b[i]), acc);
+    }
+    return acc;
+}
+
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(256) expert_up_kernel(const T* __restrict__ h, long long h_stride, const T* __restrict__ Wu,
+                                                        const int* __restrict__ idx, int top, int E, int H, int F, int act,
+                                                        T* __restrict__ out) {
+    const int pair = blockIdx.y, t = pair / top;
+    const int r = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    const int e = idx[pair];
+    if (r >= F || e >= E) return;
+    const float acc = warp_sum(lane_dot<T, VEC>(Wu + ((size_t)e * F + r) * H, h + (size_t)t * h_stride, H, lane));
+    if (lane == 0) out[(size_t)pair * F + r] = from_f32<T>(act_of(act, acc));
+}
+
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(256) expert_down_plain_kernel(const T* __restrict__ act, const T* __restrict__ Wd, const int* __restrict__ idx,
+                                                                const float* __restrict__ wts, int top, int E, int H, int F,
+                                                                const T* __restrict__ h, long long h_stride,
+                                                                const float* __restrict__ extra, float* __restrict__ out) {
+    const int t = blockIdx.y;
+    const int c = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
+    if (c >= H) return;
+    float total = 0.f, self = 0.f;                       // total: this lane's share; self: the weight of the input itself
+    for (int k = 0; k < top; ++k) {
+        const int e = idx[(size_t)t * top + k];
+        const float w = wts[(size_t)t * top + k];
+        if (e >= E) { self += w; continue; }
+        total = fmaf(w, lane_dot<T, VEC>(Wd + ((size_t)e * H + c) * F, act + ((size_t)t * top + k) * F, F, lane), total);
+    }
+    total = warp_sum(total);
+    if (lane == 0) {
+        if (self != 0.f) total = fmaf(self, to_f32<T>(h[(size_t)t * h_stride + c]), total);
+        if (extra) total += extra[(size_t)t * H + c];
+        out[(size_t)t * H + c] = total;
+    }
+}
+
+MSGL_API int msgl_plain_experts_few(const void* h, long long h_stride, const void* Wu, const void* Wd, const int* idx, const float* wts,
+                                    int top, int E, int H, int F, int act_kind, void* act, const float* extra, float* out, int T_,
+                                    int dtype, cudaStream_t stream) {
+    if (T_ <= 0) return MSGL_OK;
+    if (top < 1 || H <= 0 || F <= 0 || E < 0 || act_kind < 0 || act_kind > 4) return MSGL_ERR_SIZE;
+    if (dtype != MSGL_F32 && dtype != MSGL_BF16) return MSGL_ERR_DTYPE;
+    const int V = dtype == MSGL_F32 ? 4 : 8;
+    // a matter of the sizes and of where the tensors lie, the same in every step of a model
+    const bool up_vec = H % V == 0 && h_stride % V == 0 && ((uintptr_t)h % 16) == 0 && ((uintptr_t)Wu % 16) == 0;
+    const bool dn_vec = F % V == 0 && ((uintptr_t)act % 16) == 0 && ((uintptr_t)Wd % 16) == 0;
+    const dim3 g1((F + 7) / 8, T_ * top), g2((H + 7) / 8, T_);
+#define PLAIN_UP(T, VEC) expert_up_kernel<T, VEC><<<g1, 256, 0, stream>>>((const T*)h, h_stride, (const T*)Wu, idx, top, E, H, F, act_kind, (T*)act)
+#define PLAIN_DN(T, VEC) expert_down_plain_kernel<T, VEC><<<g2, 256, 0, stream>>>((const T*)act, (const T*)Wd, idx, wts, top, E, H, F, (const T*)h, h_stride, extra, out)
+    if (dtype == MSGL_F32) {
+        if (up_vec) PLAIN_UP(float, true); else PLAIN_UP(float, false);
+        if (dn_vec) PLAIN_DN(float, true); else PLAIN_DN(float, false);
+    } else {
+        if (up_vec) PLAIN_UP(__nv_bfloat16, true); else PLAIN_UP(__nv_bfloat16, false);
+        if (dn_vec) PLAIN_DN(__nv_bfloat16, true); else PLAIN_DN(__nv_bfloat16, false);
+    }
+#undef PLAIN_UP
+#undef PLAIN_DN
+    return msgl_check_launch();
+}
+
+// ---------------------------------------------------------------------------------------
 // Many tokens: the (token, choice) pairs in the order of their experts
 //
 //   expert_count_kernel   counts[e] = pairs whose expert is e                                   (one block per expert)
 //   expert_place_kernel   place[pair] = row of the pair in expert order, stable within an expert  (one block per expert)
 //   expert_gather_kernel  rows[place[pair]] = h[token of the pair]
 //   expert_combine_kernel out[t] = c * sum_k wts[t, k] * y[place[t * top + k]] in float32
+// Pairs whose expert number is E or more (the input itself: `self_h`) have no row: place = -1, nothing gathered, and the
+// combination adds wts[t, k] * self_h[t].
 // ---------------------------------------------------------------------------------------
 __global__ void __launch_bounds__(256) expert_count_kernel(const int* __restrict__ idx, int n_pairs, int* __restrict__ counts) {
     __shared__ float scratch[32];
@@ -1795,10 +1899,15 @@ __global__ void __launch_bounds__(256) expert_count_kernel(const int* __restrict
 }
 
 __global__ void __launch_bounds__(256) expert_place_kernel(const int* __restrict__ idx, int n_pairs, const int* __restrict__ counts,
-                                                           int* __restrict__ place) {
+                                                           int n_experts, int* __restrict__ place) {
     __shared__ int warp_tot[8];
     __shared__ int base_sh;
     const int e = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+    if (e == n_experts) {                                // the last block: pairs whose expert has no rows
+        for (int i = tid; i < n_pairs; i += 256)
+            if (idx[i] >= n_experts) place[i] = -1;
+        return;
+    }
     if (tid == 0) {
         int b = 0;
         for (int i = 0; i < e; ++i) b += counts[i];
@@ -1824,9 +1933,80 @@ template <typename T>
 __global__ void expert_gather_kernel(const T* __restrict__ h, long long h_stride, const int* __restrict__ place, int top, int H,
                                      T* __restrict__ rows) {
     const int pair = blockIdx.x, t = pair / top;
+    const int at = place[pair];
+    if (at < 0) return;
     const T* src = h + (size_t)t * h_stride;
-    T* dst = rows + (size_t)place[pair] * H;
+    T* dst = rows + (size_t)at * H;
     for (int i = threadIdx.x; i < H; i += blockDim.x) dst[i] = src[i];
+}
+
+// 16 bytes a thread; H a multiple of the vector, rows on 16-byte boundaries
+template <typename T>
+__global__ void __launch_bounds__(128) expert_gather_vec_kernel(const T* __restrict__ h, long long h_stride, const int* __restrict__ place,
+                                                                int top, int H, T* __restrict__ rows) {
+    constexpr int V = VecOf<T>::N;
+    const int pair = blockIdx.x, t = pair / top;
+    const int at = place[pair];
+    if (at < 0) return;
+    const uint4* src = reinterpret_cast<const uint4*>(h + (size_t)t * h_stride);
+    uint4* dst = reinterpret_cast<uint4*>(rows + (size_t)at * H);
+    for (int i = threadIdx.x; i < H / V; i += blockDim.x) dst[i] = src[i];
+}
+
+// V elements a thread: 1, or 4 where the rows lie on 16-byte (float) resp. 8-byte (bfloat16) boundaries
+template <typename Y, int V> __device__ __forceinline__ void ex_load(const Y* p, float (&v)[V]) {
+    if constexpr (V == 1) v[0] = to_f32<Y>(p[0]);
+    else if constexpr (sizeof(Y) == 4) { const float4 a = *reinterpret_cast<const float4*>(p); v[0] = a.x; v[1] = a.y; v[2] = a.z; v[3] = a.w; }
+    else {
+        const uint2 a = *reinterpret_cast<const uint2*>(p);
+        const float2 f0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&a.x));
+        const float2 f1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&a.y));
+        v[0] = f0.x; v[1] = f0.y; v[2] = f1.x; v[3] = f1.y;
+    }
+}
+
+template <typename Y, typename S, int V>
+__global__ void __launch_bounds__(256) expert_combine_self_kernel(const Y* __restrict__ y, const int* __restrict__ place, const float* __restrict__ wts,
+                                                                  int top, int H, const S* __restrict__ self_h, long long self_stride,
+                                                                  const float* __restrict__ extra, float* __restrict__ out) {
+    const int t = blockIdx.x;
+    for (int i = (blockIdx.y * blockDim.x + threadIdx.x) * V; i < H; i += gridDim.y * blockDim.x * V) {
+        float acc[V], v[V];
+#pragma unroll
+        for (int k = 0; k < V; ++k) acc[k] = 0.f;
+        if (extra) ex_load<float, V>(extra + (size_t)t * H + i, acc);
+        for (int j = 0; j < top; ++j) {
+            const int at = place[(size_t)t * top + j];
+            const float w = wts[(size_t)t * top + j];
+            if (at >= 0) ex_load<Y, V>(y + (size_t)at * H + i, v);
+            else ex_load<S, V>(self_h + (size_t)t * self_stride + i, v);
+#pragma unroll
+            for (int k = 0; k < V; ++k) acc[k] = fmaf(w, v[k], acc[k]);
+        }
+        if constexpr (V == 4) *reinterpret_cast<float4*>(out + (size_t)t * H + i) = make_float4(acc[0], acc[1], acc[2], acc[3]);
+        else out[(size_t)t * H + i] = acc[0];
+    }
+}
+
+// y: rows in expert order, float32 or the activation type; self_h [T rows] of the activation type (`dtype`)
+MSGL_API int msgl_expert_combine_self(const void* y, int y_is_f32, const int* place, const float* wts, int top, int H, const void* self_h,
+                                      long long self_stride, const float* extra, float* out, int T_, int dtype, cudaStream_t stream) {
+    if (T_ <= 0) return MSGL_OK;
+    if (top < 1 || H <= 0 || self_h == nullptr) return MSGL_ERR_SIZE;
+    const uintptr_t all = (uintptr_t)y | (uintptr_t)self_h | (uintptr_t)extra | (uintptr_t)out;
+    const bool v4 = H % 4 == 0 && self_stride % 4 == 0 && (all & 15) == 0;
+    const int per = v4 ? 4 : 1;
+    const dim3 grid(T_, max(1, min((H + 256 * per - 1) / (256 * per), 16)));
+#define COMBINE(Y, S)                                                                                                        \
+    do {                                                                                                                     \
+        if (v4) expert_combine_self_kernel<Y, S, 4><<<grid, 256, 0, stream>>>((const Y*)y, place, wts, top, H, (const S*)self_h, self_stride, extra, out); \
+        else expert_combine_self_kernel<Y, S, 1><<<grid, 256, 0, stream>>>((const Y*)y, place, wts, top, H, (const S*)self_h, self_stride, extra, out);    \
+    } while (0)
+    if (dtype == MSGL_F32) COMBINE(float, float);
+    else if (dtype == MSGL_BF16) { if (y_is_f32) COMBINE(float, __nv_bfloat16); else COMBINE(__nv_bfloat16, __nv_bfloat16); }
+    else return MSGL_ERR_DTYPE;
+#undef COMBINE
+    return msgl_check_launch();
 }
 
 template <typename Y>
@@ -1847,13 +2027,19 @@ MSGL_API int msgl_expert_order(const int* idx, int n_pairs, int E, int* counts, 
     if (n_pairs <= 0) return MSGL_OK;
     if (E <= 0 || n_pairs >= (1 << 24)) return MSGL_ERR_SIZE;
     expert_count_kernel<<<E, 256, 0, stream>>>(idx, n_pairs, counts);
-    expert_place_kernel<<<E, 256, 0, stream>>>(idx, n_pairs, counts, place);
+    expert_place_kernel<<<E + 1, 256, 0, stream>>>(idx, n_pairs, counts, E, place);
     return msgl_check_launch();
 }
 
 MSGL_API int msgl_expert_gather(const void* h, long long h_stride, const int* place, int top, int H, void* rows, int n_pairs, int dtype,
                                 cudaStream_t stream) {
     if (n_pairs <= 0) return MSGL_OK;
+    const int V = dtype == MSGL_F32 ? 4 : 8;
+    if ((dtype == MSGL_F32 || dtype == MSGL_BF16) && H % V == 0 && h_stride % V == 0 && (((uintptr_t)h | (uintptr_t)rows) & 15) == 0) {
+        if (dtype == MSGL_F32) expert_gather_vec_kernel<float><<<n_pairs, 128, 0, stream>>>((const float*)h, h_stride, place, top, H, (float*)rows);
+        else expert_gather_vec_kernel<__nv_bfloat16><<<n_pairs, 128, 0, stream>>>((const __nv_bfloat16*)h, h_stride, place, top, H, (__nv_bfloat16*)rows);
+        return msgl_check_launch();
+    }
     if (dtype == MSGL_F32) expert_gather_kernel<float><<<n_pairs, 128, 0, stream>>>((const float*)h, h_stride, place, top, H, (float*)rows);
     else if (dtype == MSGL_BF16) expert_gather_kernel<__nv_bfloat16><<<n_pairs, 128, 0, stream>>>((const __nv_bfloat16*)h, h_stride, place, top, H, (__nv_bfloat16*)rows);
     else return MSGL_ERR_DTYPE;

@@ -327,7 +327,8 @@ class ModelRunner:
         self.last_plan: Dict[str, object] = {}       # the last step's kv splits per group and the decode graph it replayed
         self._group_geom = []
         for g in self.mgr.groups:
-            cid = g.cache_ids[0]
+            # the kv splits are planned for the caches whose launches take them: the first of the engine's attention kernels
+            cid = next((c for c in g.cache_ids if needs[c].library == "attention"), g.cache_ids[0])
             need = needs[cid]
             G = max(need.q_heads // need.n_kv_heads, 1) if need.q_heads else 1
             if need.library != "attention":

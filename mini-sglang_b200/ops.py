@@ -81,7 +81,7 @@ def _lib():
         lib.msgl_table_delta.argtypes = [c_void_p, c_int, c_void_p, c_int, c_void_p]
         lib.msgl_decode_meta.argtypes = [c_void_p] * 4 + [c_int, c_int, c_void_p, c_int, c_int, c_int, c_int] + [c_void_p] * 9 + [c_int, c_void_p, c_void_p, c_void_p, c_int,
                                          c_void_p]
-        lib.msgl_rmsnorm.argtypes = [c_void_p, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_float, c_void_p,
+        lib.msgl_rmsnorm.argtypes = [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_float, c_int, c_void_p,
                                      c_int, c_int, c_int, c_void_p]
         lib.msgl_qknorm_rope_kvwrite.argtypes = [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
                                                  c_float, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p,
@@ -171,10 +171,11 @@ def decode_meta(ids: torch.Tensor, slots_in: torch.Tensor, pos: torch.Tensor, ns
 def rmsnorm(weight: torch.Tensor, eps: float, *, x: Optional[torch.Tensor] = None,
             residual: Optional[torch.Tensor] = None, residual_out: Optional[torch.Tensor] = None,
             rows: Optional[torch.Tensor] = None, out_dtype: Optional[torch.dtype] = None,
-            out: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """y = rmsnorm(residual + x) * weight, the sum and the norm in float32.
+            out: Optional[torch.Tensor] = None, center: bool = False) -> torch.Tensor:
+    """y = rmsnorm(residual + x) * weight, the sum and the norm in float32; with `center` the row's mean is taken off first
+    (a layer norm without bias: the variance is the mean of the squared deviations).
 
-    x: activation dtype [N, H] or None; residual: float32 [N, H] or None; residual_out: float32
+    x: float32 or activation dtype [N, H] or None; residual: float32 [N, H] or None; residual_out: float32
     buffer that receives the sum (may be `residual` itself when `rows` is None);
     rows: int32 [R] picks input rows (outputs are then [R, H]).  Returns y in `out_dtype`
     (default: x's dtype)."""
@@ -186,16 +187,17 @@ def rmsnorm(weight: torch.Tensor, eps: float, *, x: Optional[torch.Tensor] = Non
     if out_dtype is None:
         out_dtype = x.dtype if x is not None else torch.float32
     if x is not None:
-        assert x.dtype == out_dtype
+        assert x.dtype in (out_dtype, torch.float32) and x.is_contiguous()
     if residual is not None:
         assert residual.dtype == torch.float32 and residual.shape[1] == H
     assert weight.numel() == H and weight.dtype in (torch.float32, torch.bfloat16)
     if out is None:
         out = torch.empty((n_out, H), dtype=out_dtype, device=src.device)
-    code = _lib().msgl_rmsnorm(_ptr(x), _ptr(residual), _ptr(residual_out), _ptr(rows), _ptr(weight),
-                               int(weight.dtype == torch.float32), float(eps), _ptr(out), n_out, H, _DT[out_dtype],
+    x_f32 = int(x is not None and x.dtype == torch.float32)
+    code = _lib().msgl_rmsnorm(_ptr(x), x_f32, _ptr(residual), _ptr(residual_out), _ptr(rows), _ptr(weight),
+                               int(weight.dtype == torch.float32), float(eps), int(bool(center)), _ptr(out), n_out, H, _DT[out_dtype],
                                _stream())
-    _check(code, "rmsnorm")
+    _check(code, "layernorm" if center else "rmsnorm")
     return out
 
 
@@ -661,7 +663,7 @@ def linear_swiglu(x: torch.Tensor, gate_up: torch.Tensor) -> torch.Tensor:
 # norms, convolutions, windowed and linear attention, gated activations (csrc/mixers.cu)
 # ---------------------------------------------------------------------------------------
 _mixers = None
-ACT_SILU, ACT_GELU_TANH, ACT_SIGMOID = 0, 1, 2
+ACT_SILU, ACT_GELU_TANH, ACT_SIGMOID, ACT_RELU2, ACT_RELU = 0, 1, 2, 3, 4
 WINDOW_ATTENTION_ROWS = 8         # (token, head) rows of a block of the windowed attention kernel
 CONV_MAX_TAPS = 16
 WINDOW_ATTENTION_MAX_HEAD_DIM = 512
@@ -875,8 +877,8 @@ def rms_gate(x: torch.Tensor, weight: torch.Tensor, eps: float, gate: Optional[t
 
 
 def gated_act(gate: torch.Tensor, up: torch.Tensor, out: torch.Tensor, act: int) -> None:
-    """out = act(gate) * up, act = ACT_SILU, ACT_GELU_TANH (0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)))) or ACT_SIGMOID;
-    all three [T, I] views into packed rows, gate and up in the same rows."""
+    """out = act(gate) * up, act = ACT_SILU, ACT_GELU_TANH (0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)))), ACT_SIGMOID,
+    ACT_RELU2 or ACT_RELU; all three [T, I] views into packed rows, gate and up in the same rows."""
     _need_cuda(gate, up, out)
     T, I = gate.shape
     stride = _rows_view(gate, I, "gate")
@@ -1040,7 +1042,6 @@ def group_rms_gate(x: torch.Tensor, heads: int, weight: torch.Tensor, eps: float
 # sigmoid attention, gated recurrences, state-space scan, routed experts (csrc/mixers_gated.cu)
 # ---------------------------------------------------------------------------------------
 _gated = None
-ACT_RELU2, ACT_RELU = 3, 4
 SIGMOID_ATTENTION_ROWS = 8          # (token, head) rows of a block of the sigmoid attention kernel
 SIGMOID_ATTENTION_MAX_HEAD_DIM = 512
 MINGRU_CHUNK = 32                   # tokens of a chunk when a long portion's recurrence runs in chunks side by side
@@ -1077,8 +1078,10 @@ def _gated_lib():
         lib.msgl_gate_group_norm.argtypes = [c_void_p, c_int, c_int, c_void_p, c_float, c_void_p, c_ll, c_void_p, c_ll, c_float, c_int,
                                              c_int, c_void_p]
         lib.msgl_unary_act.argtypes = [c_void_p, c_ll, c_void_p, c_ll, c_int, c_int, c_float, c_int, c_int, c_void_p]
-        lib.msgl_route.argtypes = [c_void_p, c_ll, c_void_p, c_void_p] + [c_int] * 5 + [c_void_p, c_void_p, c_int, c_int, c_int, c_void_p,
-                                   c_void_p, c_void_p]
+        lib.msgl_route.argtypes = [c_void_p, c_ll, c_void_p, c_void_p] + [c_int] * 5 + [c_void_p, c_void_p] + [c_int] * 5 + [c_void_p] * 3
+        lib.msgl_plain_experts_few.argtypes = [c_void_p, c_ll] + [c_void_p] * 4 + [c_int] * 5 + [c_void_p] * 3 + [c_int, c_int, c_void_p]
+        lib.msgl_expert_combine_self.argtypes = [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_void_p, c_ll, c_void_p, c_void_p, c_int,
+                                                 c_int, c_void_p]
         lib.msgl_experts_few.argtypes = [c_void_p, c_ll] + [c_void_p] * 4 + [c_int, c_int, c_int, c_void_p, c_float, c_void_p, c_int, c_int,
                                                                             c_float, c_void_p, c_void_p, c_void_p]
         lib.msgl_clamped_glu.argtypes = [c_void_p, c_ll, c_int, c_float, c_void_p, c_int, c_int, c_void_p]
@@ -1331,19 +1334,25 @@ def unary_act(x: torch.Tensor, act: int, scale: float = 1.0, out: Optional[torch
     return out
 
 
+ROUTE_SCORES = {"sigmoid": 0, "logits": 1, "softmax": 2}
+
+
 def route(h: torch.Tensor, router: torch.Tensor, correction: Optional[torch.Tensor], *, n_groups: int, keep: int,
-          top: int, softmax: bool = False, gate_row: Optional[torch.Tensor] = None):
-    """The experts a token uses and their weights.  Scores s = sigmoid(router h) with float32 sums; the choice goes by s +
-    correction among the experts of the `keep` best of `n_groups` equal groups of neighbouring experts (a group counts by the sum
-    of its two largest choice scores), the `top` largest win; the weights are the winners' s over their sum.
+          top: int, score: str = "sigmoid", group_score: str = "top2", renormalize: bool = True,
+          gate_row: Optional[torch.Tensor] = None):
+    """The experts a token uses and their weights.  Scores s = sigmoid(router h), or with score = "softmax" the softmax of the
+    logits over all E outputs, in float32; the choice goes by s + correction among the experts of the `keep` best of `n_groups`
+    equal groups of neighbouring experts (a group counts by the sum of its two largest choice scores, or with group_score = "max"
+    by the largest), the `top` largest win; the weights are the winners' s, over their sum unless renormalize = False.
     h [T, H], router [E, H] -> (int32 [T, top], float32 [T, top]).
-    softmax: the logits router h themselves are what the choice goes by (the largest win, the lower index at a tie), and the
-    weights are the softmax over the chosen logits only.  gate_row [H]: one more row that is no expert; the call then returns
-    a third tensor, float32 [T] = sigmoid(gate_row . h)."""
+    score = "logits": the logits router h themselves are what the choice goes by (the largest win, the lower index at a tie), and
+    the weights are the softmax over the chosen logits only.  gate_row [H]: one more row that is no expert.  With either of
+    the two the call returns a third item, float32 [T] = sigmoid(gate_row . h) or None."""
     _need_cuda(h, router, correction, gate_row)
     T, H = h.shape
     E = router.shape[0]
     assert router.shape == (E, H) and router.is_contiguous() and router.dtype == h.dtype
+    assert group_score in ("top2", "max")
     if correction is not None:
         assert correction.dtype == torch.float32 and correction.numel() == E
     idx = torch.empty((T, top), dtype=torch.int32, device=h.device)
@@ -1353,11 +1362,52 @@ def route(h: torch.Tensor, router: torch.Tensor, correction: Optional[torch.Tens
         assert gate_row.dtype == h.dtype and gate_row.numel() == H and gate_row.is_contiguous()
         gate_out = torch.empty(T, dtype=torch.float32, device=h.device)
     code = _gated_lib().msgl_route(_ptr(h), _rows_view(h, H, "h"), _ptr(router), _ptr(correction), H, E, int(n_groups), int(keep),
-                                   int(top), _ptr(idx), _ptr(wts), T, _dt(h), int(bool(softmax)), _ptr(gate_row), _ptr(gate_out), _stream())
+                                   int(top), _ptr(idx), _ptr(wts), T, _dt(h), ROUTE_SCORES[score], int(group_score == "max"),
+                                   int(bool(renormalize)), _ptr(gate_row), _ptr(gate_out), _stream())
     _check(code, f"route ({E} experts)")
-    if softmax or gate_row is not None:
+    if score == "logits" or gate_row is not None:
         return idx, wts, gate_out
     return idx, wts
+
+
+def plain_experts_few(h: torch.Tensor, up: torch.Tensor, down: torch.Tensor, idx: torch.Tensor, wts: torch.Tensor, act: int,
+                      extra: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """-> float32 [T, H] = sum_k wts[t, k] * y_k + extra[t] for experts without a gate: y_k = down[e] act(up[e] h_t), e = idx[t, k],
+    the chosen experts' rows read straight from the stacked weights up [E, F, H] and down [E, H, F]; e >= E stands for the input
+    itself, y_k = h_t.  For a few tokens.  act: one of the ACT_ numbers; extra: float32 [T, H] (a shared expert's output)."""
+    _need_cuda(h, up, down, idx, wts, extra)
+    T, H = h.shape
+    E, F, _ = up.shape
+    top = idx.shape[1]
+    assert up.shape == (E, F, H) and down.shape == (E, H, F) and up.is_contiguous() and down.is_contiguous()
+    assert up.dtype == down.dtype == h.dtype
+    assert idx.dtype == torch.int32 and wts.dtype == torch.float32 and idx.is_contiguous() and wts.is_contiguous()
+    if extra is not None:
+        assert extra.dtype == torch.float32 and extra.is_contiguous() and tuple(extra.shape) == (T, H)
+    a = torch.empty((T * top, F), dtype=h.dtype, device=h.device)
+    out = torch.empty((T, H), dtype=torch.float32, device=h.device)
+    code = _gated_lib().msgl_plain_experts_few(_ptr(h), _rows_view(h, H, "h"), _ptr(up), _ptr(down), _ptr(idx), _ptr(wts), top, E, H, F,
+                                               int(act), _ptr(a), _ptr(extra), _ptr(out), T, _dt(h), _stream())
+    _check(code, "plain_experts_few")
+    global LAUNCHES
+    LAUNCHES += 1
+    return out
+
+
+def expert_combine_self(y: torch.Tensor, place: torch.Tensor, wts: torch.Tensor, h: torch.Tensor,
+                        extra: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """-> float32 [T, H] = extra[t] + sum_k wts[t, k] * (y[place[t * top + k]], or h[t] where that place is -1)."""
+    _need_cuda(y, place, wts, h, extra)
+    T, top = wts.shape
+    H = y.shape[1]
+    assert y.is_contiguous() and y.dtype in (torch.float32, h.dtype) and wts.dtype == torch.float32 and wts.is_contiguous()
+    assert h.shape == (T, H) and place.numel() == T * top
+    if extra is not None:
+        assert extra.dtype == torch.float32 and extra.is_contiguous() and tuple(extra.shape) == (T, H)
+    out = torch.empty((T, H), dtype=torch.float32, device=y.device)
+    _check(_gated_lib().msgl_expert_combine_self(_ptr(y), int(y.dtype == torch.float32), _ptr(place), _ptr(wts), top, H, _ptr(h),
+                                                 _rows_view(h, H, "h"), _ptr(extra), _ptr(out), T, _dt(h), _stream()), "expert_combine_self")
+    return out
 
 
 def experts_few(h: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, idx: torch.Tensor, wts: torch.Tensor,
@@ -1391,7 +1441,8 @@ def experts_few(h: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, idx:
 
 def expert_order(idx: torch.Tensor, n_experts: int) -> Tuple[torch.Tensor, torch.Tensor]:
     """idx int32 [T, top] -> (counts int32 [E]: pairs per expert; place int32 [T * top]: row of every (token, choice) pair when the
-    pairs are put in the order of their experts, pairs of one expert in their own order)."""
+    pairs are put in the order of their experts, pairs of one expert in their own order; -1 for a pair whose number is n_experts
+    or more, which has no row)."""
     _need_cuda(idx)
     assert idx.dtype == torch.int32 and idx.is_contiguous()
     counts = torch.empty(n_experts, dtype=torch.int32, device=idx.device)
@@ -1403,7 +1454,7 @@ def expert_order(idx: torch.Tensor, n_experts: int) -> Tuple[torch.Tensor, torch
 
 
 def expert_gather(h: torch.Tensor, place: torch.Tensor, top: int) -> torch.Tensor:
-    """rows[place[t * top + k]] = h[t]: every token's row once per expert it uses, in expert order."""
+    """rows[place[t * top + k]] = h[t]: every token's row once per expert it uses, in expert order (places below 0: no row)."""
     _need_cuda(h, place)
     T, H = h.shape
     rows = torch.empty((T * top, H), dtype=h.dtype, device=h.device)
@@ -1457,11 +1508,12 @@ def _delta_lib():
         lib = _build.delta_mixers_library()
         lib.msgl_scaled_add_norm.argtypes = [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_int, c_void_p]
         lib.msgl_rotary_angles.argtypes = [c_void_p, c_void_p, ctypes.c_double, c_void_p, c_int, c_int, c_void_p]
-        lib.msgl_sink_qkv_prep.argtypes = [c_void_p, c_ll, c_void_p, c_int, c_void_p, c_ll, c_float] + [c_void_p] * 4 + [c_int] * 7 + [c_void_p]
+        lib.msgl_sink_qkv_prep.argtypes = [c_void_p, c_ll, c_void_p, c_int, c_void_p, c_ll, c_float] + [c_void_p] * 4 + [c_int] * 7 + \
+            [c_void_p, c_void_p, c_int, c_float, c_void_p]
         lib.msgl_sink_attention.argtypes = [c_void_p] * 6 + [c_int, c_int, c_int, c_void_p, c_void_p, c_ll, c_void_p, c_void_p] + \
-            [c_int] * 12 + [c_float, c_float, c_int, c_void_p]
+            [c_int] * 12 + [c_float, c_float, c_int, c_void_p, c_ll, c_void_p]
         lib.msgl_sink_attention_mma.argtypes = [c_void_p] * 6 + [c_int, c_int, c_int, c_void_p, c_void_p, c_ll, c_void_p, c_void_p] + \
-            [c_int] * 10 + [c_float, c_float, c_void_p]
+            [c_int] * 10 + [c_float, c_float, c_void_p, c_ll, c_void_p]
         lib.msgl_delta_rule.argtypes = [c_void_p, c_void_p, c_ll, c_int, c_int] + [c_void_p] * 7 + [c_int] * 7 + [c_void_p]
         lib.msgl_delta_rule_scratch.argtypes = [c_int] * 4
         lib.msgl_delta_rule_scratch.restype = c_ll
@@ -1501,11 +1553,13 @@ def rotary_angles(positions: torch.Tensor, freq: torch.Tensor, magnitude: float,
 
 def sink_qkv_prep(proj: torch.Tensor, *, n_q: int, n_kv: int, d: int, dv: int, angles: Optional[torch.Tensor],
                   v_first: Optional[torch.Tensor], lam: float, out_loc: Optional[torch.Tensor], k_cache: Optional[torch.Tensor],
-                  v_cache: Optional[torch.Tensor], page_size: int) -> torch.Tensor:
-    """proj [T, >= n_q * d + n_kv * d + n_kv * dv] packed rows [q | k | v | ...].  The first angles.shape[1] elements of every q and
+                  v_cache: Optional[torch.Tensor], page_size: int, q_norm: Optional[torch.Tensor] = None,
+                  k_norm: Optional[torch.Tensor] = None, v_unit: bool = False, eps: float = 0.0) -> torch.Tensor:
+    """proj [T, >= n_q * d + n_kv * d + n_kv * dv] packed rows [q | k | v | ...].  Where weights are given (q_norm, k_norm float32
+    [d], one for all heads) every q and k head is RMS-normed by itself first; the first angles.shape[1] elements of every q and
     k head turn in halves (element i against i + rot / 2) by `angles` float32 [T, rot] = cos | sin of the tokens' positions; v
-    becomes (1 - lam) v + lam v_first where `v_first` [T, n_kv * dv] (a view into packed rows) is given; k goes to `k_cache`
-    [pages, n_kv, page, d] and v to `v_cache` [pages, n_kv, page, dv] at token slots `out_loc`; the q rows come back as [T, n_q, d]."""
+    becomes (1 - lam) v + lam v_first where `v_first` [T, n_kv * dv] (a view into packed rows) is given, and with
+    v_unit every v head is then divided by its root mean square (eps inside the root); k goes to `k_cache` [pages, n_kv, page, d] and v to `v_cache` [pages, n_kv, page, dv] at token slots `out_loc`; the q rows come back as [T, n_q, d]."""
     _need_cuda(proj, angles, v_first, out_loc, k_cache, v_cache)
     T = proj.shape[0]
     width = (n_q + n_kv) * d + n_kv * dv
@@ -1523,9 +1577,15 @@ def sink_qkv_prep(proj: torch.Tensor, *, n_q: int, n_kv: int, d: int, dv: int, a
         assert k_cache.dtype == proj.dtype and v_cache.dtype == proj.dtype and k_cache.is_contiguous() and v_cache.is_contiguous()
         assert tuple(k_cache.shape[1:]) == (n_kv, page_size, d) and tuple(v_cache.shape[1:]) == (n_kv, page_size, dv)
         assert out_loc is not None and out_loc.dtype == torch.int32 and out_loc.numel() >= T
+    assert (q_norm is None) == (k_norm is None)
+    if q_norm is not None:
+        assert q_norm.dtype == k_norm.dtype == torch.float32 and q_norm.numel() == k_norm.numel() == d
+        assert q_norm.is_contiguous() and k_norm.is_contiguous()
+        _need_cuda(q_norm, k_norm)
     q_out = torch.empty((T, n_q, d), dtype=proj.dtype, device=proj.device)
     code = _delta_lib().msgl_sink_qkv_prep(_ptr(proj), stride, _ptr(angles), rot, _ptr(v_first), vf_stride, float(lam), _ptr(out_loc),
-                                           _ptr(q_out), _ptr(k_cache), _ptr(v_cache), page_size, n_q, n_kv, d, dv, T, _dt(proj), _stream())
+                                           _ptr(q_out), _ptr(k_cache), _ptr(v_cache), page_size, n_q, n_kv, d, dv, T, _dt(proj), _ptr(q_norm), _ptr(k_norm),
+                                           int(bool(v_unit)), float(eps), _stream())
     _check(code, "sink_qkv_prep")
     return q_out
 
@@ -1557,7 +1617,7 @@ def sink_attention_splits(table_width: int, page_size: int, window: int) -> int:
 def sink_attention(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, *, q_start: torch.Tensor,
                    kv_len: torch.Tensor, block_table: torch.Tensor, n_kv: int, page_size: int, scale: float, softcap: float,
                    window: int, sink: torch.Tensor, q_lens: Optional[Sequence[int]], workspace=None,
-                   tensor_cores: Optional[bool] = None) -> None:
+                   tensor_cores: Optional[bool] = None, gate: Optional[torch.Tensor] = None) -> None:
     """Causal softmax attention over the paged cache: the query at position i sees the keys j <= i with i - j < window (window 0:
     all), score = q . k * scale, capped as softcap * tanh(score / softcap) where softcap > 0, and every softmax's denominator
     holds exp(sink[head]) besides the seen keys' terms.  q [T, heads, d]; K cache [pages, n_kv, page, d], V cache [pages, n_kv,
@@ -1565,16 +1625,22 @@ def sink_attention(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_
     size the launch), or None when every request brings one token: the keys are then cut into pieces of
     SINK_ATTENTION_SPLIT_KEYS for blocks of their own, joined in order by a second kernel (workspace: a parts.Workspace for
     the pieces).  tensor_cores: None = the bfloat16 kernel with mma products where it takes the sizes
-    (`sink_attention_on_tensor_cores`), the float32-arithmetic one elsewhere; False = the float32-arithmetic kernel in any case."""
-    _need_cuda(q, out, k_cache, v_cache, q_start, kv_len, block_table, sink)
+    (`sink_attention_on_tensor_cores`), the float32-arithmetic one elsewhere; False = the float32-arithmetic kernel in any case.
+    gate [T, heads * dv] (a view into packed rows): the output is multiplied by sigmoid(gate), element by element."""
+    _need_cuda(q, out, k_cache, v_cache, q_start, kv_len, block_table, sink, gate)
     T, n_q, d = q.shape
     dv = v_cache.shape[3]
     assert q.is_contiguous() and k_cache.dtype == q.dtype and v_cache.dtype == q.dtype and out.dtype == q.dtype
     assert sink.dtype == torch.float32 and sink.numel() == n_q
     out_stride = _rows_view(out, n_q * dv, "out")
+    gate_stride = 0
+    if gate is not None:
+        assert gate.dtype == q.dtype and gate.shape[0] == T
+        gate_stride = _rows_view(gate, n_q * dv, "gate")
     B = kv_len.numel()
     if tensor_cores is None:
-        tensor_cores = sink_attention_on_tensor_cores(q.dtype, d, dv) and out_stride % 2 == 0 and out.data_ptr() % 4 == 0
+        tensor_cores = sink_attention_on_tensor_cores(q.dtype, d, dv) and out_stride % 2 == 0 and out.data_ptr() % 4 == 0 and \
+            gate_stride % 2 == 0 and (gate is None or gate.data_ptr() % 4 == 0)
     QT, GH = sink_attention_geometry(n_q, n_kv, tensor_cores)
     uniform = q_lens is None
     n_tiles = B if uniform else sum(-(-n // QT) for n in q_lens)
@@ -1592,12 +1658,12 @@ def sink_attention(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_
         code = _delta_lib().msgl_sink_attention_mma(
             _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(q_start), _ptr(kv_len), _ptr(block_table), block_table.stride(0), int(uniform),
             n_tiles, _ptr(sink), _ptr(out), out_stride, _ptr(part_o), _ptr(part_ml), splits, SINK_ATTENTION_SPLIT_KEYS, T, B, n_q, n_kv, d,
-            dv, page_size, int(window), float(scale), float(softcap), _stream())
+            dv, page_size, int(window), float(scale), float(softcap), _ptr(gate), gate_stride, _stream())
     else:
         code = _delta_lib().msgl_sink_attention(
             _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(q_start), _ptr(kv_len), _ptr(block_table), block_table.stride(0), int(uniform),
             n_tiles, _ptr(sink), _ptr(out), out_stride, _ptr(part_o), _ptr(part_ml), splits, SINK_ATTENTION_SPLIT_KEYS, T, B, n_q, n_kv, d,
-            dv, page_size, QT, GH, int(window), float(scale), float(softcap), _dt(q), _stream())
+            dv, page_size, QT, GH, int(window), float(scale), float(softcap), _dt(q), _ptr(gate), gate_stride, _stream())
     _check(code, f"sink_attention (head sizes {d}, {dv})")
     if splits > 1:
         global LAUNCHES

@@ -20,7 +20,8 @@ class LatentAttention(Mixer):
     q = Wq x, or through a latent of its own: q = Wuq rmsnorm(Wdq x) (`q_rank`); per head [key_dim | rot_dim].
     Wdkv x has kv_rank + rot_dim rows: the first kv_rank, RMS-normed, are the latent c; the last rot_dim are the rotated key
     part.  Per head k = Wuk_h c, v = Wuv_h c; score = (q_plain . k + q_rot . k_rot) * scale; causal, optionally only the last
-    `window` keys; softmax; optionally the heads side by side times sigmoid(Wg x); output projection.
+    `window` keys; softmax; optionally the heads side by side times sigmoid(Wg x), element by element or with one number per
+    head; output projection.
 
     Computed with the up-projections folded into the query and the output: score = (Wuk_h^T q_plain | q_rot) . (c | k_rot), so a
     token's cache row [c | k_rot] is key and value at once for all heads (one kv head of size kv_rank + rot_dim, its values the
@@ -28,7 +29,7 @@ class LatentAttention(Mixer):
     attention kernels return.  The attention launches are the paged ones every other softmax mixer of the engine uses.
 
     params: hidden_size, num_heads, key_dim, rot_dim (0: no rotated part), value_dim, kv_rank, q_rank (None: no query latent),
-            scale, window (None: all keys), gate (None | "sigmoid"), norm_eps, names.  The position encoding (a part with
+            scale, window (None: all keys), gate (None | "sigmoid" | "head_sigmoid"), norm_eps, names.  The position encoding (a part with
             `inv_freq`, `magnitude`, `rotary_dim`) comes from the layer.
     """
 
@@ -43,8 +44,9 @@ class LatentAttention(Mixer):
         self.scale = float(s["scale"])
         self.window = int(s["window"]) if s.get("window") else None
         self.gate = s.get("gate")
-        if self.gate not in (None, "sigmoid"):
-            raise ValueError(f"unknown output gate {self.gate!r}; known: sigmoid")
+        if self.gate not in (None, "sigmoid", "head_sigmoid"):
+            raise ValueError(f"unknown output gate {self.gate!r}; known: sigmoid, head_sigmoid")
+        self.gate_w = {None: 0, "sigmoid": self.H * self.dv, "head_sigmoid": self.H}[self.gate]
         self.eps = float(s["norm_eps"])
         self.position = position if self.rd else None
         if self.rd and (position is None or not hasattr(position, "inv_freq")):
@@ -75,7 +77,7 @@ class LatentAttention(Mixer):
         else:
             t[n["q"]] = TensorDecl((qd, self.E))
         if self.gate:
-            t[n["gate"]] = TensorDecl((self.H * self.dv, self.E))
+            t[n["gate"]] = TensorDecl((self.gate_w, self.E))
         return t
 
     def load(self, src) -> None:
@@ -124,7 +126,9 @@ class LatentAttention(Mixer):
         # the value up-projection on what the heads gathered of the latent
         heads = torch.empty((T, H * self.dv), dtype=x.dtype, device=x.device)
         torch.bmm(of[:, :, :r].transpose(0, 1), self.w_uvT, out=heads.view(T, H, self.dv).transpose(0, 1))
-        if self.gate:
-            g0 = self.q_w + r + rd
-            ops.gate_mul(proj[:, g0:g0 + H * self.dv], heads, heads, ops.ACT_SIGMOID)
+        g0 = self.q_w + r + rd
+        if self.gate == "sigmoid":
+            ops.gate_mul(proj[:, g0:g0 + self.gate_w], heads, heads, ops.ACT_SIGMOID)
+        elif self.gate == "head_sigmoid":
+            ops.head_gate(heads.view(T, H, self.dv), proj[:, g0:g0 + H], heads)
         return ops.linear(heads, self.w_o)

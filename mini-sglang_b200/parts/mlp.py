@@ -38,14 +38,15 @@ class SwiGLUMLP(FeedForward):
         return {"kind": "swiglu_mlp", "gate_up": self.gate_up, "down": self.down, "H": self.H, "I": self.I}
 
 
-ACTIVATIONS = {"silu": ops.ACT_SILU, "gelu_tanh": ops.ACT_GELU_TANH}
+ACTIVATIONS = {"silu": ops.ACT_SILU, "gelu_tanh": ops.ACT_GELU_TANH, "relu": ops.ACT_RELU, "relu2": ops.ACT_RELU2}
 
 
 @register_feed_forward("gated_mlp")
 class GatedMLP(FeedForward, Projected):
-    """down(act(gate(x)) * up(x)), dense, no biases, with act = "silu" or "gelu_tanh" (0.5 z (1 + tanh(sqrt(2/pi) (z +
-    0.044715 z^3)))).  gate and up are packed row-wise into one [2I, H] matrix.  params: hidden_size, intermediate_size,
-    activation, names (what the checkpoint calls gate, up and down below the part's prefix; default "gate_proj.weight" ...)."""
+    """down(act(gate(x)) * up(x)), dense, with act = "silu", "gelu_tanh" (0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)))),
+    "relu" or "relu2" (its square); with `bias` all three projections have one.  gate and up are packed row-wise into one
+    [2I, H] matrix.  params: hidden_size, intermediate_size, activation, bias, names (what the checkpoint calls gate, up, down
+    and their biases gate_bias, up_bias, down_bias below the part's prefix; default "gate_proj.weight", "gate_proj.bias" ...)."""
 
     def __init__(self, spec, prefix, env):
         super().__init__(spec, prefix, env)
@@ -57,17 +58,31 @@ class GatedMLP(FeedForward, Projected):
         names = spec.get("names") or {}
         self.n_gate, self.n_up, self.n_down = (self.name(names.get(k, d)) for k, d in
                                                 (("gate", "gate_proj.weight"), ("up", "up_proj.weight"), ("down", "down_proj.weight")))
-        self.gate_up = self.down = None
+        self.bias = bool(spec.get("bias", False))
+        self.n_gate_b, self.n_up_b, self.n_down_b = (self.name(names.get(k, d)) for k, d in
+                                                      (("gate_bias", "gate_proj.bias"), ("up_bias", "up_proj.bias"),
+                                                       ("down_bias", "down_proj.bias")))
+        self.gate_up = self.down = self.gate_up_b = self.down_b = None
 
     def tensors(self) -> Dict[str, TensorDecl]:
-        return {self.n_gate: TensorDecl((self.I, self.H)), self.n_up: TensorDecl((self.I, self.H)),
-                self.n_down: TensorDecl((self.H, self.I))}
+        t = {self.n_gate: TensorDecl((self.I, self.H)), self.n_up: TensorDecl((self.I, self.H)),
+             self.n_down: TensorDecl((self.H, self.I))}
+        if self.bias:
+            t[self.n_gate_b] = TensorDecl((self.I,), kind="vector", std=0.1)
+            t[self.n_up_b] = TensorDecl((self.I,), kind="vector", std=0.1)
+            t[self.n_down_b] = TensorDecl((self.H,), kind="vector", std=0.1)
+        return t
 
     def load(self, src) -> None:
         self.gate_up = torch.cat((src.fetch(self.n_gate), src.fetch(self.n_up)), dim=0).contiguous()
         self.down = src.fetch(self.n_down).contiguous()
+        if self.bias:
+            self.gate_up_b = torch.cat((src.fetch(self.n_gate_b), src.fetch(self.n_up_b))).to(self.env.dtype).contiguous()
+            self.down_b = src.fetch(self.n_down_b).to(self.env.dtype).contiguous()
 
     def in_weight(self):
+        if self.bias:
+            raise ValueError("a feed-forward with biases is not stacked with other products")
         return self.gate_up
 
     def out_weight(self):
@@ -78,9 +93,12 @@ class GatedMLP(FeedForward, Projected):
         ops.gated_act(proj[:, :self.I], proj[:, self.I:2 * self.I], act, self.act)
 
     def forward(self, x, ctx):
-        if self.act == ops.ACT_SILU:        # product and activation in one kernel where the engine has it (few rows; many rows in bfloat16)
+        if self.act == ops.ACT_SILU and not self.bias:        # product and activation in one kernel where the engine has it (few rows; many rows in bfloat16)
             return ops.linear(ops.linear_swiglu(x, self.gate_up), self.down)
-        return self.forward_projected(x, ctx)
+        gu = ops.linear(x, self.gate_up, self.gate_up_b)
+        a = torch.empty((x.shape[0], self.I), dtype=x.dtype, device=x.device)
+        ops.gated_act(gu[:, :self.I], gu[:, self.I:], a, self.act)
+        return ops.linear(a, self.down, self.down_b)
 
 
 UNARY_ACTIVATIONS = {"silu": ops.ACT_SILU, "gelu_tanh": ops.ACT_GELU_TANH, "relu2": ops.ACT_RELU2, "relu": ops.ACT_RELU}

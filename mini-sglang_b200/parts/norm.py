@@ -35,6 +35,19 @@ class RMSNorm(Norm):
         return {"kind": "rmsnorm", "weight": self.weight, "eps": self.eps, "size": self.size}
 
 
+@register_norm("layernorm")
+class LayerNorm(RMSNorm):
+    """y = (v - mean(v)) / sqrt(mean((v - mean(v))^2) + eps) * weight with v = residual + x, in float32; a weight, no bias.
+    params as `rmsnorm`."""
+
+    def forward(self, x=None, residual=None, residual_out=None, rows=None):
+        return ops.rmsnorm(self.weight, self.eps, x=x, residual=residual, residual_out=residual_out, rows=rows,
+                           out_dtype=self.env.dtype, center=True)
+
+    def fused_decode_fields(self):
+        return None
+
+
 @register_norm("dynamic_tanh")
 class DynamicTanh(Norm):
     """y = tanh(alpha * v) * weight + bias with v = residual + x in float32, element by element: a norm that takes no mean

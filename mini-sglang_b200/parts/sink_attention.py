@@ -19,8 +19,13 @@ class SinkAttention(Mixer):
     position encoding turns the first elements of every q and k head (a partial rotation in halves; v is not turned);
     score(i, j) = q_i . k_j * scale, then cap * tanh(score / cap) where the part has a `softcap`; the query at i sees the keys
     j <= i with i - j < window (all earlier keys without a window); weights = exp(score) / (sum_seen exp(score) + exp(sink_h))
-    with a learned number per head that has no key and no value, is neither scaled nor capped and counts once; output
-    projection on the heads side by side.
+    with a learned number per head that has no key and no value, is neither scaled nor capped and counts once (`sink` gives
+    all heads one fixed number instead); optionally the heads side by side times sigmoid(Wg x), element by element (`gate`);
+    output projection.
+
+    Optionally (`qk_norm`) every q and k head is RMS-normed by itself before the rotation, with one weight of key_dim for all
+    q heads and one for all k heads, and (`value_norm`) every value head is divided by its root mean square, without a weight,
+    and cached so.
 
     Blended values (`value_mix`): the first layer of a model that has it ("first") hands its values of the step's tokens on
     under `value_mix_key`; a later layer ("blend") caches and reads v <- (1 - lambda) v + lambda v_first with a learned number
@@ -30,7 +35,8 @@ class SinkAttention(Mixer):
     bfloat16 the rotated q and k, the (blended) v as cached and the weights as operands of the value product are rounded.
 
     params: hidden_size, num_heads, num_kv_heads, key_dim, value_dim, scale, window (None: all keys), softcap (None: none),
-            bias, value_mix (None, "first", "blend"), value_mix_key, names (q, k, v, q_bias, k_bias, v_bias, sink, mix, out).
+            bias, value_mix (None, "first", "blend"), value_mix_key, sink (None: learned), qk_norm, value_norm, norm_eps,
+            gate (None, "sigmoid"), names (q, k, v, q_bias, k_bias, v_bias, sink, mix, q_norm, k_norm, gate, out).
     """
 
     graph_safe = True
@@ -51,20 +57,33 @@ class SinkAttention(Mixer):
         self.value_mix, self.value_mix_key = s.get("value_mix"), s.get("value_mix_key", "first_values")
         if self.value_mix not in (None, "first", "blend"):
             raise ValueError(f"value_mix {self.value_mix!r}: None, 'first' or 'blend'")
+        self.fixed_sink = float(s["sink"]) if s.get("sink") is not None else None
+        self.qk_norm, self.value_norm, self.eps = bool(s.get("qk_norm", False)), bool(s.get("value_norm", False)), float(s.get("norm_eps", 0.0))
+        self.gate = s.get("gate")
+        if self.gate not in (None, "sigmoid"):
+            raise ValueError(f"unknown output gate {self.gate!r}; known: sigmoid")
         self.position = position
         if position is not None and not hasattr(position, "step_angles"):
             raise ValueError("this mixer takes a position encoding that makes the angles of a step's positions (step_angles)")
-        names = {"q": "q", "k": "k", "v": "v", "q_bias": "q.b", "k_bias": "k.b", "v_bias": "v.b", "sink": "sink", "mix": "vmix", "out": "o"}
+        names = {"q": "q", "k": "k", "v": "v", "q_bias": "q.b", "k_bias": "k.b", "v_bias": "v.b", "sink": "sink", "mix": "vmix",
+                 "q_norm": "q.norm", "k_norm": "k.norm", "gate": "g", "out": "o"}
         names.update(s.get("names") or {})
         self.names = {k: self.name(v) for k, v in names.items()}
         self.Cq, self.Ck, self.Cv = self.n_q * self.d, self.n_kv * self.d, self.n_kv * self.dv
-        self.w_in = self.b_in = self.w_out = self.sink = None
+        self.w_in = self.b_in = self.w_out = self.sink = self.q_norm = self.k_norm = None
         self.lam = 0.0
 
     def tensors(self) -> Dict[str, TensorDecl]:
         n = self.names
         t = {n["q"]: TensorDecl((self.Cq, self.E)), n["k"]: TensorDecl((self.Ck, self.E)), n["v"]: TensorDecl((self.Cv, self.E)),
-             n["sink"]: TensorDecl((self.n_q,), kind="vector", std=1.0), n["out"]: TensorDecl((self.E, self.n_q * self.dv))}
+             n["out"]: TensorDecl((self.E, self.n_q * self.dv))}
+        if self.fixed_sink is None:
+            t[n["sink"]] = TensorDecl((self.n_q,), kind="vector", std=1.0)
+        if self.qk_norm:
+            t[n["q_norm"]] = TensorDecl((self.d,), kind="vector", init="norm")
+            t[n["k_norm"]] = TensorDecl((self.d,), kind="vector", init="norm")
+        if self.gate:
+            t[n["gate"]] = TensorDecl((self.n_q * self.dv, self.E))
         if self.bias:
             t[n["q_bias"]] = TensorDecl((self.Cq,), kind="vector", std=0.1)
             t[n["k_bias"]] = TensorDecl((self.Ck,), kind="vector", std=0.1)
@@ -75,11 +94,20 @@ class SinkAttention(Mixer):
 
     def load(self, src) -> None:
         f, n = src.fetch, self.names
-        self.w_in = torch.cat((f(n["q"]), f(n["k"]), f(n["v"])), dim=0).contiguous()
+        rows = [f(n["q"]), f(n["k"]), f(n["v"])] + ([f(n["gate"])] if self.gate else [])        # one product: [q | k | v | gate]
+        self.w_in = torch.cat(rows, dim=0).contiguous()
         self.w_out = f(n["out"]).contiguous()
         if self.bias:
-            self.b_in = torch.cat((f(n["q_bias"]), f(n["k_bias"]), f(n["v_bias"])), dim=0).to(self.env.dtype).contiguous()
-        self.sink = f(n["sink"]).float().contiguous()
+            b = [f(n["q_bias"]), f(n["k_bias"]), f(n["v_bias"])]
+            if self.gate:
+                b.append(torch.zeros_like(b[0][:1]).expand(self.n_q * self.dv))
+            self.b_in = torch.cat(b, dim=0).to(self.env.dtype).contiguous()
+        if self.fixed_sink is None:
+            self.sink = f(n["sink"]).float().contiguous()
+        else:
+            self.sink = torch.full((self.n_q,), self.fixed_sink, dtype=torch.float32, device=self.w_in.device)
+        if self.qk_norm:
+            self.q_norm, self.k_norm = f(n["q_norm"]).float().contiguous(), f(n["k_norm"]).float().contiguous()
         if self.value_mix == "blend":
             self.lam = float(f(n["mix"]).float().item())
 
@@ -101,9 +129,11 @@ class SinkAttention(Mixer):
         angles = self.position.step_angles(ctx) if self.position is not None else None
         q = ops.sink_qkv_prep(proj, n_q=self.n_q, n_kv=self.n_kv, d=self.d, dv=self.dv, angles=angles, v_first=v_first, lam=self.lam,
                               out_loc=cache.group.out_loc if writes_cache else None, k_cache=cache.k if writes_cache else None,
-                              v_cache=cache.v if writes_cache else None, page_size=cache.page_size)
+                              v_cache=cache.v if writes_cache else None, page_size=cache.page_size, q_norm=self.q_norm,
+                              k_norm=self.k_norm, v_unit=self.value_norm, eps=self.eps)
+        gate = proj[:, Cq + Ck + Cv:Cq + Ck + Cv + self.n_q * self.dv] if self.gate else None
         out = torch.empty((ctx.T, self.n_q * self.dv), dtype=x.dtype, device=x.device)
         ops.sink_attention(q, out, cache.k, cache.v, q_start=ctx.q_start, kv_len=ctx.kv_len, block_table=cache.group.block_table,
                            n_kv=self.n_kv, page_size=cache.page_size, scale=self.scale, softcap=self.softcap, window=self.window or 0,
-                           sink=self.sink, q_lens=None if ctx.uniform_decode else ctx.host_q_lens, workspace=ctx.workspace)
+                           sink=self.sink, q_lens=None if ctx.uniform_decode else ctx.host_q_lens, workspace=ctx.workspace, gate=gate)
         return ops.linear(out, self.w_out)
