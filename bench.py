@@ -615,6 +615,35 @@ def lifulorn_config(size, layers, vocab, window=1024):
             "token_side": {"dim": 128}, "layers": [kinds[i % 4] for i in range(layers)]}
 
 
+def pokatar_config(size, layers, vocab):
+    """A Pokatar model with the given layer sizes.  The attention has the heads of the Qwen3 layer (key and value size of the
+    head); the latent attention as many heads with key and value size 128 over a cache row of 256 elements (latent 192 + 64
+    rotated; at the smaller size 96 + 32) as the Nametar model's; the dense feed-forward has the layer's width, the routed one 28
+    plain experts and 4 identity outputs in 4 groups (2 kept) of which a token uses 4, each a quarter as wide, beside a shared
+    expert of that width.  Kinds of layers in turn: attention + dense, latent attention + routed, attention + routed, latent
+    attention + dense."""
+    s = COMPARE_SIZES[size]
+    row = 128 if s["width"] <= 2048 else 256
+    rot = row // 4
+    att = {"type": "attention", "mixer": {"heads": s["heads"], "kv_heads": s["kv_heads"], "dim": s["dim"], "vdim": s["dim"],
+                                          "scale": s["dim"] ** -0.5}}
+    lat = {"type": "latent_attention",
+           "mixer": {"heads": s["heads"], "dim": s["dim"], "rot_dim": rot, "vdim": s["dim"], "kv_rank": row - rot, "scale": (s["dim"] + rot) ** -0.5,
+                     "rot": {"base": 10000.0, "dims": rot, "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}}
+    dense = {"kind": "dense", "ff": s["ff"]}
+    moe = {"kind": "moe", "expert": {"ff": s["ff"] // 4}, "router": {"experts": 28, "identity": 4, "top": 4, "groups": {"count": 4, "keep": 2}},
+           "shared": {"ff": s["ff"] // 4}}
+    kinds = [dict(att, mlp=dense), dict(lat, mlp=moe), dict(att, mlp=moe), dict(lat, mlp=dense)]
+    return {"architecture": "Pokatar", "width": s["width"], "vocab": vocab, "norm": {"eps": 1e-5}, "layers": [kinds[i % 4] for i in range(layers)]}
+
+
+def workload_pokatar(args):
+    """As --workload vekurax_compare, with a Pokatar model (`pokatar_config`) beside the Lifulorn model (the engine's other design
+    with an attention with a term in the denominator and routed experts beside a shared one), the Nametar model (its other latent
+    attention) and the Qwen3 model of equal sizes."""
+    return workload_vekurax(args, name="pokatar", config=pokatar_config, beside=("lifulorn", "nametar", "qwen3"))
+
+
 def workload_lifulorn(args):
     """As --workload vekurax_compare, with a Lifulorn model (`lifulorn_config`) beside the Pepevik model of equal sizes (the
     engine's other design with routed experts, a recurrence with a short convolution and an attention whose key and value rows
@@ -659,8 +688,11 @@ def workload_vekurax(args, name="vekurax", config=None, beside="qwen3"):
                     num_key_value_heads=s["kv_heads"], head_dim=s["dim"], intermediate_size=s["ff"], vocab_size=V,
                     tie_word_embeddings=True, max_position_embeddings=CTX + 4096)
         res = {}
-        others = {"qwen3": lambda: qwen, "vekurax": lambda: vekurax_config(size, L, V), "pepevik": lambda: pepevik_config(size, L, V)}
-        archs = ((name, config(size, L, V)),) if args.alone else ((name, config(size, L, V)), (beside, others[beside]()))
+        others = {"qwen3": lambda: qwen, "vekurax": lambda: vekurax_config(size, L, V), "pepevik": lambda: pepevik_config(size, L, V),
+                  "lifulorn": lambda: lifulorn_config(size, L, V), "nametar": lambda: nametar_config(size, L, V)}
+        archs = [(name, config(size, L, V))]
+        if not args.alone:
+            archs += [(b, others[b]()) for b in ((beside,) if isinstance(beside, str) else beside)]
         for arch, cfg in archs:
             tmp = tempfile.mkdtemp(prefix="msgl_bench_")
             with open(os.path.join(tmp, "config.json"), "w") as f:
@@ -737,9 +769,9 @@ def main():
                     help="cudaProfilerStart/Stop around the timed region (ncu --profile-from-start off)")
     ap.add_argument("--no-graph", action="store_true", help="decode without CUDA graphs")
     ap.add_argument("--workload", default="headline", choices=["headline", "qwen3_0.6b_mixed", "qwen3_32b_long", "sweep", "vekurax_compare", "nametar_compare", "pepevik_compare",
-                                                              "lifulorn_compare"],
+                                                              "lifulorn_compare", "pokatar_compare"],
                     help="headline: the default line; the others: further workloads, one JSON line each")
-    ap.add_argument("--sizes", default=None, help="--workload vekurax_compare / nametar_compare / pepevik_compare / lifulorn_compare: layer sizes to run, of " + ",".join(COMPARE_SIZES))
+    ap.add_argument("--sizes", default=None, help="--workload vekurax_compare / nametar_compare / pepevik_compare / lifulorn_compare / pokatar_compare: layer sizes to run, of " + ",".join(COMPARE_SIZES))
     ap.add_argument("--alone", action="store_true", help="the compare workloads: run the named design only, not the one beside it")
     ap.add_argument("--skip-sanity", action="store_true", help="no comparison with the plain implementation before timing")
     ap.add_argument("--model", default="8b", choices=["8b", "32b", "0.6b"], help="layer sizes for --only decode / prefill")
@@ -768,6 +800,8 @@ def main():
         return workload_pepevik(args)
     if args.workload == "lifulorn_compare":
         return workload_lifulorn(args)
+    if args.workload == "pokatar_compare":
+        return workload_pokatar(args)
 
     import torch
 

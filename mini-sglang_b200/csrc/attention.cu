@@ -75,7 +75,28 @@ struct AttnParams {
     // null, or [n_q][bias_len] float32 in log2 units: added to the scaled score by distance min(position - key, bias_len - 1)
     const float* bias = nullptr;
     int bias_len = 0;
+    // null, or [n_q] float32 in log2 units: the score of one more term in every softmax's denominator that has no key and no
+    // value (joined once, where a row is normalised: in the direct epilogues or in the merge of the kv splits)
+    const float* null_log2 = nullptr;
+    // null, or rows of the activation type ([T] rows of gate_stride elements, [n_q * d] used): the output is multiplied by
+    // sigmoid(gate), element by element (likewise where a row is normalised)
+    const void* gate = nullptr;
+    long long gate_stride = 0;
 };
+
+// weight of the term without a key against the reference m (log2 units) of a row's exponentials
+__device__ __forceinline__ float null_weight(const float* null_log2, int head, float m) {
+    return null_log2 != nullptr ? exp2f(null_log2[head] - m) : 0.f;
+}
+template <typename T>
+__device__ __forceinline__ float gate_factor(const void* gate, long long gate_stride, size_t tok, int col) {
+    if (gate == nullptr) return 1.f;
+    return 1.f / (1.f + expf(-to_f32<T>(reinterpret_cast<const T*>(gate)[tok * gate_stride + col])));
+}
+__device__ __forceinline__ float2 gate_pair(unsigned g) {              // two neighbouring bfloat16 gates -> their sigmoids
+    const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&g));
+    return make_float2(1.f / (1.f + __expf(-f.x)), 1.f / (1.f + __expf(-f.y)));
+}
 
 // position -> (page index within the request, slot within the page)
 __device__ __forceinline__ int page_index(const AttnParams& p, int key) {
@@ -495,13 +516,19 @@ __global__ void __launch_bounds__(MMA_THREADS) attn_mma_kernel(const AttnParams 
             const int head = kvh * G + hg;
             const float l = half ? l_hi : l_lo, m = half ? m_hi : m_lo;
             if (direct) {
-                const float inv = l > 0.f ? 1.f / l : 0.f;
+                const float L = l + null_weight(p.null_log2, head, m);
+                const float inv = L > 0.f ? 1.f / L : 0.f;
                 __nv_bfloat16* dst = og + (tok * p.n_q + head) * D;
+                const __nv_bfloat16* gt = p.gate ? reinterpret_cast<const __nv_bfloat16*>(p.gate) + tok * p.gate_stride + (size_t)head * D : nullptr;
 #pragma unroll
                 for (int nd = 0; nd < NDB; ++nd) {
                     const int col = nd * 8 + (lane & 3) * 2;
-                    *reinterpret_cast<__nv_bfloat162*>(dst + col) =
-                        __floats2bfloat162_rn(o[nd][half * 2] * inv, o[nd][half * 2 + 1] * inv);
+                    float a = o[nd][half * 2] * inv, b = o[nd][half * 2 + 1] * inv;
+                    if (gt != nullptr) {
+                        const float2 g = gate_pair(*reinterpret_cast<const unsigned*>(gt + col));
+                        a *= g.x; b *= g.y;
+                    }
+                    *reinterpret_cast<__nv_bfloat162*>(dst + col) = __floats2bfloat162_rn(a, b);
                 }
             } else {
                 const size_t prow = ((size_t)split * p.T + tok) * p.n_q + head;
@@ -747,7 +774,9 @@ __global__ void __launch_bounds__(NW * 32) attn_decode_kernel(const AttnParams p
         const size_t tok = (size_t)(ti.q_base + ti.t0 + tl);
         const int head = kvh * G + hg;
         if (ns == 1) {
-            og[(tok * p.n_q + head) * D + col] = __float2bfloat16_rn(L > 0.f ? acc / L : 0.f);
+            L += null_weight(p.null_log2, head, Mu);
+            og[(tok * p.n_q + head) * D + col] =
+                __float2bfloat16_rn((L > 0.f ? acc / L : 0.f) * gate_factor<__nv_bfloat16>(p.gate, p.gate_stride, tok, head * D + col));
         } else {
             const size_t prow = ((size_t)split * p.T + tok) * p.n_q + head;
             p.part_o[prow * D + col] = acc;
@@ -1107,7 +1136,9 @@ __device__ __forceinline__ void decode_t_run(const AttnParams& p, const TileInfo
         const size_t tok = (size_t)(ti.q_base + ti.t0 + tl);
         const int head = kvh * G + hg;
         if (ns == 1) {
-            og[(tok * p.n_q + head) * D + col] = __float2bfloat16_rn(L > 0.f ? acc / L : 0.f);
+            L += null_weight(p.null_log2, head, Mu);
+            og[(tok * p.n_q + head) * D + col] =
+                __float2bfloat16_rn((L > 0.f ? acc / L : 0.f) * gate_factor<__nv_bfloat16>(p.gate, p.gate_stride, tok, head * D + col));
         } else {
             const size_t prow = ((size_t)split * p.T + tok) * p.n_q + head;
             p.part_o[prow * D + col] = acc;
@@ -1324,8 +1355,8 @@ __global__ void __launch_bounds__(SIMT_THREADS) attn_simt_kernel(const AttnParam
         const size_t tok = (size_t)(ti.q_base + ti.t0 + tl);
         const int head = kvh * G + hg;
         if (ns == 1) {
-            const float l = Ls[r];
-            og[(tok * p.n_q + head) * D + c] = from_f32<T>(l > 0.f ? Os[idx] / l : 0.f);
+            const float l = Ls[r] + null_weight(p.null_log2, head, Ms[r]);
+            og[(tok * p.n_q + head) * D + c] = from_f32<T>((l > 0.f ? Os[idx] / l : 0.f) * gate_factor<T>(p.gate, p.gate_stride, tok, head * D + c));
         } else {
             const size_t prow = ((size_t)split * p.T + tok) * p.n_q + head;
             p.part_o[prow * D + c] = Os[idx];
@@ -1335,12 +1366,14 @@ __global__ void __launch_bounds__(SIMT_THREADS) attn_simt_kernel(const AttnParam
 }
 
 // ---------------------------------------------------------------------------------------
-// merge of the kv splits, in split order: out = sum_s 2^(m_s - M) o_s / sum_s 2^(m_s - M) l_s
+// merge of the kv splits, in split order: out = sum_s 2^(m_s - M) o_s / (sum_s 2^(m_s - M) l_s + the term without a key),
+// times sigmoid(gate) where gates are given
 // ---------------------------------------------------------------------------------------
 template <typename T>
 __global__ void attn_combine_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
                                     const int* __restrict__ token_req, const int* __restrict__ nsplit,
-                                    T* __restrict__ out, int T_, int n_q, int d, int max_split) {
+                                    T* __restrict__ out, int T_, int n_q, int d, int max_split, const float* __restrict__ null_log2,
+                                    const void* __restrict__ gate, long long gate_stride) {
     // one block per (token, head); threads over the head's elements
     pdl_launch_dependents();
     pdl_wait();
@@ -1358,6 +1391,7 @@ __global__ void attn_combine_kernel(const float* __restrict__ part_o, const floa
         const size_t prow = ((size_t)s * T_ + tok) * n_q + h;
         L += exp2f(part_ml[prow * 2] - Mu) * part_ml[prow * 2 + 1];
     }
+    L += null_weight(null_log2, h, Mu);
     const float inv = L > 0.f ? 1.f / L : 0.f;
     for (int c = threadIdx.x; c < d; c += blockDim.x) {
         float acc = 0.f;
@@ -1365,7 +1399,7 @@ __global__ void attn_combine_kernel(const float* __restrict__ part_o, const floa
             const size_t prow = ((size_t)s * T_ + tok) * n_q + h;
             acc += exp2f(part_ml[prow * 2] - Mu) * part_o[prow * d + c];
         }
-        out[((size_t)tok * n_q + h) * d + c] = from_f32<T>(acc * inv);
+        out[((size_t)tok * n_q + h) * d + c] = from_f32<T>(acc * inv * gate_factor<T>(gate, gate_stride, tok, h * d + c));
     }
 }
 
@@ -1424,17 +1458,18 @@ static int attention_launch(const void* q, void* out, const void* k_cache, const
                             float* part_ml, int B, int T_, int n_q, int n_kv, int d, int page_size, int bt_stride,
                             int window, int max_split, float scale, int qlen_min, int qlen_max, int uniform_decode,
                             int variant, int grid_x, int dtype, const int* order, const int* even, int even_nb,
-                            int keep_first, const float* bias, int bias_len, cudaStream_t stream);
+                            int keep_first, const float* bias, int bias_len, const float* null_log2, const void* gate,
+                            long long gate_stride, cudaStream_t stream);
 
 MSGL_API int msgl_attention(const void* q, void* out, const void* k_cache, const void* v_cache, const int* q_start,
                             const int* kv_len, const int* block_table, const int* nsplit, float* part_o,
                             float* part_ml, int B, int T_, int n_q, int n_kv, int d, int page_size, int bt_stride,
                             int window, int max_split, float scale, int qlen_min, int qlen_max, int uniform_decode,
                             int variant, int grid_x, int dtype, const int* order, const int* even, int even_nb,
-                            cudaStream_t stream) {
+                            const float* null_log2, const void* gate, long long gate_stride, cudaStream_t stream) {
     return attention_launch(q, out, k_cache, v_cache, q_start, kv_len, block_table, nsplit, part_o, part_ml, B, T_, n_q, n_kv, d,
                             page_size, bt_stride, window, max_split, scale, qlen_min, qlen_max, uniform_decode, variant, grid_x,
-                            dtype, order, even, even_nb, 0, nullptr, 0, stream);
+                            dtype, order, even, even_nb, 0, nullptr, 0, null_log2, gate, gate_stride, stream);
 }
 
 // The same with a window that keeps the first `keep_first` keys of every request visible and with a bias by distance
@@ -1451,7 +1486,7 @@ MSGL_API int msgl_attention_window(const void* q, void* out, const void* k_cache
     if (!(variant == 1 || (variant == 2 && MSGL_HEAD_DIM % 32 == 0 && G <= 16))) return MSGL_ERR_SIZE;
     return attention_launch(q, out, k_cache, v_cache, q_start, kv_len, block_table, nsplit, part_o, part_ml, B, T_, n_q, n_kv, d,
                             page_size, bt_stride, window, max_split, scale, qlen_min, qlen_max, uniform_decode, variant, grid_x,
-                            dtype, order, nullptr, 0, keep_first, bias, bias_len, stream);
+                            dtype, order, nullptr, 0, keep_first, bias, bias_len, nullptr, nullptr, 0, stream);
 }
 
 static int attention_launch(const void* q, void* out, const void* k_cache, const void* v_cache, const int* q_start,
@@ -1459,7 +1494,9 @@ static int attention_launch(const void* q, void* out, const void* k_cache, const
                             float* part_ml, int B, int T_, int n_q, int n_kv, int d, int page_size, int bt_stride,
                             int window, int max_split, float scale, int qlen_min, int qlen_max, int uniform_decode,
                             int variant, int grid_x, int dtype, const int* order, const int* even, int even_nb,
-                            int keep_first, const float* bias, int bias_len, cudaStream_t stream) {
+                            int keep_first, const float* bias, int bias_len, const float* null_log2, const void* gate,
+                            long long gate_stride, cudaStream_t stream) {
+    if (gate != nullptr && dtype == MSGL_BF16 && ((gate_stride & 1) || ((uintptr_t)gate & 3))) return MSGL_ERR_ALIGN;
     if (grid_x <= 0 || B <= 0) return MSGL_OK;
     if (n_kv <= 0 || n_q % n_kv != 0 || d <= 0 || page_size <= 0 || max_split < 1) return MSGL_ERR_SIZE;
     if (max_split > 1 && (part_o == nullptr || part_ml == nullptr || nsplit == nullptr)) return MSGL_ERR_SIZE;
@@ -1473,6 +1510,7 @@ static int attention_launch(const void* q, void* out, const void* k_cache, const
     if ((page_size & (page_size - 1)) == 0) { int sh = 0; while ((1 << sh) < page_size) ++sh; p.page_shift = sh; } p.scale = scale; p.qlen_min = qlen_min; p.qlen_max = qlen_max;
     p.uniform_decode = uniform_decode;
     p.keep_first = window > 0 ? keep_first : 0; p.bias = bias; p.bias_len = bias_len;
+    p.null_log2 = null_log2; p.gate = gate; p.gate_stride = gate_stride;
     const int G = n_q / n_kv;
     const int R = variant == 1 ? 64 : 16;
     const int n_chunks = G <= R ? 1 : (G + R - 1) / R;
@@ -1575,8 +1613,9 @@ MSGL_API int msgl_attention_tc(const void* q, void* out, const void* k_cache, co
                                const int* kv_len, const int* block_table, int B, int T_, int n_q, int n_kv, int d,
                                int page_size, int bt_stride, int window, float scale, int qlen_min, int qlen_max,
                                int grid_x, int cache_pages, int version, int* status, int keep_first, const float* bias,
-                               int bias_len, cudaStream_t stream) {
+                               int bias_len, const float* null_log2, const void* gate, long long gate_stride, cudaStream_t stream) {
 #if MSGL_HEAD_DIM == 128
+    if (gate != nullptr && ((gate_stride & 7) || ((uintptr_t)gate & 15))) return MSGL_ERR_ALIGN;
     // kept first tokens under the window and a bias by distance ([n_q][bias_len] float32, log2 units): version 2 only
     const bool ext = (window > 0 && keep_first > 0) || bias != nullptr;
     if (ext && (version != 2 || keep_first < 0 || (bias != nullptr && bias_len < 1))) return MSGL_ERR_SIZE;
@@ -1592,6 +1631,7 @@ MSGL_API int msgl_attention_tc(const void* q, void* out, const void* k_cache, co
     p.page_shift = -1;
     if ((page_size & (page_size - 1)) == 0) { int sh = 0; while ((1 << sh) < page_size) ++sh; p.page_shift = sh; }
     p.scale = scale; p.qlen_min = qlen_min; p.qlen_max = qlen_max; p.uniform_decode = 0;
+    p.null_log2 = null_log2; p.gate = gate; p.gate_stride = gate_stride;
     p.keep_first = window > 0 ? keep_first : 0; p.bias = bias; p.bias_len = bias_len;
     const int G = n_q / n_kv;
     const int n_chunks = G <= TC_ROWS ? 1 : (G + TC_ROWS - 1) / TC_ROWS;
@@ -1629,15 +1669,16 @@ MSGL_API int msgl_attention_tc(const void* q, void* out, const void* k_cache, co
 
 MSGL_API int msgl_attention_combine(const float* part_o, const float* part_ml, const int* token_req,
                                     const int* nsplit, void* out, int T_, int n_q, int d, int max_split, int dtype,
-                                    cudaStream_t stream) {
+                                    const float* null_log2, const void* gate, long long gate_stride, cudaStream_t stream) {
     if (T_ <= 0 || max_split <= 1) return MSGL_OK;
     const int threads = d >= 128 ? 128 : (d >= 64 ? 64 : 32);
     const dim3 grid(T_, n_q);
     if (dtype == MSGL_F32)
-        msgl_launch_pdl(attn_combine_kernel<float>, grid, dim3(threads), 0, stream, part_o, part_ml, token_req, nsplit, (float*)out, T_, n_q, d, max_split);
+        msgl_launch_pdl(attn_combine_kernel<float>, grid, dim3(threads), 0, stream, part_o, part_ml, token_req, nsplit, (float*)out, T_, n_q, d, max_split,
+                        null_log2, gate, gate_stride);
     else if (dtype == MSGL_BF16)
         msgl_launch_pdl(attn_combine_kernel<__nv_bfloat16>, grid, dim3(threads), 0, stream, part_o, part_ml, token_req, nsplit,
-                        (__nv_bfloat16*)out, T_, n_q, d, max_split);
+                        (__nv_bfloat16*)out, T_, n_q, d, max_split, null_log2, gate, gate_stride);
     else
         return MSGL_ERR_DTYPE;
     return msgl_check_launch();

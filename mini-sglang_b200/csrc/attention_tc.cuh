@@ -401,10 +401,13 @@ __global__ void __launch_bounds__(TC_THREADS, 2) attn_tc_kernel(const AttnParams
             tc_fence_after();
         }
         if (!__any_sync(0xffffffffu, fail) && n_tiles > 0) {
-            const float inv = l_run > 0.f ? 1.f / l_run : 0.f;
             const int hl = tid - my_tl * Gc;
-            __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(p.out) +
-                                 ((size_t)(ti.q_base + ti.t0 + (my_valid ? my_tl : 0)) * p.n_q + (size_t)kvh * G + (my_valid ? chunk * TC_ROWS + hl : 0)) * TC_D;
+            const int my_head = kvh * G + (my_valid ? chunk * TC_ROWS + hl : 0);
+            const size_t my_tok = (size_t)(ti.q_base + ti.t0 + (my_valid ? my_tl : 0));
+            const float l_all = l_run + null_weight(p.null_log2, my_head, m_run);
+            const float inv = l_all > 0.f ? 1.f / l_all : 0.f;
+            const __nv_bfloat16* gt = p.gate ? reinterpret_cast<const __nv_bfloat16*>(p.gate) + my_tok * p.gate_stride + (size_t)my_head * TC_D : nullptr;
+            __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(p.out) + (my_tok * p.n_q + my_head) * TC_D;
 #pragma unroll 1
             for (int cb = 0; cb < 4; ++cb) {
                 float v[32];
@@ -414,6 +417,15 @@ __global__ void __launch_bounds__(TC_THREADS, 2) attn_tc_kernel(const AttnParams
 #pragma unroll
                     for (int j = 0; j < 32; j += 8) {
                         uint4 pk;
+                        if (gt != nullptr) {
+                            const uint4 g = *reinterpret_cast<const uint4*>(gt + cb * 32 + j);
+                            const unsigned gw[4] = {g.x, g.y, g.z, g.w};
+#pragma unroll
+                            for (int e = 0; e < 4; ++e) {
+                                const float2 f = gate_pair(gw[e]);
+                                v[j + 2 * e] *= f.x; v[j + 2 * e + 1] *= f.y;
+                            }
+                        }
                         pk.x = pack_bf16(v[j] * inv, v[j + 1] * inv);
                         pk.y = pack_bf16(v[j + 2] * inv, v[j + 3] * inv);
                         pk.z = pack_bf16(v[j + 4] * inv, v[j + 5] * inv);

@@ -58,6 +58,14 @@ __device__ __forceinline__ float block_sum(float v, float* scratch) {
     return r;
 }
 
+// Products with a gated activation in their epilogue, act(gate) * up: the kind is a template argument and the entry
+// points' `mode`.  0: plain product.
+enum { MSGL_GLU_NONE = 0, MSGL_GLU_SILU = 1, MSGL_GLU_RELU = 2 };
+template <int GLU> __device__ __forceinline__ float glu_act(float gate) {
+    if (GLU == MSGL_GLU_RELU) return fmaxf(gate, 0.f);
+    return gate / (1.f + expf(-gate));
+}
+
 // Programmatic dependent launch: a kernel launched with msgl_launch_pdl may start while the kernel
 // before it in the stream is still running.  It must call pdl_wait() before it reads anything an
 // earlier kernel wrote and before it writes anything at all; what comes before the wait (index

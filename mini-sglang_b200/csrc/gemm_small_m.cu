@@ -15,12 +15,12 @@
 //   * the warps' partial sums are added in warp order through shared memory (a fixed order, so
 //     the result does not depend on timing), then bias / SwiGLU and one rounding to the output type.
 //
-// SwiGLU mode: W is [2I, K] with the gate rows first; a block takes 8 gate rows and the 8 up rows
-// that belong to them, which land in the two row halves of the accumulator fragment, so
-// out[M, I] = silu(gate) * up is formed in registers and the [M, 2I] intermediate never exists.
+// Gated modes (SwiGLU, ReGLU): W is [2I, K] with the gate rows first; a block takes 8 gate rows and the
+// 8 up rows that belong to them, which land in the two row halves of the accumulator fragment, so
+// out[M, I] = act(gate (+ bias)) * (up (+ bias)) is formed in registers and the [M, 2I] intermediate never exists.
 //
 // Requirements (checked by the entry point, which returns MSGL_ERR_SIZE otherwise and the caller
-// uses the library GEMM): bfloat16 inputs, K % 32 == 0, N % 16 == 0 (I % 8 == 0 in SwiGLU mode),
+// uses the library GEMM): bfloat16 inputs, K % 32 == 0, N % 16 == 0 (I % 8 == 0 in gated modes),
 // 16-byte aligned rows.
 #include "common.cuh"
 
@@ -64,7 +64,7 @@ __device__ __forceinline__ void cp_async16_a(void* smem, const void* gmem) {    
     asm volatile("cp.async.ca.shared.global [%0], [%1], 16;\n" ::"r"(s_), "l"(gmem));
 }
 
-template <int NB, bool SWIGLU, typename OutT>
+template <int NB, int GLU, typename OutT>
 __global__ void __launch_bounds__(GS_WARPS * 32) gemm_small_m_kernel(
     const __nv_bfloat16* __restrict__ W, const __nv_bfloat16* __restrict__ X, const __nv_bfloat16* __restrict__ bias,
     OutT* __restrict__ out, int M, int N, int K, long long ldx, long long ldo, int I) {
@@ -78,7 +78,7 @@ __global__ void __launch_bounds__(GS_WARPS * 32) gemm_small_m_kernel(
 
     // the two weight rows this lane feeds into the A fragment
     size_t row_lo, row_hi;
-    if (SWIGLU) {
+    if (GLU) {
         row_lo = (size_t)blockIdx.x * 8 + g;          // gate row
         row_hi = (size_t)I + row_lo;                  // its up row
     } else {
@@ -157,7 +157,7 @@ __global__ void __launch_bounds__(GS_WARPS * 32) gemm_small_m_kernel(
         red[warp][g + 8][nb * 8 + 2 * t + 1] = c[nb][3];
     }
     __syncthreads();
-    if (SWIGLU) {
+    if (GLU) {
         // 8 output columns x (8 NB) tokens
         for (int idx = threadIdx.x; idx < 8 * 8 * NB; idx += GS_WARPS * 32) {
             const int r = idx / (8 * NB), tok = idx - r * (8 * NB);
@@ -165,8 +165,9 @@ __global__ void __launch_bounds__(GS_WARPS * 32) gemm_small_m_kernel(
             float gate = 0.f, up = 0.f;
 #pragma unroll
             for (int w = 0; w < GS_WARPS; ++w) { gate += red[w][r][tok]; up += red[w][r + 8][tok]; }
-            const float y = gate / (1.f + expf(-gate)) * up;
-            store_out<OutT>(out + (size_t)tok * ldo + (size_t)blockIdx.x * 8 + r, y);
+            const size_t col = (size_t)blockIdx.x * 8 + r;
+            if (bias) { gate += __bfloat162float(bias[col]); up += __bfloat162float(bias[(size_t)I + col]); }
+            store_out<OutT>(out + (size_t)tok * ldo + col, glu_act<GLU>(gate) * up);
         }
     } else {
         for (int idx = threadIdx.x; idx < 16 * 8 * NB; idx += GS_WARPS * 32) {
@@ -182,7 +183,7 @@ __global__ void __launch_bounds__(GS_WARPS * 32) gemm_small_m_kernel(
     }
 }
 
-// mode: 0 = plain (out [M, N]), 1 = SwiGLU (W [2I, K], out [M, I], N = 2I).  out_f32: output type.
+// mode: 0 = plain (out [M, N]), 1 / 2 = SwiGLU / ReGLU (W [2I, K], bias [2I], out [M, I], N = 2I).  out_f32: output type.
 MSGL_API int msgl_gemm_small_m(const void* W, const void* X, const void* bias, void* out, int M, int N, int K,
                                long long ldx, long long ldo, int mode, int out_f32, cudaStream_t stream) {
     if (M <= 0) return MSGL_OK;
@@ -196,34 +197,38 @@ MSGL_API int msgl_gemm_small_m(const void* W, const void* X, const void* bias, v
     const size_t smem1 = (size_t)GS_WARPS * GS_PF * 3 * 32 * 16, smem2 = (size_t)GS_WARPS * GS_PF * 4 * 32 * 16;
     static MsglOncePerDevice attr_set;
     if (attr_set.due()) {      // first call on this device, never inside a stream capture
-        cudaFuncSetAttribute(gemm_small_m_kernel<1, true, __nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem1);
-        cudaFuncSetAttribute(gemm_small_m_kernel<2, true, __nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem2);
-        cudaFuncSetAttribute(gemm_small_m_kernel<1, false, __nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem1);
-        cudaFuncSetAttribute(gemm_small_m_kernel<2, false, __nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem2);
-        cudaFuncSetAttribute(gemm_small_m_kernel<1, false, float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem1);
-        cudaFuncSetAttribute(gemm_small_m_kernel<2, false, float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem2);
+        cudaFuncSetAttribute(gemm_small_m_kernel<1, 1, __nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem1);
+        cudaFuncSetAttribute(gemm_small_m_kernel<2, 1, __nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem2);
+        cudaFuncSetAttribute(gemm_small_m_kernel<1, 2, __nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem1);
+        cudaFuncSetAttribute(gemm_small_m_kernel<2, 2, __nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem2);
+        cudaFuncSetAttribute(gemm_small_m_kernel<1, 0, __nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem1);
+        cudaFuncSetAttribute(gemm_small_m_kernel<2, 0, __nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem2);
+        cudaFuncSetAttribute(gemm_small_m_kernel<1, 0, float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem1);
+        cudaFuncSetAttribute(gemm_small_m_kernel<2, 0, float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem2);
         attr_set.mark();
     }
-    if (mode == 1) {
-        if ((N & 15) || bias != nullptr) return MSGL_ERR_SIZE;
+    if (mode < 0 || mode > 2) return MSGL_ERR_SIZE;
+    if (mode != MSGL_GLU_NONE) {
+        if (N & 15) return MSGL_ERR_SIZE;
         const int I = N / 2;
         if (I & 7) return MSGL_ERR_SIZE;
         const int grid = I / 8;
         if (out_f32) return MSGL_ERR_DTYPE;
-        if (M <= 8)
-            msgl_launch_pdl(gemm_small_m_kernel<1, true, __nv_bfloat16>, dim3(grid), dim3(threads), smem1, stream, w, x, nullptr, (__nv_bfloat16*)out, M, N, K, ldx, ldo, I);
-        else
-            msgl_launch_pdl(gemm_small_m_kernel<2, true, __nv_bfloat16>, dim3(grid), dim3(threads), smem2, stream, w, x, nullptr, (__nv_bfloat16*)out, M, N, K, ldx, ldo, I);
+#define SMALL_M_GLU(NB, GLU, SMEM) \
+    msgl_launch_pdl(gemm_small_m_kernel<NB, GLU, __nv_bfloat16>, dim3(grid), dim3(threads), SMEM, stream, w, x, b, (__nv_bfloat16*)out, M, N, K, ldx, ldo, I)
+        if (mode == MSGL_GLU_SILU) { if (M <= 8) SMALL_M_GLU(1, 1, smem1); else SMALL_M_GLU(2, 1, smem2); }
+        else { if (M <= 8) SMALL_M_GLU(1, 2, smem1); else SMALL_M_GLU(2, 2, smem2); }
+#undef SMALL_M_GLU
         return msgl_check_launch();
     }
     if (N & 15) return MSGL_ERR_SIZE;
     const int grid = N / 16;
     if (out_f32) {
-        if (M <= 8) msgl_launch_pdl(gemm_small_m_kernel<1, false, float>, dim3(grid), dim3(threads), smem1, stream, w, x, b, (float*)out, M, N, K, ldx, ldo, 0);
-        else msgl_launch_pdl(gemm_small_m_kernel<2, false, float>, dim3(grid), dim3(threads), smem2, stream, w, x, b, (float*)out, M, N, K, ldx, ldo, 0);
+        if (M <= 8) msgl_launch_pdl(gemm_small_m_kernel<1, 0, float>, dim3(grid), dim3(threads), smem1, stream, w, x, b, (float*)out, M, N, K, ldx, ldo, 0);
+        else msgl_launch_pdl(gemm_small_m_kernel<2, 0, float>, dim3(grid), dim3(threads), smem2, stream, w, x, b, (float*)out, M, N, K, ldx, ldo, 0);
     } else {
-        if (M <= 8) msgl_launch_pdl(gemm_small_m_kernel<1, false, __nv_bfloat16>, dim3(grid), dim3(threads), smem1, stream, w, x, b, (__nv_bfloat16*)out, M, N, K, ldx, ldo, 0);
-        else msgl_launch_pdl(gemm_small_m_kernel<2, false, __nv_bfloat16>, dim3(grid), dim3(threads), smem2, stream, w, x, b, (__nv_bfloat16*)out, M, N, K, ldx, ldo, 0);
+        if (M <= 8) msgl_launch_pdl(gemm_small_m_kernel<1, 0, __nv_bfloat16>, dim3(grid), dim3(threads), smem1, stream, w, x, b, (__nv_bfloat16*)out, M, N, K, ldx, ldo, 0);
+        else msgl_launch_pdl(gemm_small_m_kernel<2, 0, __nv_bfloat16>, dim3(grid), dim3(threads), smem2, stream, w, x, b, (__nv_bfloat16*)out, M, N, K, ldx, ldo, 0);
     }
     return msgl_check_launch();
 }

@@ -28,13 +28,13 @@ constexpr unsigned GT_SMEM_ALLOC = GT_STAGES * GT_STAGE_BYTES + 256u + 1024u;
 constexpr int GT_THREADS = 192;
 
 // One thread's row of a finished accumulator (256 float32 columns at `acc`, this thread's lane already selected)
-// -> bfloat16 output: SwiGLU of columns c and 128 + c, or the plain values (+ bias).
-// c_lo, c_hi: the 32-column chunks to drain (of 4 for SwiGLU, of 8 else), so that two warps can share a row.
-template <bool SWIGLU>
+// -> bfloat16 output: the gated activation of columns c and 128 + c, or the plain values (+ bias).
+// c_lo, c_hi: the 32-column chunks to drain (of 4 for gated products, of 8 else), so that two warps can share a row.
+template <int GLU>
 __device__ __forceinline__ void gt_drain(unsigned acc, int row, int col0, int M, int n_valid, const __nv_bfloat16* __restrict__ bias,
                                          __nv_bfloat16* __restrict__ out, long long ldo, int c_lo, int c_hi) {
     __nv_bfloat16* orow = out + (size_t)(row < M ? row : 0) * ldo + col0;
-    if (SWIGLU) {
+    if (GLU) {                                             // n_valid = I: gate column c has its up column (and bias) at I + c
 #pragma unroll 1
         for (int c = c_lo; c < c_hi; ++c) {
             float gate[32], up[32];
@@ -45,22 +45,25 @@ __device__ __forceinline__ void gt_drain(unsigned acc, int row, int col0, int M,
             if (row < M) {
 #pragma unroll
                 for (int j = 0; j < 32; j += 8) {
+                    if (bias != nullptr) {
+                        const __nv_bfloat16* bg = bias + col0 + c * 32 + j;
+#pragma unroll
+                        for (int e = 0; e < 8; ++e)
+                            if (col0 + c * 32 + j + e < n_valid) { gate[j + e] += __bfloat162float(bg[e]); up[j + e] += __bfloat162float(bg[n_valid + e]); }
+                    }
                     if (col0 + c * 32 + j + 8 <= n_valid) {
                         unsigned pk[4];
 #pragma unroll
                         for (int e = 0; e < 4; ++e) {
-                            const float g0 = gate[j + 2 * e], g1 = gate[j + 2 * e + 1];
-                            const __nv_bfloat162 v = __floats2bfloat162_rn(g0 / (1.f + expf(-g0)) * up[j + 2 * e],
-                                                                           g1 / (1.f + expf(-g1)) * up[j + 2 * e + 1]);
+                            const __nv_bfloat162 v = __floats2bfloat162_rn(glu_act<GLU>(gate[j + 2 * e]) * up[j + 2 * e],
+                                                                           glu_act<GLU>(gate[j + 2 * e + 1]) * up[j + 2 * e + 1]);
                             pk[e] = *reinterpret_cast<const unsigned*>(&v);
                         }
                         *reinterpret_cast<uint4*>(orow + c * 32 + j) = make_uint4(pk[0], pk[1], pk[2], pk[3]);
                     } else {
                         for (int e = 0; e < 8; ++e)
-                            if (col0 + c * 32 + j + e < n_valid) {
-                                const float g0 = gate[j + e];
-                                orow[c * 32 + j + e] = __float2bfloat16_rn(g0 / (1.f + expf(-g0)) * up[j + e]);
-                            }
+                            if (col0 + c * 32 + j + e < n_valid)
+                                orow[c * 32 + j + e] = __float2bfloat16_rn(glu_act<GLU>(gate[j + e]) * up[j + e]);
                     }
                 }
             }
@@ -124,7 +127,7 @@ __device__ __forceinline__ void gt_drain_partial(unsigned acc, int row, int M, f
     }
 }
 
-template <bool SWIGLU>
+template <int GLU>
 __global__ void __launch_bounds__(GT_THREADS, 1) gemm_tc_kernel(const __grid_constant__ CUtensorMap xmap,
                                                                 const __grid_constant__ CUtensorMap wmap,
                                                                 const __nv_bfloat16* __restrict__ bias, __nv_bfloat16* __restrict__ out,
@@ -144,8 +147,8 @@ __global__ void __launch_bounds__(GT_THREADS, 1) gemm_tc_kernel(const __grid_con
     auto bar_acc_empty = [&](int b) { return smem_base + 80u + 8u * (unsigned)b; };       // the epilogue has read accumulator b (4 warps)
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
 
-    const int n_valid = SWIGLU ? I : N;                            // output columns
-    const int bn_out = SWIGLU ? GT_BN / 2 : GT_BN;                 // output columns of a tile
+    const int n_valid = GLU ? I : N;                            // output columns
+    const int bn_out = GLU ? GT_BN / 2 : GT_BN;                 // output columns of a tile
     const int MT = (M + GT_BM - 1) / GT_BM, NT = (n_valid + bn_out - 1) / bn_out;
     const int n_tiles = MT * NT, n_slabs = (K + GT_BK - 1) / GT_BK;
 
@@ -176,7 +179,7 @@ __global__ void __launch_bounds__(GT_THREADS, 1) gemm_tc_kernel(const __grid_con
                     const unsigned a_s = tiles0 + (unsigned)st * GT_STAGE_BYTES, b_s = a_s + GT_A_BYTES;
                     tc_mbar_expect_tx(bar_full(st), GT_STAGE_BYTES);
                     tc_tma_load(a_s, &xmap, k * GT_BK, m * GT_BM, bar_full(st));
-                    if (SWIGLU) {
+                    if (GLU) {
                         tc_tma_load(b_s, &wmap, k * GT_BK, n * 128, bar_full(st));                       // gate rows
                         tc_tma_load(b_s + 128u * 128u, &wmap, k * GT_BK, I + n * 128, bar_full(st));     // their up rows
                     } else {
@@ -222,7 +225,7 @@ __global__ void __launch_bounds__(GT_THREADS, 1) gemm_tc_kernel(const __grid_con
             const int m = t % MT, n = t / MT, b = it & 1;
             if (!tc_mbar_wait(bar_acc_full(b), (it >> 1) & 1)) { fail = 1; break; }
             tc_fence_after();
-            gt_drain<SWIGLU>(tmem + (unsigned)b * 256u + lane_sel, m * GT_BM + q * 32 + lane, n * bn_out, M, n_valid, bias, out, ldo, 0, SWIGLU ? 4 : 8);
+            gt_drain<GLU>(tmem + (unsigned)b * 256u + lane_sel, m * GT_BM + q * 32 + lane, n * bn_out, M, n_valid, bias, out, ldo, 0, GLU ? 4 : 8);
             tc_fence_before();
             __syncwarp();
             if (lane == 0) tc_mbar_arrive(bar_acc_empty(b));
@@ -296,7 +299,7 @@ __device__ __forceinline__ void gt2_commit_pair(unsigned bar) {       // the bar
                  ::"r"(bar), "h"((unsigned short)3) : "memory");
 }
 
-template <bool SWIGLU>
+template <int GLU>
 __global__ void __launch_bounds__(GT2_THREADS, 1) gemm_tc2_kernel(const __grid_constant__ CUtensorMap xmap,
                                                                  const __grid_constant__ CUtensorMap wmap,
                                                                  const __nv_bfloat16* __restrict__ bias, __nv_bfloat16* __restrict__ out,
@@ -317,8 +320,8 @@ __global__ void __launch_bounds__(GT2_THREADS, 1) gemm_tc2_kernel(const __grid_c
     auto bar_acc_empty = [&](int b) { return smem_base + 144u + 8u * (unsigned)b; };
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
 
-    const int n_valid = SWIGLU ? I : N;
-    const int bn_out = SWIGLU ? 128 : 256;
+    const int n_valid = GLU ? I : N;
+    const int bn_out = GLU ? 128 : 256;
     const int MT = (M + 255) / 256, NT = (n_valid + bn_out - 1) / bn_out;
     const int n_slabs = (K + GT_BK - 1) / GT_BK;
     const int n_tiles = MT * NT * splits;                   // work items: the ranges of a tile are neighbours, so they run at the same time
@@ -353,7 +356,7 @@ __global__ void __launch_bounds__(GT2_THREADS, 1) gemm_tc2_kernel(const __grid_c
             for (int t = pair; t < n_tiles && !fail; t += n_pairs) {
                 int m, n, k_begin, k_end;
                 item(t, m, n, k_begin, k_end);
-                const int w_row = SWIGLU ? (rank == 0 ? n * 128 : I + n * 128) : n * 256 + (int)rank * 128;
+                const int w_row = GLU ? (rank == 0 ? n * 128 : I + n * 128) : n * 256 + (int)rank * 128;
                 for (int k = k_begin; k < k_end; ++k, ++g) {
                     const int st = g % GT2_STAGES;
                     if (!tc_mbar_wait(bar_empty(st), ((g / GT2_STAGES) & 1) ^ 1)) { fail = 1; break; }
@@ -396,7 +399,7 @@ __global__ void __launch_bounds__(GT2_THREADS, 1) gemm_tc2_kernel(const __grid_c
     } else if (!fail) {
         // =========================== epilogue (both blocks): the accumulator rows of the block's own 128 tokens
         const int q = warp & 3, second = warp >= 6 ? 1 : 0;              // warps 2-5: first half of the columns, 6-9: second half
-        constexpr int n_chunks = SWIGLU ? 4 : 8;
+        constexpr int n_chunks = GLU ? 4 : 8;
         const unsigned lane_sel = (unsigned)(q * 32) << 16;
         const unsigned acc_empty0 = gt2_map_to(bar_acc_empty(0), 0);
         int it = 0;
@@ -409,10 +412,10 @@ __global__ void __launch_bounds__(GT2_THREADS, 1) gemm_tc2_kernel(const __grid_c
             const int row = m * 256 + (int)rank * 128 + q * 32 + lane;
             if (part != nullptr) {
                 float* mine = part + (size_t)(t % splits) * (size_t)M * (size_t)N;
-                if (SWIGLU) gt_drain_partial(tmem + (unsigned)b * 256u + lane_sel, row, M, mine, N, n * 128, I + n * 128, I, N, second * 4, second * 4 + 4);
+                if (GLU) gt_drain_partial(tmem + (unsigned)b * 256u + lane_sel, row, M, mine, N, n * 128, I + n * 128, I, N, second * 4, second * 4 + 4);
                 else gt_drain_partial(tmem + (unsigned)b * 256u + lane_sel, row, M, mine, N, n * 256, n * 256 + 128, N, N, second * 4, second * 4 + 4);
             } else {
-                gt_drain<SWIGLU>(tmem + (unsigned)b * 256u + lane_sel, row, n * bn_out, M, n_valid, bias, out, ldo,
+                gt_drain<GLU>(tmem + (unsigned)b * 256u + lane_sel, row, n * bn_out, M, n_valid, bias, out, ldo,
                                  second * (n_chunks / 2), (second + 1) * (n_chunks / 2));
             }
             tc_fence_before();
@@ -427,8 +430,9 @@ __global__ void __launch_bounds__(GT2_THREADS, 1) gemm_tc2_kernel(const __grid_c
     if (warp == 0) asm volatile("tcgen05.dealloc.cta_group::2.sync.aligned.b32 %0, 512;\n" ::"r"(tmem) : "memory");
 }
 
-// mode 0: out[M, N] = x . W^T (+ bias); mode 1: W = [gate; up] ([2I, K], N = 2I), out[M, I] = silu(gate) * up.
-// bfloat16 everywhere; x rows ldx elements apart, out rows ldo; K, ldx multiples of 8 and ldo, (mode 1: I) multiples
+// mode 0: out[M, N] = x . W^T (+ bias); mode 1, 2: W = [gate; up] ([2I, K], N = 2I, bias [2I]), out[M, I] = act(gate) * up with
+// act = silu (1) or relu (2).
+// bfloat16 everywhere; x rows ldx elements apart, out rows ldo; K, ldx multiples of 8 and ldo, (gated modes: I) multiples
 // of 8 for the 16-byte stores; bases 16-byte aligned.  status: device int[>= 3]; word 2 is set if a block gave up.
 // Returns MSGL_ERR_SIZE where the tensor maps cannot be made (the caller then uses the library GEMM).
 MSGL_API int msgl_gemm_tc(const void* W, const void* X, const void* bias, void* out, int M, int N, int K, long long ldx,
@@ -437,64 +441,65 @@ MSGL_API int msgl_gemm_tc(const void* W, const void* X, const void* bias, void* 
     if (N <= 0 || K <= 0 || (K & 7) || (ldx & 7) || (ldo & 7) || status == nullptr) return MSGL_ERR_SIZE;
     if (((uintptr_t)W | (uintptr_t)X | (uintptr_t)out) & 15) return MSGL_ERR_ALIGN;
     const int I = N / 2;
-    if (mode == 1 && ((N & 1) || (I & 7) || bias != nullptr)) return MSGL_ERR_SIZE;
+    if (mode < 0 || mode > 2 || (mode != MSGL_GLU_NONE && ((N & 1) || (I & 7)))) return MSGL_ERR_SIZE;
     CUtensorMap xm, wm;
     if (!tc_matrix_map(X, M, K, ldx * 2, 128, &xm) || !tc_matrix_map(W, N, K, (long long)K * 2, 128, &wm)) return MSGL_ERR_SIZE;
     static MsglOncePerDevice attr_set;
     if (attr_set.due()) {      // first call on this device, never inside a stream capture
-        if (cudaFuncSetAttribute(gemm_tc_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)GT_SMEM_ALLOC) != cudaSuccess ||
-            cudaFuncSetAttribute(gemm_tc_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)GT_SMEM_ALLOC) != cudaSuccess)
+        if (cudaFuncSetAttribute(gemm_tc_kernel<0>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)GT_SMEM_ALLOC) != cudaSuccess ||
+            cudaFuncSetAttribute(gemm_tc_kernel<1>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)GT_SMEM_ALLOC) != cudaSuccess ||
+            cudaFuncSetAttribute(gemm_tc_kernel<2>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)GT_SMEM_ALLOC) != cudaSuccess)
             return msgl_check_launch();
         attr_set.mark();
     }
-    const int n_valid = mode == 1 ? I : N, bn_out = mode == 1 ? GT_BN / 2 : GT_BN;
+    const int n_valid = mode ? I : N, bn_out = mode ? GT_BN / 2 : GT_BN;
     const long long tiles = (long long)((M + GT_BM - 1) / GT_BM) * ((n_valid + bn_out - 1) / bn_out);
     const int sms = msgl_sm_count();
     const int grid = (int)(tiles < sms ? tiles : sms);
-    if (mode == 1)
-        gemm_tc_kernel<true><<<grid, GT_THREADS, GT_SMEM_ALLOC, stream>>>(xm, wm, nullptr, (__nv_bfloat16*)out, M, N, K, ldo, I, (int*)status);
-    else
-        gemm_tc_kernel<false><<<grid, GT_THREADS, GT_SMEM_ALLOC, stream>>>(xm, wm, (const __nv_bfloat16*)bias, (__nv_bfloat16*)out, M, N, K, ldo, 0,
-                                                                           (int*)status);
+    auto* kernel = mode == 0 ? gemm_tc_kernel<0> : mode == 1 ? gemm_tc_kernel<1> : gemm_tc_kernel<2>;
+    kernel<<<grid, GT_THREADS, GT_SMEM_ALLOC, stream>>>(xm, wm, (const __nv_bfloat16*)bias, (__nv_bfloat16*)out, M, N, K, ldo, mode ? I : 0,
+                                                        (int*)status);
     return msgl_check_launch();
 }
 
 // out = sum over the ranges of part[range][M][N], added in range order (the result does not depend on timing), then bias or
 // SwiGLU and one rounding; a thread takes 4 neighbouring output columns of one token.
-template <bool SWIGLU>
+template <int GLU>
 __global__ void gemm_splitk_reduce_kernel(const float* __restrict__ part, int splits, int M, int N, int I,
                                           const __nv_bfloat16* __restrict__ bias, __nv_bfloat16* __restrict__ out, long long ldo) {
     pdl_launch_dependents();
     pdl_wait();
     pdl_after_wait();
-    const int n_out = SWIGLU ? I : N;
+    const int n_out = GLU ? I : N;
     const int per_row = (n_out + 3) / 4;
     const long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x;
     if (idx >= (long long)M * per_row) return;
     const int m = (int)(idx / per_row), c = (int)(idx - (long long)m * per_row) * 4;
     const size_t plane = (size_t)M * N;
     float a[4] = {0.f, 0.f, 0.f, 0.f}, u[4] = {0.f, 0.f, 0.f, 0.f};
-    const bool whole = c + 4 <= n_out && (!SWIGLU || (I & 3) == 0);
+    const bool whole = c + 4 <= n_out && (!GLU || (I & 3) == 0);
     for (int sp = 0; sp < splits; ++sp) {
         const float* row = part + sp * plane + (size_t)m * N;
         if (whole) {
             const float4 v = __ldcg(reinterpret_cast<const float4*>(row + c));
             a[0] += v.x; a[1] += v.y; a[2] += v.z; a[3] += v.w;
-            if (SWIGLU) {
+            if (GLU) {
                 const float4 w = __ldcg(reinterpret_cast<const float4*>(row + I + c));
                 u[0] += w.x; u[1] += w.y; u[2] += w.z; u[3] += w.w;
             }
         } else {
             for (int e = 0; e < 4; ++e)
-                if (c + e < n_out) { a[e] += __ldcg(row + c + e); if (SWIGLU) u[e] += __ldcg(row + I + c + e); }
+                if (c + e < n_out) { a[e] += __ldcg(row + c + e); if (GLU) u[e] += __ldcg(row + I + c + e); }
         }
     }
     __nv_bfloat16* orow = out + (size_t)m * ldo + c;
     for (int e = 0; e < 4; ++e) {
         if (c + e >= n_out) break;
         float y = a[e];
-        if (SWIGLU) y = y / (1.f + expf(-y)) * u[e];
-        else if (bias != nullptr) y += __bfloat162float(bias[c + e]);
+        if (GLU) {
+            if (bias != nullptr) { y += __bfloat162float(bias[c + e]); u[e] += __bfloat162float(bias[I + c + e]); }
+            y = glu_act<GLU>(y) * u[e];
+        } else if (bias != nullptr) y += __bfloat162float(bias[c + e]);
         orow[e] = __float2bfloat16_rn(y);
     }
 }
@@ -508,10 +513,10 @@ MSGL_API int msgl_gemm_tc2_splitk(const void* W, const void* X, const void* bias
     if (N <= 0 || K <= 0 || (K & 7) || (ldx & 7) || (ldo & 7) || status == nullptr) return MSGL_ERR_SIZE;
     if (((uintptr_t)W | (uintptr_t)X | (uintptr_t)out) & 15) return MSGL_ERR_ALIGN;
     const int I = N / 2;
-    if (mode == 1 && ((N & 1) || (I & 7) || bias != nullptr)) return MSGL_ERR_SIZE;
+    if (mode < 0 || mode > 2 || (mode != MSGL_GLU_NONE && ((N & 1) || (I & 7)))) return MSGL_ERR_SIZE;
     CUtensorMap xm, wm;
     if (!tc_matrix_map(X, M, K, ldx * 2, 128, &xm) || !tc_matrix_map(W, N, K, (long long)K * 2, 128, &wm)) return MSGL_ERR_SIZE;
-    const int n_valid = mode == 1 ? I : N, bn_out = mode == 1 ? 128 : 256;
+    const int n_valid = mode ? I : N, bn_out = mode ? 128 : 256;
     const long long tiles = (long long)((M + 255) / 256) * ((n_valid + bn_out - 1) / bn_out) * splits;      // work items
     cudaLaunchConfig_t cfg = {};
     cudaLaunchAttribute attr[2];
@@ -521,40 +526,37 @@ MSGL_API int msgl_gemm_tc2_splitk(const void* W, const void* X, const void* bias
     attr[1].val.programmaticStreamSerializationAllowed = 1;
     cfg.blockDim = dim3(GT2_THREADS); cfg.dynamicSmemBytes = GT2_SMEM_ALLOC; cfg.stream = stream; cfg.attrs = attr;
     cfg.numAttrs = msgl_pdl_enabled() ? 2 : 1;
-    static int pairs_of[MSGL_MAX_DEVICES][2] = {};      // per device and mode: how many pairs the device holds at once (asked once, outside any capture)
+    auto* kernel = mode == 0 ? gemm_tc2_kernel<0> : mode == 1 ? gemm_tc2_kernel<1> : gemm_tc2_kernel<2>;
+    static int pairs_of[MSGL_MAX_DEVICES][3] = {};      // per device and mode: how many pairs the device holds at once (asked once, outside any capture)
     int* max_pairs = pairs_of[msgl_device()];
     if (max_pairs[mode] == 0) {
-        cudaError_t e = mode == 1
-            ? cudaFuncSetAttribute(gemm_tc2_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)GT2_SMEM_ALLOC)
-            : cudaFuncSetAttribute(gemm_tc2_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)GT2_SMEM_ALLOC);
+        cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)GT2_SMEM_ALLOC);
         if (e != cudaSuccess) return msgl_check_launch();
         const int sms = msgl_sm_count();
         int n = 0;
         cfg.gridDim = dim3(2 * (sms / 2));
-        e = mode == 1 ? cudaOccupancyMaxActiveClusters(&n, gemm_tc2_kernel<true>, &cfg)
-                      : cudaOccupancyMaxActiveClusters(&n, gemm_tc2_kernel<false>, &cfg);
+        e = cudaOccupancyMaxActiveClusters(&n, kernel, &cfg);
         if (e != cudaSuccess || n <= 0) { cudaGetLastError(); return MSGL_ERR_SIZE; }
         max_pairs[mode] = n < sms / 2 ? n : sms / 2;
     }
     const int pairs = (int)(tiles < max_pairs[mode] ? tiles : max_pairs[mode]);
     cfg.gridDim = dim3(2 * pairs);
-    const __nv_bfloat16* b = mode == 1 ? nullptr : (const __nv_bfloat16*)bias;
+    const __nv_bfloat16* b = (const __nv_bfloat16*)bias;
     __nv_bfloat16* o = (__nv_bfloat16*)out;
     int* st = (int*)status;
-    const int Iarg = mode == 1 ? I : 0;
+    const int Iarg = mode ? I : 0;
     float* part = (float*)partials;
     if (splits <= 1) part = nullptr;
-    cudaError_t e = mode == 1 ? cudaLaunchKernelEx(&cfg, gemm_tc2_kernel<true>, xm, wm, b, o, M, N, K, ldo, Iarg, st, splits, part)
-                              : cudaLaunchKernelEx(&cfg, gemm_tc2_kernel<false>, xm, wm, b, o, M, N, K, ldo, Iarg, st, splits, part);
+    const cudaError_t e = cudaLaunchKernelEx(&cfg, kernel, xm, wm, b, o, M, N, K, ldo, Iarg, st, splits, part);
     (void)e;
     if (part == nullptr) return msgl_check_launch();
     // the ranges' partial sums -> output (bias / SwiGLU, one rounding), in range order
-    const int n_out = mode == 1 ? I : N;
+    const int n_out = mode ? I : N;
     const long long groups = (long long)M * ((n_out + 3) / 4);
     const int threads = 256;
     const unsigned blocks = (unsigned)((groups + threads - 1) / threads);
-    if (mode == 1) msgl_launch_pdl(gemm_splitk_reduce_kernel<true>, dim3(blocks), dim3(threads), 0, stream, (const float*)part, splits, M, N, I, b, o, ldo);
-    else msgl_launch_pdl(gemm_splitk_reduce_kernel<false>, dim3(blocks), dim3(threads), 0, stream, (const float*)part, splits, M, N, I, b, o, ldo);
+    auto* reduce = mode == 0 ? gemm_splitk_reduce_kernel<0> : mode == 1 ? gemm_splitk_reduce_kernel<1> : gemm_splitk_reduce_kernel<2>;
+    msgl_launch_pdl(reduce, dim3(blocks), dim3(threads), 0, stream, (const float*)part, splits, M, N, I, b, o, ldo);
     return msgl_check_launch();
 }
 
@@ -566,7 +568,7 @@ MSGL_API int msgl_gemm_tc2(const void* W, const void* X, const void* bias, void*
 // How many ranges of K the split-K product should use for these sizes on the current device: the count (at most 8, at
 // least 8 slabs of 64 each) for which the work items fill the pairs of SMs in the fewest rounds of the shortest items.
 MSGL_API int msgl_gemm_tc2_splits(int M, int N, int K, int mode) {
-    const int n_out = mode == 1 ? N / 2 : N, bn_out = mode == 1 ? 128 : 256;
+    const int n_out = mode ? N / 2 : N, bn_out = mode ? 128 : 256;
     const long long tiles = (long long)((M + 255) / 256) * ((n_out + bn_out - 1) / bn_out);
     const int n_slabs = (K + GT_BK - 1) / GT_BK;
     const int pairs = msgl_sm_count() / 2;

@@ -18,17 +18,18 @@
 //                              (a chunk's own sum and decay; the chunks' start states in order; outputs from both)
 //   gate_group_norm_kernel     (y * silu(z)) RMS-normed in equal parts of the row, times a weight
 //   unary_act_kernel           relu(x)^2 (and the other activations), times a constant
-//   route_kernel               router logits in float32, sigmoid scores, correction, limitation to the best groups, the top
-//                              experts and their weights: one block per token
-//                              (or, in its softmax mode, the largest logits and the softmax over the chosen ones; a further row's
-//                              sigmoid per token beside them)
+//   route_kernel               router logits in float32, sigmoid or softmax scores, correction, limitation to the best groups,
+//                              the top experts and their weights: one block per token
+//                              (or the largest logits and the softmax over the chosen ones; a further row's sigmoid per token
+//                              beside them)
 //   expert_gate_up_kernel, expert_down_kernel      the chosen experts' products for a few tokens, straight from the experts'
 //                              stacked weights (weight-streaming, one warp per output row); silu(gate) * up or the clamped
 //                              form; an extra term (a shared expert's output times a gate per token) joins the sum
+//   expert_up_kernel, expert_down_plain_kernel     the same for experts without a gate, of which some stand for the input itself
 //   clamped_glu_kernel         min(gate, limit) * sigmoid(1.702 ...) * (clamp(up) + 1) of a packed [gate | up] row
 //   expert_count_kernel, expert_place_kernel, expert_gather_kernel, expert_combine_kernel    many tokens: the (token, choice)
 //                              pairs in the order of their experts (stable), rows gathered for one product per expert, and the
-//                              weighted sum of every token's rows
+//                              weighted sum of every token's rows (expert_combine_self_kernel: pairs without a row add the input)
 //
 // Scores, weights, norms, gates, decays, states and everything that enters a recurrence are float32; T is the type of the
 // activations between kernels (float or bfloat16).  The order of every sum at a position is fixed by absolute positions, never
@@ -1899,7 +1900,7 @@ __global__ void __launch_bounds__(256) expert_count_kernel(const int* __restrict
 }
 
 __global__ void __launch_bounds__(256) expert_place_kernel(const int* __restrict__ idx, int n_pairs, const int* __restrict__ counts,
-                                                           int n_experts, int* __restrict__ place) {
+                                                           int n_experts, int* __restrict__ place, int* __restrict__ ends) {
     __shared__ int warp_tot[8];
     __shared__ int base_sh;
     const int e = blockIdx.x, tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
@@ -1912,6 +1913,7 @@ __global__ void __launch_bounds__(256) expert_place_kernel(const int* __restrict
         int b = 0;
         for (int i = 0; i < e; ++i) b += counts[i];
         base_sh = b;
+        if (ends != nullptr) ends[e] = b + counts[e];    // the expert's rows end here
     }
     __syncthreads();
     int base = base_sh;
@@ -2023,11 +2025,11 @@ __global__ void expert_combine_kernel(const Y* __restrict__ y, const int* __rest
     }
 }
 
-MSGL_API int msgl_expert_order(const int* idx, int n_pairs, int E, int* counts, int* place, cudaStream_t stream) {
+MSGL_API int msgl_expert_order(const int* idx, int n_pairs, int E, int* counts, int* place, int* ends, cudaStream_t stream) {
     if (n_pairs <= 0) return MSGL_OK;
     if (E <= 0 || n_pairs >= (1 << 24)) return MSGL_ERR_SIZE;
     expert_count_kernel<<<E, 256, 0, stream>>>(idx, n_pairs, counts);
-    expert_place_kernel<<<E + 1, 256, 0, stream>>>(idx, n_pairs, counts, E, place);
+    expert_place_kernel<<<E + 1, 256, 0, stream>>>(idx, n_pairs, counts, E, place, ends);
     return msgl_check_launch();
 }
 

@@ -58,9 +58,11 @@ def _align4(n: int) -> int:
 
 
 class _Layout:
-    """Offsets of the fields inside the int32 staging buffer of a step."""
+    """Offsets of the fields inside the int32 staging buffer of a step.  The per-group lists have one entry per plan (see
+    ModelRunner): `owner[p]` is the first plan of plan p's cache group, whose token slots and block-table rows p shares."""
 
-    def __init__(self, T: int, B: int, W: int, max_pages: Sequence[int], even_nb: Optional[Sequence[int]] = None):
+    def __init__(self, T: int, B: int, W: int, max_pages: Sequence[int], even_nb: Optional[Sequence[int]] = None,
+                 owner: Optional[Sequence[int]] = None):
         self.T, self.B, self.W, self.max_pages = T, B, W, list(max_pages)
         self.even_nb = list(even_nb) if even_nb is not None else [0] * len(self.max_pages)      # 0: no even cut for the group
         off = 0
@@ -74,12 +76,13 @@ class _Layout:
         self.input_ids, self.positions, self.token_req = take(T), take(T), take(T)
         self.q_start, self.kv_len, self.slots, self.want = take(B + 1), take(B), take(B), take(W)
         self.out_loc, self.nsplit, self.order, self.even, self.table = [], [], [], [], []
-        for mp, nb in zip(max_pages, self.even_nb):
-            self.out_loc.append(take(T))
+        for p, (mp, nb) in enumerate(zip(max_pages, self.even_nb)):
+            own = owner is None or owner[p] == p
+            self.out_loc.append(take(T) if own else self.out_loc[owner[p]])
             self.nsplit.append(take(B))
             self.order.append(take(B))
             self.even.append(take(ops.even_cut_size(B, nb) if nb else 0))
-            self.table.append(take(B * mp))
+            self.table.append(take(B * mp) if own else self.table[owner[p]])
         self.size = off
 
 
@@ -324,28 +327,44 @@ class ModelRunner:
         self.device_meta = os.environ.get("MSGL_DEVICE_META", "1") != "0"
         self._dev_compact = None
         self.last_h2d_bytes = 0          # bytes of the last step's host-to-device copy of its fields
-        self.last_plan: Dict[str, object] = {}       # the last step's kv splits per group and the decode graph it replayed
-        self._group_geom = []
-        for g in self.mgr.groups:
-            # the kv splits are planned for the caches whose launches take them: the first of the engine's attention kernels
-            cid = next((c for c in g.cache_ids if needs[c].library == "attention"), g.cache_ids[0])
-            need = needs[cid]
-            G = max(need.q_heads // need.n_kv_heads, 1) if need.q_heads else 1
-            if need.library != "attention":
-                # a mixer with attention kernels of its own: its launches take every request whole (no kv splits)
-                self._group_geom.append((need.n_kv_heads, G, 0, 0))
-                continue
-            qt = ops.attention_tile_tokens(ops.VARIANT_MMA_DECODE, G, need.head_dim) if ops.mma_supported(need.head_dim, self.dtype) \
-                else ops.attention_tile_tokens(ops.VARIANT_SIMT, G)
-            self._group_geom.append((need.n_kv_heads, G, ops.decode_blocks_per_sm(need.head_dim, self.dtype, G), qt))
+        self.last_plan: Dict[str, object] = {}       # the last step's kv splits per plan and the decode graph it replayed
+        # Plans: the attention launches of a cache group whose caches differ in geometry (a grouped-query attention with 8 kv
+        # heads beside a cache of latents with one, say) want their keys cut differently, so every geometry of a group has kv
+        # splits and an order of its own; token slots and block tables are the group's.  Mixers with attention kernels of their
+        # own take every request whole (or cut it themselves): they share the group's first plan, or have one without splits.
+        self._group_geom: List[Tuple[int, int, int, int]] = []       # per plan: kv heads, q heads per kv head, blocks per SM, tile
+        self._plan_group: List[int] = []                             # per plan: its cache group
+        self._plan_of_cache: Dict[object, int] = {}
+        for gi, g in enumerate(self.mgr.groups):
+            first, of_geom = len(self._plan_group), {}
+            for cid in g.cache_ids:
+                need = needs[cid]
+                if need.library != "attention":
+                    continue
+                G = max(need.q_heads // need.n_kv_heads, 1) if need.q_heads else 1
+                qt = ops.attention_tile_tokens(ops.VARIANT_MMA_DECODE, G, need.head_dim) if ops.mma_supported(need.head_dim, self.dtype) \
+                    else ops.attention_tile_tokens(ops.VARIANT_SIMT, G)
+                geom = (need.n_kv_heads, G, ops.decode_blocks_per_sm(need.head_dim, self.dtype, G), qt)
+                if geom not in of_geom:
+                    of_geom[geom] = len(self._plan_group)
+                    self._plan_group.append(gi)
+                    self._group_geom.append(geom)
+                self._plan_of_cache[cid] = of_geom[geom]
+            if not of_geom:
+                need = needs[g.cache_ids[0]]
+                self._plan_group.append(gi)
+                self._group_geom.append((need.n_kv_heads, max(need.q_heads // need.n_kv_heads, 1) if need.q_heads else 1, 0, 0))
+            for cid in g.cache_ids:
+                self._plan_of_cache.setdefault(cid, first)
+        self._plan_owner = [self._plan_group.index(gi) for gi in self._plan_group]
         # blocks per kv head of a decode launch with an even cut of the keys: what the SMs hold at once; empty unless the
         # decode kernel of every group takes such a cut
         self._even_nb: List[int] = []
         if self.dtype == torch.bfloat16 and self.mgr.groups and all(geom[2] for geom in self._group_geom) and \
                 all(needs[cid].even_cut for g in self.mgr.groups for cid in g.cache_ids):
             ok = True
-            for g, (n_kv, G, per_sm, _) in zip(self.mgr.groups, self._group_geom):
-                head_dim = needs[g.cache_ids[0]].head_dim
+            for p, (n_kv, G, per_sm, _) in enumerate(self._group_geom):
+                head_dim = next(needs[cid].head_dim for cid, q in self._plan_of_cache.items() if q == p)
                 ok = ok and ops.decode_even_ok(head_dim, self.dtype, G) and self.sm_count * per_sm >= n_kv
             if ok:
                 self._even_nb = [max(1, self.sm_count * per_sm // n_kv) for (n_kv, G, per_sm, _) in self._group_geom]
@@ -402,9 +421,13 @@ class ModelRunner:
         """Blocks of the whole-step decode kernel for a step of `tokens` single tokens with all logits wanted; 0 if the
         model or the size goes kernel by kernel."""
         fd = self.model.fused_decode
-        if fd is None or not 0 < tokens <= ops.FUSED_DECODE_MAX_TOKENS or len(self.mgr.groups) != 1:
+        if fd is None or not 0 < tokens <= ops.FUSED_DECODE_MAX_TOKENS or len(self._plan_group) != 1:
             return 0
         return fd.blocks_for(tokens)
+
+    def _plans(self):
+        """(plan, its cache group) of every plan."""
+        return [(p, self.mgr.groups[gi]) for p, gi in enumerate(self._plan_group)]
 
     def _plan_splits(self, gi: int, q_lens: Sequence[int], kv_lens: Sequence[int], cap: int,
                      long_cap: Optional[int] = None, fused_blocks: int = 0) -> List[int]:
@@ -415,7 +438,7 @@ class ModelRunner:
         if fused_blocks:          # the whole-step kernel: its blocks are the places, a unit is a (request, kv head, split)
             per_sm, warps, qt = max(fused_blocks // self.sm_count, 1), self.FUSED_WARPS, 1
         return plan_kv_splits(q_lens, kv_lens, n_kv=n_kv, group=G, blocks_per_sm=per_sm, tile_tokens=qt,
-                              window=self.mgr.groups[gi].window, cap=cap, long_cap=long_cap, sm_count=self.sm_count,
+                              window=self.mgr.groups[self._plan_group[gi]].window, cap=cap, long_cap=long_cap, sm_count=self.sm_count,
                               warps=warps)
 
     def _fill(self, host: np.ndarray, lay: _Layout, entries: Sequence[StepEntry], starts: Sequence[int],
@@ -425,7 +448,7 @@ class ModelRunner:
         T, B = lay.T, lay.B
         host[:lay.size] = 0
         n_ent = len(entries)
-        for gi in range(len(self.mgr.groups)):
+        for gi, _ in self._plans():
             host[lay.order[gi]: lay.order[gi] + B] = np.arange(B, dtype=np.int32)
         if n_ent and all(len(e.tokens) == 1 for e in entries):
             # one token per request (decode): every field with a handful of vector operations
@@ -438,7 +461,7 @@ class ModelRunner:
             host[lay.kv_len: lay.kv_len + n_ent] = pos + 1
             host[lay.slots: lay.slots + n_ent] = slots
             P = self.page_size
-            for gi, g in enumerate(self.mgr.groups):
+            for gi, g in self._plans():
                 mp = lay.max_pages[gi]
                 host[lay.out_loc[gi]: lay.out_loc[gi] + n_ent] = g.table[slots, pos // P].astype(np.int64) * P + pos % P
                 host[lay.nsplit[gi]: lay.nsplit[gi] + n_ent] = nsplits[gi]
@@ -459,18 +482,20 @@ class ModelRunner:
                 host[lay.q_start + r] = t
                 host[lay.kv_len + r] = s + n
                 host[lay.slots + r] = e.slot
-                for gi in range(len(self.mgr.groups)):
-                    host[lay.out_loc[gi] + t: lay.out_loc[gi] + t + n] = self.mgr.slot_mapping(gi, e.slot, s, n)
-                    row = self.mgr.block_table_row(gi, e.slot)
+                for gi, group in enumerate(self._plan_group):
+                    host[lay.nsplit[gi] + r] = nsplits[gi][r]
+                    if self._plan_owner[gi] != gi:
+                        continue
+                    host[lay.out_loc[gi] + t: lay.out_loc[gi] + t + n] = self.mgr.slot_mapping(group, e.slot, s, n)
+                    row = self.mgr.block_table_row(group, e.slot)
                     mp = lay.max_pages[gi]
                     host[lay.table[gi] + r * mp: lay.table[gi] + r * mp + len(row)] = row
-                    host[lay.nsplit[gi] + r] = nsplits[gi][r]
                 t += n
         for r in range(len(entries), B):          # padding rows of a captured batch size
             host[lay.token_req + t] = r
             host[lay.q_start + r] = t
             host[lay.kv_len + r] = 1
-            for gi in range(len(self.mgr.groups)):
+            for gi, _ in self._plans():
                 host[lay.nsplit[gi] + r] = 1
             t += 1
         host[lay.q_start + B] = t
@@ -482,7 +507,7 @@ class ModelRunner:
             return dev[off: off + n]
 
         groups = []
-        for gi, g in enumerate(self.mgr.groups):
+        for gi, g in self._plans():
             mp = lay.max_pages[gi]
             groups.append(GroupContext(block_table=v(lay.table[gi], lay.B * mp).view(lay.B, mp),
                                        out_loc=v(lay.out_loc[gi], lay.T),
@@ -502,7 +527,7 @@ class ModelRunner:
     def _caches(self, ctx: StepContext) -> Dict[int, object]:
         views: Dict[int, object] = {}
         for cid, (k, v) in self.storage.kv.items():
-            views[cid] = KVCacheView(k, v, ctx.groups[self.mgr.group_of_cache[cid]], self.page_size)
+            views[cid] = KVCacheView(k, v, ctx.groups[self._plan_of_cache[cid]], self.page_size)
         for cid, st in self.storage.state.items():
             views[cid] = StateCacheView(st)
         # the caches of a mixer with several needs, (c, 0), (c, 1), ..., reach it as one tuple under the run's id c
@@ -572,11 +597,11 @@ class ModelRunner:
                 ops.poll_status()
         else:
             fused = self._fused_blocks(B) if all_last else 0
-            nsplits = [self._plan_splits(gi, q_lens, kv_lens, MAX_KV_SPLIT, fused_blocks=fused) for gi in range(len(self.mgr.groups))]
+            nsplits = [self._plan_splits(gi, q_lens, kv_lens, MAX_KV_SPLIT, fused_blocks=fused) for gi, _ in self._plans()]
             max_splits = [max(ns) for ns in nsplits]
             self.last_plan = {"graph_key": None, "nsplits": nsplits, "max_split": max_splits}
-            max_pages = [max(int(g.n_pages[e.slot]) for e in entries) for g in self.mgr.groups]
-            lay = _Layout(T, B, len(want_rows), max_pages)
+            max_pages = [max(int(g.n_pages[e.slot]) for e in entries) for _, g in self._plans()]
+            lay = _Layout(T, B, len(want_rows), max_pages, owner=self._plan_owner)
             host, idx = self._pinned_buffer(lay.size)
             self._fill(host.numpy(), lay, entries, starts, want_rows, nsplits)
             if self._dev_staging is None or self._dev_staging.numel() < lay.size:
@@ -624,18 +649,18 @@ class ModelRunner:
     def _step_graph(self, entries, starts, q_lens, kv_lens, prev_ids=None) -> torch.Tensor:
         B = len(entries)
         b = self._bucket(B)
-        need_pages = [max(int(g.n_pages[e.slot]) for e in entries) for g in self.mgr.groups]
+        need_pages = [max(int(g.n_pages[e.slot]) for e in entries) for _, g in self._plans()]
         mp = tuple(max(8, 1 << (n - 1).bit_length()) for n in need_pages)
         # the graph fixes the launch's split dimension: the narrow one suits requests of like length; a batch
         # with a request far longer than the rest takes a second graph with room for more pieces
-        room = [self._graph_max_split(gi, b) for gi in range(len(self.mgr.groups))]
+        room = [self._graph_max_split(gi, b) for gi, _ in self._plans()]
         narrow = [min(c, MANY_SPLITS) for c in room]
         fused = self._fused_blocks(b)
         even_cuts = None
         if not fused and self._even_nb and self._wants_even_cut(kv_lens):
             # long contexts: the keys of all requests dealt out evenly over as many blocks as the SMs hold at once
             pieces = [min(EVEN_MAX_PIECES, nb) for nb in self._even_nb]
-            even_cuts = [plan_even_cut(kv_lens, g.window, nb, mx) for g, nb, mx in zip(self.mgr.groups, self._even_nb, pieces)]
+            even_cuts = [plan_even_cut(kv_lens, g.window, nb, mx) for (_, g), nb, mx in zip(self._plans(), self._even_nb, pieces)]
             nsplits = [c[5].tolist() for c in even_cuts]
             key = (b, mp, "even")
             gr = self._graphs.get(key)
@@ -644,7 +669,7 @@ class ModelRunner:
                 self._graphs[key] = gr
         else:
             nsplits = [self._plan_splits(gi, q_lens, kv_lens, room[gi], max(narrow[gi], WIDE_KV_SPLIT), fused_blocks=fused)
-                       for gi in range(len(self.mgr.groups))]
+                       for gi, _ in self._plans()]
             # blocks of pieces that a request does not have leave at once, but they are launched: a graph with the split
             # dimension of long contexts (up to MAX_KV_SPLIT) is kept apart from the one that every other step replays
             wide = any(max(ns) > cap for ns, cap in zip(nsplits, narrow))
@@ -690,8 +715,8 @@ class ModelRunner:
         buffer: token id, slot and position of every request, its kv splits per cache group, and per group the table
         rows of the requests whose pages changed since the last such step (whole rows; a request gets a page every
         page_size tokens)."""
-        lay, B, G = gr.layout, len(entries), len(self.mgr.groups)
-        rows = [self.mgr.take_dirty_rows(gi) for gi in range(G)]
+        lay, B, G = gr.layout, len(entries), len(self._plan_group)
+        rows = [self.mgr.take_dirty_rows(g) if self._plan_owner[p] == p else [] for p, g in enumerate(self._plan_group)]
         n_delta = [1 + 3 * len(r) + sum(len(t) for _, t in r) for r in rows]
         n_even = [ops.even_cut_size(b, nb) if (nb and even_cuts is not None) else 0 for nb in lay.even_nb]
         size = (3 + G) * B + sum(_align4(n) for n in n_delta) + sum(_align4(n) for n in n_even)
@@ -732,25 +757,25 @@ class ModelRunner:
         g0 = gr.dev
         for gi in range(G):
             if rows[gi]:
-                ops.table_delta(dev[d_off[gi]: d_off[gi] + n_delta[gi]], len(rows[gi]), self.storage.tables[gi])
+                ops.table_delta(dev[d_off[gi]: d_off[gi] + n_delta[gi]], len(rows[gi]), self.storage.tables[self._plan_group[gi]])
             mp = lay.max_pages[gi]
-            ops.decode_meta(dev[0:B], dev[B:2 * B], dev[2 * B:3 * B], dev[ns_off[gi]:ns_off[gi] + B], B, b, self.storage.tables[gi],
+            ops.decode_meta(dev[0:B], dev[B:2 * B], dev[2 * B:3 * B], dev[ns_off[gi]:ns_off[gi] + B], B, b, self.storage.tables[self._plan_group[gi]],
                             self.page_size, mp, gi == 0,
                             input_ids=g0[lay.input_ids:], positions=g0[lay.positions:], token_req=g0[lay.token_req:],
                             q_start=g0[lay.q_start:], kv_len=g0[lay.kv_len:], slots=g0[lay.slots:],
                             out_loc=g0[lay.out_loc[gi]:], nsplit=g0[lay.nsplit[gi]:], block_table=g0[lay.table[gi]:],
-                            order=g0[lay.order[gi]:], window=int(self.mgr.groups[gi].window or 0),
+                            order=g0[lay.order[gi]:], window=int(self.mgr.groups[self._plan_group[gi]].window or 0),
                             even_in=dev[e_off[gi]: e_off[gi] + n_even[gi]] if n_even[gi] else None,
                             even_out=g0[lay.even[gi]:] if n_even[gi] else None)
 
     def _capture(self, b: int, mp: Tuple[int, ...], max_split: Sequence[int], even_nb: Optional[Sequence[int]] = None) -> _Graph:
         gr = _Graph()
-        lay = _Layout(b, b, b, mp, even_nb)
+        lay = _Layout(b, b, b, mp, even_nb, owner=self._plan_owner)
         gr.layout = lay
         gr.dev = torch.zeros(lay.size, dtype=torch.int32, device=self.device)
         gr.max_split = list(max_split)
         host = np.zeros(lay.size, dtype=np.int32)
-        self._fill(host, lay, [], [], list(range(b)), [[1] * b for _ in self.mgr.groups])
+        self._fill(host, lay, [], [], list(range(b)), [[1] * b for _ in self._plan_group])
         gr.dev.copy_(torch.from_numpy(host))
         ctx = self._context(gr.dev, lay, [1] * b, [1] * b, [0] * b, gr.max_split, True, all_rows_wanted=True)
         caches = self._caches(ctx)

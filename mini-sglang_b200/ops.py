@@ -108,10 +108,12 @@ def _attn_lib(head_dim: int):
     lib = _attn.get(hd)
     if lib is None:
         lib = _build.attention_library(hd)
-        lib.msgl_attention.argtypes = [c_void_p] * 10 + [c_int] * 9 + [c_float] + [c_int] * 6 + [c_void_p, c_void_p, c_int, c_void_p]
+        lib.msgl_attention.argtypes = [c_void_p] * 10 + [c_int] * 9 + [c_float] + [c_int] * 6 + [c_void_p, c_void_p, c_int, c_void_p, c_void_p,
+                                       c_ll, c_void_p]
         lib.msgl_attention_window.argtypes = [c_void_p] * 10 + [c_int] * 9 + [c_float] + [c_int] * 6 + [c_void_p, c_int, c_void_p, c_int, c_void_p]
-        lib.msgl_attention_combine.argtypes = [c_void_p] * 5 + [c_int] * 5 + [c_void_p]
-        lib.msgl_attention_tc.argtypes = [c_void_p] * 7 + [c_int] * 8 + [c_float] + [c_int] * 5 + [c_void_p, c_int, c_void_p, c_int, c_void_p]
+        lib.msgl_attention_combine.argtypes = [c_void_p] * 5 + [c_int] * 5 + [c_void_p, c_void_p, c_ll, c_void_p]
+        lib.msgl_attention_tc.argtypes = [c_void_p] * 7 + [c_int] * 8 + [c_float] + [c_int] * 5 + [c_void_p, c_int, c_void_p, c_int, c_void_p,
+                                         c_void_p, c_ll, c_void_p]
         lib.msgl_attention_head_dim.restype = c_int
         _attn[hd] = lib
     return lib
@@ -370,12 +372,14 @@ _tc2_usable = True
 def attention_tc(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, *,
                  q_start: torch.Tensor, kv_len: torch.Tensor, block_table: torch.Tensor, n_kv: int, page_size: int,
                  window: int, scale: float, qlen_min: int, qlen_max: int, q_lens: Sequence[int], keep_first: int = 0,
-                 bias_log2: Optional[torch.Tensor] = None) -> bool:
+                 bias_log2: Optional[torch.Tensor] = None, null_log2: Optional[torch.Tensor] = None,
+                 gate: Optional[torch.Tensor] = None) -> bool:
     """Prefill attention on tcgen05 tensor cores for the requests with q_len in [qlen_min, qlen_max];
     q_lens: the host's copy of every request's number of query tokens (to size the grid).  keep_first, bias_log2: as in
     `attention`; they are taken by the kernel on pairs of query tiles only (TMA page sizes), and the call returns False,
-    having launched nothing, where that kernel cannot run."""
+    having launched nothing, where that kernel cannot run.  null_log2, gate: as in `attention`, taken by both kernels."""
     global _tc2_usable
+    gate_stride = _attention_extras(q, null_log2, gate)
     _need_cuda(q, out, k_cache, v_cache, q_start, kv_len, block_table)
     T, n_q, d = q.shape
     B = kv_len.numel()
@@ -401,7 +405,8 @@ def attention_tc(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_ca
         code = _attn_lib(d).msgl_attention_tc(
             _ptr(q), _ptr(out), _ptr(k_cache), _ptr(v_cache), _ptr(q_start), _ptr(kv_len), _ptr(block_table), B, T, n_q,
             n_kv, d, page_size, block_table.stride(0), window, float(scale), qlen_min, qlen_max, grid_x, pages, version,
-            _ptr(status), int(keep_first), _ptr(bias_log2), bias_log2.shape[1] if bias_log2 is not None else 0, _stream())
+            _ptr(status), int(keep_first), _ptr(bias_log2), bias_log2.shape[1] if bias_log2 is not None else 0, _ptr(null_log2), _ptr(gate),
+            gate_stride, _stream())
         if code == 2 and version == 2:        # no tensor maps here (driver without the encoder, unaligned cache): one-tile kernel
             _tc2_usable = False
             if ext:
@@ -457,19 +462,36 @@ def mma_supported(head_dim: int, dtype: torch.dtype) -> bool:
     return dtype == torch.bfloat16 and head_dim in _build.MMA_HEAD_DIMS
 
 
+def _attention_extras(q: torch.Tensor, null_log2: Optional[torch.Tensor], gate: Optional[torch.Tensor]) -> int:
+    """Checks the term without a key and the output gate of an attention launch -> the gate's row stride."""
+    _need_cuda(null_log2, gate)
+    T, n_q, d = q.shape
+    if null_log2 is not None:
+        assert null_log2.dtype == torch.float32 and null_log2.numel() == n_q and null_log2.is_contiguous()
+    if gate is None:
+        return 0
+    assert gate.dtype == q.dtype and gate.shape[0] == T
+    return _rows_view(gate, n_q * d, "gate")
+
+
 def attention(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, *,
               q_start: torch.Tensor, kv_len: torch.Tensor, block_table: torch.Tensor,
               nsplit: Optional[torch.Tensor], part_o: Optional[torch.Tensor], part_ml: Optional[torch.Tensor],
               n_kv: int, page_size: int, window: int, max_split: int, scale: float, qlen_min: int, qlen_max: int,
               uniform_decode: bool, variant: int, grid_x: int, order: Optional[torch.Tensor] = None,
               even: Optional[torch.Tensor] = None, even_nb: int = 0, keep_first: int = 0,
-              bias_log2: Optional[torch.Tensor] = None) -> None:
+              bias_log2: Optional[torch.Tensor] = None, null_log2: Optional[torch.Tensor] = None,
+              gate: Optional[torch.Tensor] = None) -> None:
     """One launch of the paged attention kernel over the requests whose q_len lies in
     [qlen_min, qlen_max]; see csrc/attention.cu for the meaning of every argument.  keep_first: with a window, the first
     keys of a request that stay visible whatever the window; bias_log2: float32 [heads, L], added to the scaled score in
     log2 units by distance min(i - j, L - 1) (both: the bfloat16 mma kernels only, see `window_bias_supported`).  `order` (uniform decode only):
     int32 [B], a permutation of the requests; the launch's i-th block along x takes request order[i].  `even`: the even cut
-    of a decode step's keys over `even_nb` blocks per kv head (engine/step.py: plan_even_cut) in place of `grid_x` blocks."""
+    of a decode step's keys over `even_nb` blocks per kv head (engine/step.py: plan_even_cut) in place of `grid_x` blocks.
+    null_log2: float32 [heads], the score in log2 units of one more term in every softmax's denominator that has no key and no
+    value; gate [T, heads * d] (a view into packed rows): the output times sigmoid(gate), element by element.  Both enter where a
+    row is normalised, so a launch whose requests are cut hands them to `attention_combine` too."""
+    gate_stride = _attention_extras(q, null_log2, gate)
     _need_cuda(q, out, k_cache, v_cache, q_start, kv_len, block_table, nsplit, part_o, part_ml, order, even)
     T, n_q, d = q.shape
     B = kv_len.numel()
@@ -484,6 +506,7 @@ def attention(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_cache
     if keep_first or bias_log2 is not None:
         _need_cuda(bias_log2)
         assert even is None, "the even cut of a decode step knows no kept tokens and no bias"
+        assert null_log2 is None and gate is None, "a launch with kept tokens or a bias takes no further term and no gate"
         if bias_log2 is not None:
             assert bias_log2.dtype == torch.float32 and bias_log2.dim() == 2 and bias_log2.shape[0] == n_q and bias_log2.is_contiguous()
         code = _attn_lib(d).msgl_attention_window(
@@ -496,16 +519,19 @@ def attention(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_cache
     code = _attn_lib(d).msgl_attention(
         _ptr(q), _ptr(out), _ptr(k_cache), _ptr(v_cache), _ptr(q_start), _ptr(kv_len), _ptr(block_table),
         _ptr(nsplit), _ptr(part_o), _ptr(part_ml), B, T, n_q, n_kv, d, page_size, block_table.stride(0), window,
-        max_split, float(scale), qlen_min, qlen_max, int(uniform_decode), variant, grid_x, _dt(q), _ptr(order), _ptr(even), int(even_nb), _stream())
+        max_split, float(scale), qlen_min, qlen_max, int(uniform_decode), variant, grid_x, _dt(q), _ptr(order), _ptr(even), int(even_nb),
+        _ptr(null_log2), _ptr(gate), gate_stride, _stream())
     _check(code, f"attention (head size {d}, variant {variant})")
 
 
 def attention_combine(part_o: torch.Tensor, part_ml: torch.Tensor, token_req: Optional[torch.Tensor],
-                      nsplit: torch.Tensor, out: torch.Tensor, max_split: int) -> None:
+                      nsplit: torch.Tensor, out: torch.Tensor, max_split: int, null_log2: Optional[torch.Tensor] = None,
+                      gate: Optional[torch.Tensor] = None) -> None:
     _need_cuda(part_o, part_ml, token_req, nsplit, out)
+    gate_stride = _attention_extras(out, null_log2, gate)
     T, n_q, d = out.shape
     code = _attn_lib(d).msgl_attention_combine(_ptr(part_o), _ptr(part_ml), _ptr(token_req), _ptr(nsplit), _ptr(out),
-                                               T, n_q, d, max_split, _dt(out), _stream())
+                                               T, n_q, d, max_split, _dt(out), _ptr(null_log2), _ptr(gate), gate_stride, _stream())
     _check(code, "attention_combine")
 
 
@@ -549,15 +575,16 @@ _tc_gemm_usable = True
 
 
 def _tc_gemm(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor], mode: int) -> Optional[torch.Tensor]:
-    """x @ weight^T (mode 0) or SwiGLU of it (mode 1) by the tcgen05 kernel; None where it does not apply."""
+    """x @ weight^T (mode 0) or its gated activation (mode 1: SwiGLU, 2: ReGLU; bias [2I]) by the tcgen05 kernel; None where it
+    does not apply."""
     global _tc_gemm_usable
-    if not ((TC_GEMM == "all" or (TC_GEMM == "swiglu" and mode == 1)) and _tc_gemm_usable and x.dtype == torch.bfloat16 and weight.dtype == torch.bfloat16 and x.dim() == 2
+    if not ((TC_GEMM == "all" or (TC_GEMM == "swiglu" and mode != 0)) and _tc_gemm_usable and x.dtype == torch.bfloat16 and weight.dtype == torch.bfloat16 and x.dim() == 2
             and x.shape[0] >= TC_GEMM_MIN_M and x.stride(1) == 1 and x.stride(0) % 8 == 0 and weight.is_contiguous()
             and weight.shape[1] % 8 == 0 and (bias is None or bias.dtype == torch.bfloat16)):
         return None
     M, (N, K) = x.shape[0], weight.shape
-    n_out = N // 2 if mode == 1 else N
-    if n_out % 8 or (mode == 1 and N % 2):
+    n_out = N // 2 if mode else N
+    if n_out % 8 or (mode and N % 2):
         return None
     out = torch.empty((M, n_out), dtype=torch.bfloat16, device=x.device)
     fn = _lib().msgl_gemm_tc2 if TC_GEMM_CTAS == 2 else _lib().msgl_gemm_tc
@@ -581,7 +608,7 @@ _mid_splits = {}
 
 
 def _tc_gemm_mid(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor], mode: int) -> Optional[torch.Tensor]:
-    """x @ weight^T (mode 0) or SwiGLU of it (mode 1) for a middling number of rows by the split-K tcgen05 kernel; None where
+    """x @ weight^T (mode 0) or its gated activation (modes 1, 2) for a middling number of rows by the split-K tcgen05 kernel; None where
     it does not apply."""
     global _tc_gemm_usable
     if not (MID_GEMM and TC_GEMM != "0" and TC_GEMM_CTAS == 2 and _tc_gemm_usable and x.dtype == torch.bfloat16
@@ -590,8 +617,8 @@ def _tc_gemm_mid(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Ten
             and weight.shape[1] >= 512 and (bias is None or bias.dtype == torch.bfloat16)):
         return None
     M, (N, K) = x.shape[0], weight.shape
-    n_out = N // 2 if mode == 1 else N
-    if n_out % 8 or (mode == 1 and N % 16):
+    n_out = N // 2 if mode else N
+    if n_out % 8 or (mode and N % 16):
         return None
     key = (M, N, K, mode)
     splits = MID_GEMM_SPLITS or _mid_splits.get(key)
@@ -643,20 +670,37 @@ def linear(x: torch.Tensor, weight: torch.Tensor, bias: Optional[torch.Tensor] =
     return torch.nn.functional.linear(x, weight, bias)
 
 
+GLU_MODES = {0: 1, 4: 2}          # the ACT_ numbers whose gated products have fused kernels (silu, relu) -> the kernels' mode
+
+
+def linear_glu(x: torch.Tensor, gate_up: torch.Tensor, bias: Optional[torch.Tensor] = None, act: int = 0) -> torch.Tensor:
+    """act(x @ gate^T + bg) * (x @ up^T + bu) with gate_up = [gate; up] packed row-wise ([2I, H]) and bias = [bg; bu] or None;
+    act: one of the ACT_ numbers.  Where a kernel with the activation in its epilogue applies (silu and relu; a few rows, or
+    many rows in bfloat16) the [T, 2I] intermediate never exists."""
+    _need_cuda(x, gate_up, bias)
+    mode = GLU_MODES.get(act)
+    if mode is not None:
+        if _small_m_ok(x, gate_up, bias) and (gate_up.shape[0] // 2) % 8 == 0:
+            M, (N, K) = x.shape[0], gate_up.shape
+            out = torch.empty((M, N // 2), dtype=torch.bfloat16, device=x.device)
+            code = _small_m(gate_up, x, bias, out, M, N, K, N // 2, mode, 0)
+            _check(code, "gemm_small_m (gated)")
+            return out
+        y = _tc_gemm(x, gate_up, bias, mode) if x.shape[0] >= TC_GEMM_MIN_M else _tc_gemm_mid(x, gate_up, bias, mode)
+        if y is not None:
+            return y
+    gu = torch.nn.functional.linear(x, gate_up, bias)
+    if act == 0:
+        return swiglu(gu)
+    I = gate_up.shape[0] // 2
+    out = torch.empty((x.shape[0], I), dtype=x.dtype, device=x.device)
+    gated_act(gu[:, :I], gu[:, I:], out, act)
+    return out
+
+
 def linear_swiglu(x: torch.Tensor, gate_up: torch.Tensor) -> torch.Tensor:
-    """silu(x @ gate^T) * (x @ up^T) with gate_up = [gate; up] packed row-wise ([2I, H]).  For a few
-    rows the product and the activation are one kernel and the [T, 2I] intermediate never exists."""
-    _need_cuda(x, gate_up)
-    if _small_m_ok(x, gate_up, None) and (gate_up.shape[0] // 2) % 8 == 0:
-        M, (N, K) = x.shape[0], gate_up.shape
-        out = torch.empty((M, N // 2), dtype=torch.bfloat16, device=x.device)
-        code = _small_m(gate_up, x, None, out, M, N, K, N // 2, 1, 0)
-        _check(code, "gemm_small_m (swiglu)")
-        return out
-    y = _tc_gemm(x, gate_up, None, 1) if x.shape[0] >= TC_GEMM_MIN_M else _tc_gemm_mid(x, gate_up, None, 1)
-    if y is not None:
-        return y
-    return swiglu(torch.nn.functional.linear(x, gate_up))
+    """silu(x @ gate^T) * (x @ up^T): `linear_glu` without biases."""
+    return linear_glu(x, gate_up)
 
 
 # ---------------------------------------------------------------------------------------
@@ -1085,7 +1129,7 @@ def _gated_lib():
         lib.msgl_experts_few.argtypes = [c_void_p, c_ll] + [c_void_p] * 4 + [c_int, c_int, c_int, c_void_p, c_float, c_void_p, c_int, c_int,
                                                                             c_float, c_void_p, c_void_p, c_void_p]
         lib.msgl_clamped_glu.argtypes = [c_void_p, c_ll, c_int, c_float, c_void_p, c_int, c_int, c_void_p]
-        lib.msgl_expert_order.argtypes = [c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p]
+        lib.msgl_expert_order.argtypes = [c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p, c_void_p]
         lib.msgl_expert_gather.argtypes = [c_void_p, c_ll, c_void_p, c_int, c_int, c_void_p, c_int, c_int, c_void_p]
         lib.msgl_expert_combine.argtypes = [c_void_p, c_int, c_void_p, c_void_p, c_int, c_int, c_float, c_void_p, c_int, c_void_p, c_void_p,
                                             c_void_p]
@@ -1439,18 +1483,19 @@ def experts_few(h: torch.Tensor, gate_up: torch.Tensor, down: torch.Tensor, idx:
     return out
 
 
-def expert_order(idx: torch.Tensor, n_experts: int) -> Tuple[torch.Tensor, torch.Tensor]:
-    """idx int32 [T, top] -> (counts int32 [E]: pairs per expert; place int32 [T * top]: row of every (token, choice) pair when the
+def expert_order(idx: torch.Tensor, n_experts: int) -> Tuple[torch.Tensor, torch.Tensor, torch.Tensor]:
+    """idx int32 [T, top] -> (counts int32 [E]: pairs per expert; ends int32 [E]: their running sum; place int32 [T * top]: row of every (token, choice) pair when the
     pairs are put in the order of their experts, pairs of one expert in their own order; -1 for a pair whose number is n_experts
     or more, which has no row)."""
     _need_cuda(idx)
     assert idx.dtype == torch.int32 and idx.is_contiguous()
     counts = torch.empty(n_experts, dtype=torch.int32, device=idx.device)
+    ends = torch.empty(n_experts, dtype=torch.int32, device=idx.device)
     place = torch.empty(idx.numel(), dtype=torch.int32, device=idx.device)
-    _check(_gated_lib().msgl_expert_order(_ptr(idx), idx.numel(), n_experts, _ptr(counts), _ptr(place), _stream()), "expert_order")
+    _check(_gated_lib().msgl_expert_order(_ptr(idx), idx.numel(), n_experts, _ptr(counts), _ptr(place), _ptr(ends), _stream()), "expert_order")
     global LAUNCHES
     LAUNCHES += 1
-    return counts, place
+    return counts, ends, place
 
 
 def expert_gather(h: torch.Tensor, place: torch.Tensor, top: int) -> torch.Tensor:

@@ -75,11 +75,10 @@ class RoutedExperts(FeedForward):
         T = x.shape[0]
         if ctx.uniform_decode or T * self.top <= ops.EXPERTS_FEW_PAIRS:
             return ops.experts_few(x, self.gate_up, self.down, idx, wts, self.out_scale)
-        counts, place = ops.expert_order(idx, self.n_exp)
+        counts, ends, place = ops.expert_order(idx, self.n_exp)
         rows = ops.expert_gather(x, place, self.top)
         if x.dtype == torch.bfloat16 and self.H % 8 == 0 and self.F % 8 == 0 and hasattr(torch, "_grouped_mm"):
             # the library's grouped product takes the experts' row ranges from the device: two launches, nothing read on the host
-            ends = torch.cumsum(counts, 0, dtype=torch.int32)
             a = ops.swiglu(torch._grouped_mm(rows, self.gate_up.view(self.n_exp, 2 * self.F, self.H).transpose(-2, -1), offs=ends))
             y = torch._grouped_mm(a, self.down.transpose(-2, -1), offs=ends)
             return ops.expert_combine(y, place, wts, self.out_scale)
@@ -165,10 +164,9 @@ class SoftmaxExperts(FeedForward):
         T = x.shape[0]
         if ctx.uniform_decode or T * self.top <= ops.EXPERTS_FEW_PAIRS:
             return ops.experts_few(x, self.gate_up, self.down, idx, wts, limit=self.limit, extra=shared, extra_gate=sgate)
-        counts, place = ops.expert_order(idx, self.n_exp)
+        counts, ends, place = ops.expert_order(idx, self.n_exp)
         rows = ops.expert_gather(x, place, self.top)
         if x.dtype == torch.bfloat16 and self.H % 8 == 0 and self.F % 8 == 0 and hasattr(torch, "_grouped_mm"):
-            ends = torch.cumsum(counts, 0, dtype=torch.int32)
             gu = torch._grouped_mm(rows, self.gate_up.view(self.n_exp, 2 * self.F, self.H).transpose(-2, -1), offs=ends)
             y = torch._grouped_mm(ops.clamped_glu(gu, self.limit), self.down.transpose(-2, -1), offs=ends)
             return ops.expert_combine(y, place, wts, extra=shared, extra_gate=sgate)
@@ -268,10 +266,10 @@ class PlainExperts(FeedForward):
         T = x.shape[0]
         if ctx.uniform_decode or T * self.top <= ops.EXPERTS_FEW_PAIRS:
             return ops.plain_experts_few(x, self.up, self.down, idx, wts, self.act, extra=shared)
-        counts, place = ops.expert_order(idx, self.n_exp)
+        counts, ends, place = ops.expert_order(idx, self.n_exp)
         rows = ops.expert_gather(x, place, self.top)
         if x.dtype == torch.bfloat16 and self.H % 8 == 0 and self.F % 8 == 0 and hasattr(torch, "_grouped_mm"):
-            ends = torch.cumsum(counts, 0, dtype=torch.int32)          # rows behind the last end belong to nobody and are not read
+            # rows behind the last end belong to nobody and are not read
             u = torch._grouped_mm(rows, self.up.transpose(-2, -1), offs=ends)
             y = torch._grouped_mm(ops.unary_act(u, self.act, out=u), self.down.transpose(-2, -1), offs=ends)
             return ops.expert_combine_self(y, place, wts, x, extra=shared)

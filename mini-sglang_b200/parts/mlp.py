@@ -93,12 +93,8 @@ class GatedMLP(FeedForward, Projected):
         ops.gated_act(proj[:, :self.I], proj[:, self.I:2 * self.I], act, self.act)
 
     def forward(self, x, ctx):
-        if self.act == ops.ACT_SILU and not self.bias:        # product and activation in one kernel where the engine has it (few rows; many rows in bfloat16)
-            return ops.linear(ops.linear_swiglu(x, self.gate_up), self.down)
-        gu = ops.linear(x, self.gate_up, self.gate_up_b)
-        a = torch.empty((x.shape[0], self.I), dtype=x.dtype, device=x.device)
-        ops.gated_act(gu[:, :self.I], gu[:, self.I:], a, self.act)
-        return ops.linear(a, self.down, self.down_b)
+        # product and activation in one kernel where the engine has it (few rows; many rows in bfloat16)
+        return ops.linear(ops.linear_glu(x, self.gate_up, self.gate_up_b, self.act), self.down, self.down_b)
 
 
 UNARY_ACTIVATIONS = {"silu": ops.ACT_SILU, "gelu_tanh": ops.ACT_GELU_TANH, "relu2": ops.ACT_RELU2, "relu": ops.ACT_RELU}

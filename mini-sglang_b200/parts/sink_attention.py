@@ -1,5 +1,6 @@
 from __future__ import annotations
 
+import math
 from typing import Dict
 
 import torch
@@ -7,6 +8,7 @@ import torch
 from .. import ops
 from ..cache.manager import PagedKVNeed
 from ..weights.loader import TensorDecl
+from .attention import paged_attend
 from .base import Mixer, register_mixer
 from .context import KVCacheView, StepContext
 
@@ -70,7 +72,10 @@ class SinkAttention(Mixer):
         names.update(s.get("names") or {})
         self.names = {k: self.name(v) for k, v in names.items()}
         self.Cq, self.Ck, self.Cv = self.n_q * self.d, self.n_kv * self.d, self.n_kv * self.dv
-        self.w_in = self.b_in = self.w_out = self.sink = self.q_norm = self.k_norm = None
+        # equal head sizes that the engine's paged attention kernels take in bfloat16, and no cap on the scores: those kernels
+        # (tcgen05 for prompts at head size 128, kv splits in decode steps); else the ones that take any pair of head sizes
+        self.paged = self.d == self.dv and not self.softcap and ops.mma_supported(self.d, env.dtype)
+        self.w_in = self.b_in = self.w_out = self.sink = self.sink_log2 = self.q_norm = self.k_norm = None
         self.lam = 0.0
 
     def tensors(self) -> Dict[str, TensorDecl]:
@@ -106,12 +111,15 @@ class SinkAttention(Mixer):
             self.sink = f(n["sink"]).float().contiguous()
         else:
             self.sink = torch.full((self.n_q,), self.fixed_sink, dtype=torch.float32, device=self.w_in.device)
+        self.sink_log2 = (self.sink * math.log2(math.e)).contiguous()
         if self.qk_norm:
             self.q_norm, self.k_norm = f(n["q_norm"]).float().contiguous(), f(n["k_norm"]).float().contiguous()
         if self.value_mix == "blend":
             self.lam = float(f(n["mix"]).float().item())
 
     def cache_need(self) -> PagedKVNeed:
+        if self.paged:
+            return PagedKVNeed(self.n_kv, self.d, self.window, q_heads=self.n_q)
         return PagedKVNeed(self.n_kv, self.d, self.window, q_heads=self.n_q, library="mixers_delta", even_cut=False,
                            v_head_dim=self.dv)
 
@@ -132,6 +140,11 @@ class SinkAttention(Mixer):
                               v_cache=cache.v if writes_cache else None, page_size=cache.page_size, q_norm=self.q_norm,
                               k_norm=self.k_norm, v_unit=self.value_norm, eps=self.eps)
         gate = proj[:, Cq + Ck + Cv:Cq + Ck + Cv + self.n_q * self.dv] if self.gate else None
+        if self.paged:
+            o = torch.empty_like(q)
+            paged_attend(q, o, ctx, cache, n_q=self.n_q, n_kv=self.n_kv, d=self.d, window=int(self.window or 0), scale=self.scale,
+                         use_mma=True, null_log2=self.sink_log2, gate=gate)
+            return ops.linear(o.view(ctx.T, self.n_q * self.dv), self.w_out)
         out = torch.empty((ctx.T, self.n_q * self.dv), dtype=x.dtype, device=x.device)
         ops.sink_attention(q, out, cache.k, cache.v, q_start=ctx.q_start, kv_len=ctx.kv_len, block_table=cache.group.block_table,
                            n_kv=self.n_kv, page_size=cache.page_size, scale=self.scale, softcap=self.softcap, window=self.window or 0,

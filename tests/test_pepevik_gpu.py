@@ -566,7 +566,8 @@ def test_experts_both_ways(dtype, T):
     want = (0.6 * want).float()
     few = ops.experts_few(h.cuda(), gu.cuda(), dn.cuda(), idx.cuda(), wts.cuda(), 0.6).cpu()
     torch.testing.assert_close(few, want, **tol_of(dtype, 2e-5, 2e-2))
-    counts, place = ops.expert_order(idx.cuda(), E)
+    counts, ends, place = ops.expert_order(idx.cuda(), E)
+    assert torch.equal(ends.cpu(), counts.cpu().cumsum(0).int())
     assert counts.cpu().tolist() == [int((idx == e).sum()) for e in range(E)]
     flat = idx.reshape(-1)
     order = sorted(range(T * top), key=lambda i: (int(flat[i]), i))
