@@ -124,7 +124,7 @@ def _moe(cfg: PokatarConfig, f: Dict[str, Any], where: str) -> PartSpec:
         "activation": "relu2", "num_experts": int(_need(r, "experts", where + ".router")), "identity": int(r.get("identity") or 0),
         "top": int(_need(r, "top", where + ".router")), "groups": count, "keep_groups": int(g.get("keep") or count),
         "score": "softmax", "group_score": "max", "renormalize": False,
-        "shared_size": int(_need(sh, "ff", where + ".shared")) if sh else 0,
+        "shared_size": int(_need(sh, "ff", where + ".shared")) if sh is not None else 0,
         "names": {"router": "router", "correction": "correction", "expert": "e{e}", "up": "up", "down": "down", "shared": "shared"}})
 
 

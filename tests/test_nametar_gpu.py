@@ -695,8 +695,8 @@ def test_models_of_one_kind_of_layer(kinds, dtype):
 
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 def test_two_geometries_in_one_cache_group(dtype):
-    """Two latent attentions over all keys with different head counts and row sizes share a cache group (one block table, one
-    plan of kv splits made from the first one's geometry).  A long context, then portions of a few tokens and single tokens:
+    """Two latent attentions over all keys with different head counts and row sizes share a cache group (one block table, kv
+    splits of their own).  A long context, then portions of a few tokens and single tokens:
     short runs take the decode kernel with the keys cut into pieces, and which runs are short differs between the two."""
     import tiny_nametar as tn
     from mini_sglang_b200.engine.step import ModelRunner
