@@ -2,6 +2,7 @@ from __future__ import annotations
 
 from typing import Optional
 
+import numpy as np
 import torch
 
 from .base import PositionEncoding, register_position_encoding
@@ -29,13 +30,13 @@ class RotaryNeox(PositionEncoding):
 
     def rotary_table(self) -> torch.Tensor:
         if self._table is None:
-            # built on the host in float32, operation by operation as the reference does, so the
-            # table does not depend on the device's pow/sin/cos roundings; then moved to the device
+            # the angles on the host in float32, operation by operation as the reference makes them, so the table does not
+            # depend on the device's roundings; then moved to the device
             idx = torch.arange(0, self.rotary_dim, 2, dtype=torch.float32)
             inv_freq = 1.0 / (self.theta ** (idx / self.rotary_dim))
             t = torch.arange(self.max_positions, dtype=torch.float32)
             freqs = t[:, None] * inv_freq[None, :]
-            self._table = torch.cat((freqs.cos(), freqs.sin()), dim=-1).contiguous().to(self.env.device)
+            self._table = cos_sin_table(freqs).to(self.env.device)
         return self._table
 
     def fused_decode_fields(self):
@@ -81,7 +82,7 @@ class RotaryYarn(PositionEncoding):
         if self._table is None:
             t = torch.arange(self.max_positions, dtype=torch.float32)
             ang = t[:, None] * self._freq_host[None, :]
-            self._table = (torch.cat((ang.cos(), ang.sin()), dim=-1) * self.magnitude).contiguous().to(self.env.device)
+            self._table = cos_sin_table(ang, self.magnitude).to(self.env.device)
         return self._table
 
     def step_angles(self, ctx) -> torch.Tensor:
@@ -89,6 +90,15 @@ class RotaryYarn(PositionEncoding):
         layers that share this encoding: position times frequency and the circular functions in double precision, so that
         the angle of a far position is as exact as that of a near one and no table bounds the context."""
         return step_angles_of(self, ctx)
+
+
+def cos_sin_table(angles: torch.Tensor, magnitude: float = 1.0) -> torch.Tensor:
+    """host angles [P, n] -> float32 [P, 2n] = magnitude * (cos | sin), made by numpy in double precision on one thread.  (torch's
+    own cos and sin hand a large tensor out in pieces to threads of a vector-math library; a piece of a process's first such
+    call was now and then some 1e-4 off.)"""
+    a = angles.to(torch.float64).numpy()
+    table = np.concatenate((np.cos(a), np.sin(a)), axis=-1) * magnitude
+    return torch.from_numpy(table.astype(np.float32))
 
 
 def step_angles_of(enc, ctx) -> torch.Tensor:
@@ -132,7 +142,7 @@ class RotarySteppedWavelengths(PositionEncoding):
         if self._table is None:
             t = torch.arange(self.max_positions, dtype=torch.float64)
             ang = t[:, None] * self._freq_host64[None, :]
-            self._table = torch.cat((ang.cos(), ang.sin()), dim=-1).to(torch.float32).contiguous().to(self.env.device)
+            self._table = cos_sin_table(ang).to(self.env.device)
         return self._table
 
     def step_angles(self, ctx) -> torch.Tensor:
