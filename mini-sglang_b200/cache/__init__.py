@@ -1,5 +1,5 @@
-from .manager import CacheManager, KVGroup, OutOfSlots, PagedKVNeed, StateNeed
+from .manager import CacheManager, KVGroup, OutOfSlots, PagedKVNeed, StateNeed, keys_seen
 from .pages import OutOfPages, PagePool
 from .radix import PrefixTree
 
-__all__ = ["CacheManager", "KVGroup", "OutOfSlots", "PagedKVNeed", "StateNeed", "OutOfPages", "PagePool", "PrefixTree"]
+__all__ = ["CacheManager", "KVGroup", "OutOfSlots", "PagedKVNeed", "StateNeed", "keys_seen", "OutOfPages", "PagePool", "PrefixTree"]

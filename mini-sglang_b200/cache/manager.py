@@ -5,10 +5,12 @@ What a mixer keeps between steps is declared as a *need*:
   PagedKVNeed(n_kv_heads, head_dim, window)  keys and values of every token (window=None) or of
                                              the last `window` tokens only; with `keep_first` = F also
                                              of the first F tokens, whose pages a window never gives back
+  PagedKVNeed(..., chunk=C)                  keys and values of the last, unfinished chunk of C tokens only, chunks
+                                             counted from the start of the request
   StateNeed(shape, dtype)                    an array of fixed size per request
 A mixer that keeps several things (keys and values beside a recurrent state, say) declares a tuple of
 needs; the caches of run `c` are then named (c, 0), (c, 1), ... .
-Caches whose needs differ in kind (all keys / a window of them / a window and the first tokens) form groups with pages of their
+Caches whose needs differ in kind (all keys / a window of them / a window and the first tokens / a chunk) form groups with pages of their
 own: a page id of a group indexes the K and V arrays of every cache in that group, and each
 group has its own pool and its own block table per request.  A request owns one slot (a row in
 every block table and in every state array) from `open` to `close`.
@@ -20,7 +22,7 @@ every block table and in every state array) from `open` to `close`.
                                       are given back
     mgr.close(slot)                   everything the request holds is given back
 
-Pages are given back when a request ends or a window has passed them, and are handed out again
+Pages are given back when a request ends or a window or chunk has passed them, and are handed out again
 first-in first-out.  The reference's counterparts: mini_sglang/mem_cache/token2kv.py (pool and
 allocator, one group), mini_sglang/mem_cache/req2token.py (request slots and block table).
 """
@@ -48,6 +50,7 @@ class PagedKVNeed:
     even_cut: bool = True            # whether a decode step may deal this cache's keys out evenly over the blocks
     shared_kv: bool = False          # the values are read out of the key rows: one array is kept, not two
     v_head_dim: Optional[int] = None # size of a value row where it differs from a key row's (None: head_dim)
+    chunk: Optional[int] = None      # without a window: a query sees the keys of its own chunk of this many positions only
 
 
 @dataclasses.dataclass(frozen=True)
@@ -60,6 +63,13 @@ class OutOfSlots(RuntimeError):
     pass
 
 
+def keys_seen(n: int, window: Optional[int], chunk: Optional[int]) -> int:
+    """How many keys the newest of a request's n tokens sees."""
+    if window:
+        return min(n, window)
+    return (n - 1) % chunk + 1 if chunk and n > 0 else n
+
+
 def cache_id_key(cid) -> Tuple[int, int]:
     """Order of cache ids: a run's id `c`, or (c, k) for the k-th need of a mixer that declares several."""
     return (cid[0], cid[1]) if isinstance(cid, tuple) else (cid, -1)
@@ -69,8 +79,10 @@ class KVGroup:
     """Caches with the same kind of need: one pool, one block table per request."""
 
     def __init__(self, window: Optional[int], num_pages: int, max_reqs: int, max_pages_per_req: int, keep_first: int = 0,
-                 page_size: int = 1):
+                 page_size: int = 1, chunk: Optional[int] = None):
         self.window = window
+        self.chunk = chunk
+        self.span = window if window is not None else chunk        # the most keys a query sees (None: all)
         self.keep_first = keep_first if window is not None else 0
         self.keep_pages = -(-self.keep_first // page_size)        # leading pages that a window never gives back
         self.pool = PagePool(num_pages)
@@ -79,6 +91,12 @@ class KVGroup:
         self.first_live = np.zeros(max_reqs + 1, dtype=np.int64)   # entries below this were given back
         self.cache_ids: List[int] = []
         self.dirty: set = set()        # slots whose table row changed since a device copy of the table was last brought up to date
+
+    def first_seen(self, pos: int) -> int:
+        """The first position that a query at `pos` sees (kept first tokens apart)."""
+        if self.window is not None:
+            return max(0, pos - self.window + 1)
+        return pos - pos % self.chunk if self.chunk is not None else 0
 
 
 class CacheManager:
@@ -93,7 +111,7 @@ class CacheManager:
         self.needs = dict(needs)
         self.groups: List[KVGroup] = []
         self.group_of_cache: Dict[int, int] = {}
-        by_window: Dict[Tuple[Optional[int], int], int] = {}
+        by_window: Dict[Tuple[Optional[int], int, Optional[int]], int] = {}
         for cid in sorted(needs, key=cache_id_key):
             need = needs[cid]
             if isinstance(need, PagedKVNeed):
@@ -101,14 +119,16 @@ class CacheManager:
                     raise ValueError("a window must be at least 1 token")
                 if need.keep_first < 0:
                     raise ValueError("keep_first must not be negative")
-                kind = (need.window, need.keep_first if need.window is not None else 0)
+                if need.chunk is not None and (need.chunk < 1 or need.window is not None):
+                    raise ValueError("a chunk must be at least 1 token and excludes a window")
+                kind = (need.window, need.keep_first if need.window is not None else 0, need.chunk)
                 if kind not in by_window:
                     n = num_pages
-                    if need.window is not None:
-                        per_req = -(-(need.window + max(max_step_tokens, 1)) // page_size) + 2 + -(-kind[1] // page_size)
+                    if need.window is not None or need.chunk is not None:
+                        per_req = -(-((need.window or need.chunk) + max(max_step_tokens, 1)) // page_size) + 2 + -(-kind[1] // page_size)
                         n = min(num_pages, max_reqs * per_req)
                     by_window[kind] = len(self.groups)
-                    self.groups.append(KVGroup(need.window, n, max_reqs, self.max_pages_per_req, kind[1], page_size))
+                    self.groups.append(KVGroup(need.window, n, max_reqs, self.max_pages_per_req, kind[1], page_size, need.chunk))
                 g = by_window[kind]
                 self.groups[g].cache_ids.append(cid)
                 self.group_of_cache[cid] = g
@@ -160,7 +180,7 @@ class CacheManager:
         for g, n in zip(self.groups, need):
             if n > g.pool.available:
                 raise OutOfPages(f"{n} pages wanted, {g.pool.available} free of {g.pool.num_pages}"
-                                 + (f" (window {g.window})" if g.window else ""))
+                                 + (f" (window {g.window})" if g.window else f" (chunk {g.chunk})" if g.chunk else ""))
         for g, n in zip(self.groups, need):
             if n:
                 k = int(g.n_pages[slot])
@@ -173,7 +193,7 @@ class CacheManager:
         """Start a fresh request on pages that a prefix tree owns (group 0, whole pages)."""
         if self.length[slot] or self.reserved[slot]:
             raise ValueError("a prefix can only be adopted by a request that holds nothing")
-        if len(self.groups) != 1 or self.groups[0].window is not None or self.state_ids:
+        if len(self.groups) != 1 or self.groups[0].span is not None or self.state_ids:
             raise ValueError("prefix reuse needs a single group that keeps all keys and no per-request state")
         g = self.groups[0]
         n = len(pages)
@@ -214,9 +234,9 @@ class CacheManager:
         self.length[slot] = new_len
         P = self.page_size
         for g in self.groups:
-            if g.window is None:
+            if g.span is None:
                 continue
-            dead = max(0, (new_len - g.window + 1) // P)       # pages wholly before the next query's window
+            dead = g.first_seen(new_len) // P       # pages wholly before what the next query sees
             dead = min(dead, int(g.n_pages[slot]))
             first = max(int(g.first_live[slot]), g.keep_pages)   # the pages of the kept first tokens stay
             if dead > first:

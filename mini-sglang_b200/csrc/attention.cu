@@ -4,7 +4,8 @@
 // Every request r of the step brings q_len[r] = q_start[r+1] - q_start[r] new tokens whose keys
 // and values are already in the cache; kv_len[r] counts them too.  The query at offset j of
 // request r sits at position kv_len[r] - q_len[r] + j and sees keys 0..position (or the last
-// `window` of them).  Query head h reads kv head h / (n_q / n_kv).
+// `window` of them, or those of its own chunk of `chunk_keys` positions counted from the start of the sequence).  Query
+// head h reads kv head h / (n_q / n_kv).
 //
 // Cache layout (one K and one V array per layer): [page][kv head][slot in page][d]; the key at
 // position i of request r lives in page block_table[r][i / P], slot i % P.
@@ -70,6 +71,8 @@ struct AttnParams {
     float scale;
     int qlen_min, qlen_max;   // this launch takes the requests with qlen_min <= q_len <= qlen_max
     int uniform_decode;       // every request has exactly one token: tile index == request index
+    // > 0 (without a window): keys are seen within chunks of the sequence only, key / chunk_keys == position / chunk_keys
+    int chunk_keys = 0;
     // with a window: the first keep_first keys of a request stay visible whatever the window (bfloat16 mma kernels)
     int keep_first = 0;
     // null, or [n_q][bias_len] float32 in log2 units: added to the scaled score by distance min(position - key, bias_len - 1)
@@ -181,6 +184,12 @@ __device__ __forceinline__ void block_place(const AttnParams& p, int& tile_idx, 
     }
 }
 
+// The first key that the query at position `pos` sees (kept first tokens under a window lie before it).
+__device__ __forceinline__ int first_key(const AttnParams& p, int pos) {
+    if (p.window > 0) return max(0, pos - p.window + 1);
+    return p.chunk_keys > 0 ? pos - pos % p.chunk_keys : 0;
+}
+
 // Kept first tokens that lie before the first key tile of the window: keys [0, sink_keys).  Split 0 reads them ahead of its
 // share of the window's tiles; they are no part of key_tile_range.
 __device__ __forceinline__ int sink_keys(const AttnParams& p, int p_min, int KT, int split) {
@@ -188,17 +197,14 @@ __device__ __forceinline__ int sink_keys(const AttnParams& p, int p_min, int KT,
     const int k_lo = max(0, p_min - p.window + 1);
     return min(p.keep_first, (k_lo / KT) * KT);
 }
-// whether the cache row of `key` may be read by a block whose queries sit at p_min..p_max: rows behind the window may lie
-// on pages that were given back
+// whether the cache row of `key` may be read by a block whose queries sit at p_min..p_max: rows behind the window or before the
+// chunk may lie on pages that were given back
 __device__ __forceinline__ bool key_row_live(const AttnParams& p, int key, int p_min, int p_max) {
     if (key > p_max) return false;
-    if (p.window <= 0) return true;
-    return key > p_min - p.window || key < p.keep_first;
+    return key >= first_key(p, p_min) || key < p.keep_first;
 }
 __device__ __forceinline__ bool key_visible(const AttnParams& p, int key, int pos) {
-    bool ok = key <= pos;
-    if (p.window > 0) ok = ok && (key > pos - p.window || key < p.keep_first);
-    return ok;
+    return key <= pos && (key >= first_key(p, pos) || key < p.keep_first);
 }
 
 // Which key tiles a block walks: the tiles that hold keys [k_lo, p_max], cut into ns splits.
@@ -206,8 +212,7 @@ __device__ __forceinline__ void key_tile_range(const AttnParams& p, const TileIn
                                                int& p_min, int& p_max, int& kt_begin, int& kt_end) {
     p_min = ti.kv_len - ti.q_len + ti.t0;
     p_max = p_min + ti.n_tok - 1;
-    int k_lo = 0;
-    if (p.window > 0) k_lo = max(0, p_min - p.window + 1);
+    const int k_lo = first_key(p, p_min);
     const int first = k_lo / KT, last = p_max / KT;
     const int n_t = last - first + 1;
     const int per = (n_t + ns - 1) / ns;
@@ -327,13 +332,14 @@ __global__ void __launch_bounds__(MMA_THREADS) attn_mma_kernel(const AttnParams 
     const int ld_row = tid >> 1, ld_half = tid & 1;
     // iterations: first the tiles of the kept first tokens before the window (split 0 only), then the split's own tiles
     const int sink_hi = EXT ? sink_keys(p, p_min, MMA_KT, split) : 0;
+    const int k_first = first_key(p, p_min), k_first_max = first_key(p, p_max);      // the first key that any / every row sees
     const int n_sink_t = (sink_hi + MMA_KT - 1) / MMA_KT;
     const int n_tiles = n_sink_t + (kt_end - kt_begin);
     auto tile_of = [&](int it) -> int { return it < n_sink_t ? it : kt_begin + (it - n_sink_t); };
     auto tile_page = [&](int it) -> int {
         if (it >= n_tiles) return -1;
         const int key = tile_of(it) * MMA_KT + ld_row;
-        const bool live = !EXT ? key <= p_max : (it < n_sink_t ? key < sink_hi : key_row_live(p, key, p_min, p_max));
+        const bool live = !EXT ? key <= p_max && key >= k_first : (it < n_sink_t ? key < sink_hi : key_row_live(p, key, p_min, p_max));
         return live ? bt[page_index(p, key)] : -1;
     };
     constexpr unsigned STAGE_BYTES = 2u * MMA_KT * LDS * 2u, TILE_BYTES = MMA_KT * LDS * 2u;
@@ -359,6 +365,7 @@ __global__ void __launch_bounds__(MMA_THREADS) attn_mma_kernel(const AttnParams 
     const int key_base = 0;
     const int r_lo = row_base + (lane >> 2), r_hi = r_lo + 8;
     const int pos_lo = p_min + r_lo / Gc, pos_hi = p_min + r_hi / Gc;   // position of each row's query
+    const int first_lo = first_key(p, pos_lo), first_hi = first_key(p, pos_hi);
     const float sc = p.scale * 1.4426950408889634f;                     // scores in log2 units
     // per-lane parts of the ldmatrix addresses (bytes)
     const unsigned q_a = q_s + (unsigned)((row_base + (lane & 15)) * LDS + (lane >> 4) * 8) * 2u;
@@ -431,7 +438,7 @@ __global__ void __launch_bounds__(MMA_THREADS) attn_mma_kernel(const AttnParams 
         // ---- scale, mask, online softmax
         const int key0 = kt * MMA_KT + key_base;
         const bool need_mask = (kt * MMA_KT + MMA_KT - 1 > p_min) || it < n_sink_t ||
-                               (p.window > 0 && kt * MMA_KT <= p_max - p.window);
+                               kt * MMA_KT < k_first_max;
         // raw scores stay unscaled: the scale is folded into the exponent, 2^(s * sc - m)
         float mx_lo = -INFINITY, mx_hi = -INFINITY;
 #pragma unroll
@@ -446,8 +453,7 @@ __global__ void __launch_bounds__(MMA_THREADS) attn_mma_kernel(const AttnParams 
                     if (EXT) {
                         ok = !need_mask || (key_visible(p, key, pos) && (it >= n_sink_t || key < sink_hi));
                     } else {
-                        ok = key <= pos;
-                        if (p.window > 0) ok = ok && (key > pos - p.window);
+                        ok = key <= pos && key >= ((e < 2) ? first_lo : first_hi);
                     }
                     if (!ok) v = -INFINITY;
                     else if (EXT && p.bias)
@@ -606,6 +612,7 @@ __global__ void __launch_bounds__(NW * 32) attn_decode_kernel(const AttnParams p
     }
     cp_async_commit();
 
+    const int k_first = first_key(p, p_min), k_first_max = first_key(p, p_max);      // the first key that any / every row sees
     // this warp's units: u_begin + warp, + NW, ...
     const int n_my = (u_end - u_begin > warp) ? (u_end - u_begin - warp + NW - 1) / NW : 0;
     __nv_bfloat16* my_ring = ring + (size_t)warp * ST * 2 * DEC_WT * LDS;
@@ -615,7 +622,7 @@ __global__ void __launch_bounds__(NW * 32) attn_decode_kernel(const AttnParams p
     // dependent global load, so it is issued one iteration before the copy that needs it.
     auto unit_page = [&](int i) -> int {
         const int key = (u_begin + warp + i * NW) * DEC_WT + l_key;
-        return (i < n_my && key <= p_max) ? bt[page_index(p, key)] : -1;
+        return (i < n_my && key <= p_max && key >= k_first) ? bt[page_index(p, key)] : -1;
     };
     auto load_unit = [&](int i, int pg) {      // unit i of this warp into stage i % ST
         __nv_bfloat16* Ks = my_ring + (size_t)(i % ST) * 2 * DEC_WT * LDS;
@@ -679,7 +686,7 @@ __global__ void __launch_bounds__(NW * 32) attn_decode_kernel(const AttnParams p
             mma_bf16_16816(s[0], qf[kk], b[0], b[1]);
             mma_bf16_16816(s[1], qf[kk], b[2], b[3]);
         }
-        const bool need_mask = (key0 + DEC_WT - 1 > p_min) || (p.window > 0 && key0 <= p_max - p.window);
+        const bool need_mask = (key0 + DEC_WT - 1 > p_min) || key0 < k_first_max;
         float mx_lo = -INFINITY, mx_hi = -INFINITY;
 #pragma unroll
         for (int nb = 0; nb < 2; ++nb) {
@@ -689,9 +696,7 @@ __global__ void __launch_bounds__(NW * 32) attn_decode_kernel(const AttnParams p
                 if (need_mask) {
                     const int key = key0 + nb * 8 + (lane & 3) * 2 + (e & 1);
                     const int pos = (e < 2) ? pos_lo : pos_hi;
-                    bool ok = key <= pos;
-                    if (p.window > 0) ok = ok && (key > pos - p.window);
-                    if (!ok) v = -INFINITY;
+                    if (key > pos || key < first_key(p, pos)) v = -INFINITY;
                 }
                 s[nb][e] = v;
                 if (e < 2) mx_lo = fmaxf(mx_lo, v); else mx_hi = fmaxf(mx_hi, v);
@@ -851,13 +856,14 @@ __device__ __forceinline__ void decode_t_run(const AttnParams& p, const TileInfo
 #pragma unroll
         for (int e = 0; e < 2; ++e) pos_c[nb][e] = p_min + (nb * 8 + 2 * t + e) / Gc;
 
+    const int k_first = first_key(p, p_min);      // the first key that any column sees
     // the units of the kept first tokens before the window (keys [0, sink_hi)) come first, then units [u_begin, u_end)
     const int n_su = EXT ? (sink_hi + DEC_WT - 1) / DEC_WT : 0;
     const int n_units = n_su + (u_end - u_begin);
     const int n_my = (n_units > warp) ? (n_units - warp + NW - 1) / NW : 0;
     auto unit_of = [&](int i) -> int { const int lu = warp + i * NW; return lu < n_su ? lu : u_begin + (lu - n_su); };
     auto row_live = [&](int i, int key) -> bool {
-        if (!EXT) return key <= p_max;
+        if (!EXT) return key <= p_max && key >= k_first;
         return (warp + i * NW < n_su) ? key < sink_hi : key_row_live(p, key, p_min, p_max);
     };
     // bias tables of the columns this lane sees
@@ -999,7 +1005,8 @@ __device__ __forceinline__ void decode_t_run(const AttnParams& p, const TileInfo
         // ---- scale, mask, online softmax per column
         const int key0 = unit_of(i) * DEC_WT;
         const bool in_sink = EXT && warp + i * NW < n_su;
-        const bool need_mask = in_sink || (key0 + DEC_WT - 1 > p_min) || (p.window > 0 && key0 <= p_max - p.window);
+        const bool need_mask = in_sink || (key0 + DEC_WT - 1 > p_min) || key0 < k_first ||
+                               (p_min != p_max && (p.window > 0 || p.chunk_keys > 0));
         unsigned pb0[NBH], pb1[NBH];
         float v[NBH][4];
         bool behind = false;              // a score lies further above its column's reference than DEC_LAZY allows
@@ -1015,8 +1022,7 @@ __device__ __forceinline__ void decode_t_run(const AttnParams& p, const TileInfo
                     if (EXT) {
                         ok = !need_mask || (key_visible(p, key, pos) && (!in_sink || key < sink_hi));
                     } else {
-                        ok = key <= pos;
-                        if (p.window > 0) ok = ok && (key > pos - p.window);
+                        ok = key <= pos && key >= first_key(p, pos);
                     }
                     if (!ok) v[nb][e] = -INFINITY;
                     else if (EXT && p.bias) v[nb][e] += bias_c[nb][e & 1][min(max(pos - key, 0), p.bias_len - 1)];
@@ -1217,8 +1223,7 @@ __global__ void __launch_bounds__(NW * 32, (NBH == 1 && D <= 128) ? 4 : 2) attn_
         TileInfo ti;
         ti.req = r; ti.t0 = 0; ti.n_tok = 1; ti.q_len = 1; ti.kv_len = p.kv_len[r]; ti.q_base = p.q_start[r];
         const int pos = ti.kv_len - 1;
-        const int k_lo = p.window > 0 ? max(0, pos - p.window + 1) : 0;
-        const int first_unit = k_lo / DEC_WT;
+        const int first_unit = first_key(p, pos) / DEC_WT;
         const int ns = p.nsplit ? min(max(p.nsplit[r], 1), p.max_split) : 1;
         const int piece = j - req_first_blk[r];
         const bool last = seg_hi >= hi;
@@ -1271,6 +1276,7 @@ __global__ void __launch_bounds__(SIMT_THREADS) attn_simt_kernel(const AttnParam
     if (split >= ns) return;
     int p_min, p_max, kt_begin, kt_end;
     key_tile_range(p, ti, SIMT_KT, split, ns, p_min, p_max, kt_begin, kt_end);
+    const int k_first = first_key(p, p_min);
 
     const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
     const T* qg = reinterpret_cast<const T*>(p.q);
@@ -1297,7 +1303,7 @@ __global__ void __launch_bounds__(SIMT_THREADS) attn_simt_kernel(const AttnParam
             const int kl = idx / D, c = idx - kl * D;
             const int key = key0 + kl;
             float kv = 0.f, vv = 0.f;
-            if (key <= p_max) {
+            if (key <= p_max && key >= k_first) {
                 const int pg = bt[page_index(p, key)];
                 const int sl = page_slot(p, key);
                 const size_t off = (((size_t)pg * p.n_kv + kvh) * p.page_size + sl) * D + c;
@@ -1318,7 +1324,7 @@ __global__ void __launch_bounds__(SIMT_THREADS) attn_simt_kernel(const AttnParam
             const int key = key0 + kl;
             const int pos = p_min + r / Gc;
             bool ok = key <= pos && (r / Gc) < ti.n_tok;
-            if (p.window > 0) ok = ok && (key > pos - p.window);
+            ok = ok && key >= first_key(p, pos);
             Ss[idx] = ok ? acc * sc : -INFINITY;
         }
         __syncthreads();
@@ -1459,17 +1465,17 @@ static int attention_launch(const void* q, void* out, const void* k_cache, const
                             int window, int max_split, float scale, int qlen_min, int qlen_max, int uniform_decode,
                             int variant, int grid_x, int dtype, const int* order, const int* even, int even_nb,
                             int keep_first, const float* bias, int bias_len, const float* null_log2, const void* gate,
-                            long long gate_stride, cudaStream_t stream);
+                            long long gate_stride, int chunk_keys, cudaStream_t stream);
 
 MSGL_API int msgl_attention(const void* q, void* out, const void* k_cache, const void* v_cache, const int* q_start,
                             const int* kv_len, const int* block_table, const int* nsplit, float* part_o,
                             float* part_ml, int B, int T_, int n_q, int n_kv, int d, int page_size, int bt_stride,
                             int window, int max_split, float scale, int qlen_min, int qlen_max, int uniform_decode,
                             int variant, int grid_x, int dtype, const int* order, const int* even, int even_nb,
-                            const float* null_log2, const void* gate, long long gate_stride, cudaStream_t stream) {
+                            const float* null_log2, const void* gate, long long gate_stride, int chunk_keys, cudaStream_t stream) {
     return attention_launch(q, out, k_cache, v_cache, q_start, kv_len, block_table, nsplit, part_o, part_ml, B, T_, n_q, n_kv, d,
                             page_size, bt_stride, window, max_split, scale, qlen_min, qlen_max, uniform_decode, variant, grid_x,
-                            dtype, order, even, even_nb, 0, nullptr, 0, null_log2, gate, gate_stride, stream);
+                            dtype, order, even, even_nb, 0, nullptr, 0, null_log2, gate, gate_stride, chunk_keys, stream);
 }
 
 // The same with a window that keeps the first `keep_first` keys of every request visible and with a bias by distance
@@ -1486,7 +1492,7 @@ MSGL_API int msgl_attention_window(const void* q, void* out, const void* k_cache
     if (!(variant == 1 || (variant == 2 && MSGL_HEAD_DIM % 32 == 0 && G <= 16))) return MSGL_ERR_SIZE;
     return attention_launch(q, out, k_cache, v_cache, q_start, kv_len, block_table, nsplit, part_o, part_ml, B, T_, n_q, n_kv, d,
                             page_size, bt_stride, window, max_split, scale, qlen_min, qlen_max, uniform_decode, variant, grid_x,
-                            dtype, order, nullptr, 0, keep_first, bias, bias_len, nullptr, nullptr, 0, stream);
+                            dtype, order, nullptr, 0, keep_first, bias, bias_len, nullptr, nullptr, 0, 0, stream);
 }
 
 static int attention_launch(const void* q, void* out, const void* k_cache, const void* v_cache, const int* q_start,
@@ -1495,7 +1501,8 @@ static int attention_launch(const void* q, void* out, const void* k_cache, const
                             int window, int max_split, float scale, int qlen_min, int qlen_max, int uniform_decode,
                             int variant, int grid_x, int dtype, const int* order, const int* even, int even_nb,
                             int keep_first, const float* bias, int bias_len, const float* null_log2, const void* gate,
-                            long long gate_stride, cudaStream_t stream) {
+                            long long gate_stride, int chunk_keys, cudaStream_t stream) {
+    if (chunk_keys < 0 || (chunk_keys > 0 && window > 0)) return MSGL_ERR_SIZE;
     if (gate != nullptr && dtype == MSGL_BF16 && ((gate_stride & 1) || ((uintptr_t)gate & 3))) return MSGL_ERR_ALIGN;
     if (grid_x <= 0 || B <= 0) return MSGL_OK;
     if (n_kv <= 0 || n_q % n_kv != 0 || d <= 0 || page_size <= 0 || max_split < 1) return MSGL_ERR_SIZE;
@@ -1505,7 +1512,7 @@ static int attention_launch(const void* q, void* out, const void* k_cache, const
     p.block_table = block_table; p.nsplit = nsplit; p.order = order; p.even = nullptr; p.even_nb = 0;
     p.part_o = part_o; p.part_ml = part_ml;
     p.B = B; p.T = T_; p.n_q = n_q; p.n_kv = n_kv; p.d = d; p.page_size = page_size; p.bt_stride = bt_stride;
-    p.window = window; p.max_split = max_split;
+    p.window = window; p.chunk_keys = chunk_keys; p.max_split = max_split;
     p.page_shift = -1;
     if ((page_size & (page_size - 1)) == 0) { int sh = 0; while ((1 << sh) < page_size) ++sh; p.page_shift = sh; } p.scale = scale; p.qlen_min = qlen_min; p.qlen_max = qlen_max;
     p.uniform_decode = uniform_decode;
@@ -1613,11 +1620,13 @@ MSGL_API int msgl_attention_tc(const void* q, void* out, const void* k_cache, co
                                const int* kv_len, const int* block_table, int B, int T_, int n_q, int n_kv, int d,
                                int page_size, int bt_stride, int window, float scale, int qlen_min, int qlen_max,
                                int grid_x, int cache_pages, int version, int* status, int keep_first, const float* bias,
-                               int bias_len, const float* null_log2, const void* gate, long long gate_stride, cudaStream_t stream) {
+                               int bias_len, const float* null_log2, const void* gate, long long gate_stride, int chunk_keys,
+                               cudaStream_t stream) {
 #if MSGL_HEAD_DIM == 128
     if (gate != nullptr && ((gate_stride & 7) || ((uintptr_t)gate & 15))) return MSGL_ERR_ALIGN;
     // kept first tokens under the window and a bias by distance ([n_q][bias_len] float32, log2 units): version 2 only
     const bool ext = (window > 0 && keep_first > 0) || bias != nullptr;
+    if (chunk_keys < 0 || (chunk_keys > 0 && window > 0)) return MSGL_ERR_SIZE;
     if (ext && (version != 2 || keep_first < 0 || (bias != nullptr && bias_len < 1))) return MSGL_ERR_SIZE;
     if (grid_x <= 0 || B <= 0) return MSGL_OK;
     if (d != 128 || n_kv <= 0 || n_q % n_kv != 0 || page_size <= 0 || grid_x > 65535) return MSGL_ERR_SIZE;
@@ -1627,7 +1636,7 @@ MSGL_API int msgl_attention_tc(const void* q, void* out, const void* k_cache, co
     p.block_table = block_table; p.nsplit = nullptr; p.order = nullptr; p.even = nullptr; p.even_nb = 0;
     p.part_o = nullptr; p.part_ml = nullptr;
     p.B = B; p.T = T_; p.n_q = n_q; p.n_kv = n_kv; p.d = d; p.page_size = page_size; p.bt_stride = bt_stride;
-    p.window = window; p.max_split = 1;
+    p.window = window; p.chunk_keys = chunk_keys; p.max_split = 1;
     p.page_shift = -1;
     if ((page_size & (page_size - 1)) == 0) { int sh = 0; while ((1 << sh) < page_size) ++sh; p.page_shift = sh; }
     p.scale = scale; p.qlen_min = qlen_min; p.qlen_max = qlen_max; p.uniform_decode = 0;

@@ -99,7 +99,7 @@ __global__ void __launch_bounds__(TC_THREADS, 2) attn_tc_kernel(const AttnParams
     // key tiles of TC_KT anchored at absolute positions
     const int p_min = ti.kv_len - ti.q_len + ti.t0;
     const int p_max = p_min + ti.n_tok - 1;
-    const int k_lo = p.window > 0 ? max(0, p_min - p.window + 1) : 0;
+    const int k_lo = first_key(p, p_min), k_first_max = first_key(p, p_max);      // the first key that any / every row sees
     const int kt_begin = k_lo / TC_KT, kt_end = p_max / TC_KT + 1;
     const int n_tiles = kt_end - kt_begin;
 
@@ -154,7 +154,9 @@ __global__ void __launch_bounds__(TC_THREADS, 2) attn_tc_kernel(const AttnParams
             unsigned vt_phase = 0;
             for (int j = 0; j < n_tiles; ++j) {
                 const int key0 = (kt_begin + j) * TC_KT;
-                const int key_b = key0 + lane * tma_box;
+                // boxes before the first key that is seen: their pages may have been given back; the rows of that key's own box
+                // stand in for them (finite, and no row of the block gives them weight)
+                const int key_b = max(key0 + lane * tma_box, k_lo - k_lo % tma_box);
                 const bool active = lane < n_box && key_b <= p_max;      // boxes past the last visible key are not fetched
                 int y = 0;
                 if (active) y = (bt[page_index(p, key_b)] * p.n_kv + kvh) * p.page_size + page_slot(p, key_b);
@@ -187,7 +189,7 @@ __global__ void __launch_bounds__(TC_THREADS, 2) attn_tc_kernel(const AttnParams
             // ---- cp.async: lane l gathers rows l, l + 32, l + 64, l + 96 of the tile, sixteen 16-byte chunks each
             auto row_page = [&](int kt, int row) -> int {
                 const int key = kt * TC_KT + row;
-                return (kt < kt_end && key <= p_max) ? bt[page_index(p, key)] : -1;
+                return (kt < kt_end && key <= p_max && key >= k_lo) ? bt[page_index(p, key)] : -1;
             };
             int pg[4], npg[4];
 #pragma unroll
@@ -282,7 +284,7 @@ __global__ void __launch_bounds__(TC_THREADS, 2) attn_tc_kernel(const AttnParams
         // =========================== softmax: thread t owns query row t (TMEM lane t)
         const unsigned lane_sel = (unsigned)(warp * 32) << 16;
         const int my_tl = tid / Gc;
-        const int my_pos = p_min + my_tl;
+        const int my_pos = p_min + my_tl, my_first = first_key(p, my_pos);
         const bool my_valid = my_tl < ti.n_tok && my_tl < QT && (chunk * TC_ROWS + (tid - my_tl * Gc)) < G;
         const float sc = p.scale * 1.4426950408889634f;
         float m_run = -INFINITY, l_run = 0.f;
@@ -299,7 +301,7 @@ __global__ void __launch_bounds__(TC_THREADS, 2) attn_tc_kernel(const AttnParams
             TC_MARK(0)
             const unsigned ts = t_s + lane_sel;
             const int key0 = (kt_begin + it) * TC_KT;
-            const bool need_mask = (key0 + TC_KT - 1 > p_min) || (p.window > 0 && key0 <= p_max - p.window);
+            const bool need_mask = (key0 + TC_KT - 1 > p_min) || key0 < k_first_max;
             // ---- one pass over S in chunks of 32 columns (the next chunk is on its way while this one is worked on):
             // P = 2^(s*scale - m) against the reference m of the row, which follows the running maximum only when a
             // chunk exceeds it by more than 2^TC_LAZY.  P and the sums then stay far inside the range of bfloat16 and
@@ -313,9 +315,7 @@ __global__ void __launch_bounds__(TC_THREADS, 2) attn_tc_kernel(const AttnParams
 #pragma unroll
                     for (int j = 0; j < 32; ++j) {
                         const int key = key0 + cb * 32 + j;
-                        bool okk = key <= my_pos;
-                        if (p.window > 0) okk = okk && (key > my_pos - p.window);
-                        if (!okk) sv[j] = -INFINITY;
+                        if (key > my_pos || key < my_first) sv[j] = -INFINITY;
                     }
                 }
                 float c4[4] = {sv[0], sv[1], sv[2], sv[3]};

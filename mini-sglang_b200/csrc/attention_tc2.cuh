@@ -93,7 +93,7 @@ __global__ void __launch_bounds__(TC2_THREADS, 1) attn_tc2_kernel(const AttnPara
     const int p_max = p_min + ti.n_tok - 1;
     const int ntok_a = min(ti.n_tok, QH), ntok_b = ti.n_tok - ntok_a;
     const int pmax_a = p_min + ntok_a - 1;
-    const int k_lo = p.window > 0 ? max(0, p_min - p.window + 1) : 0;
+    const int k_lo = first_key(p, p_min);                        // the first key any row of the block sees
     const int kt_begin = k_lo / TC_KT;
     // kept first tokens before the window's first tile: keys [0, sink_hi) in n_sink tiles that come first for both query tiles
     const int sink_hi = (EXT && p.window > 0) ? min(p.keep_first, kt_begin * TC_KT) : 0;
@@ -142,7 +142,10 @@ __global__ void __launch_bounds__(TC2_THREADS, 1) attn_tc2_kernel(const AttnPara
         const int n_box = TC_KT / tma_box;
         unsigned vt_phase = 0;
         auto box_row = [&](int j) -> int {            // first cache row of this lane's box of tile j, or -1
-            const int key_b = tile_of(j) * TC_KT + lane * tma_box;
+            int key_b = tile_of(j) * TC_KT + lane * tma_box;
+            // boxes before the first key that is seen: their pages may have been given back; the rows of that key's own box stand
+            // in for them (finite, and no row of the block gives them weight)
+            if (!(EXT && j < n_sink)) key_b = max(key_b, k_lo - k_lo % tma_box);
             if (j >= n_tiles || lane >= n_box || key_b > p_max) return -1;          // boxes past the last visible key are not fetched
             if (EXT && j < n_sink && key_b >= sink_hi) return -1;                   // nor those past the last kept token
             return (bt[page_index(p, key_b)] * p.n_kv + kvh) * p.page_size + page_slot(p, key_b);
@@ -269,7 +272,7 @@ __global__ void __launch_bounds__(TC2_THREADS, 1) attn_tc2_kernel(const AttnPara
             TC2_MARK(0)
             const int key0 = tile_of(it) * TC_KT;
             const bool in_sink = EXT && it < n_sink;
-            const bool need_mask = in_sink || (key0 + TC_KT - 1 > pmin_x) || (p.window > 0 && key0 <= pmax_x - p.window);
+            const bool need_mask = in_sink || (key0 + TC_KT - 1 > pmin_x) || key0 < first_key(p, pmax_x);
             float s0[32], s1[32], s2[32], s3[32];
             tc_ld32(ts, s0); tc_ld32(ts + 32, s1); tc_ld32(ts + 64, s2); tc_ld32(ts + 96, s3);
             tc_wait_ld(s0); tc_wait_ld(s1); tc_wait_ld(s2); tc_wait_ld(s3);
@@ -289,17 +292,13 @@ __global__ void __launch_bounds__(TC2_THREADS, 1) attn_tc2_kernel(const AttnPara
                 add_bias(s0, 0); add_bias(s1, 1); add_bias(s2, 2); add_bias(s3, 3);
             }
             if (need_mask) {
+                const int my_first = first_key(p, my_pos);
                 auto mask = [&](float (&sv)[32], int cb) {
 #pragma unroll
                     for (int j = 0; j < 32; ++j) {
                         const int key = key0 + cb * 32 + j;
-                        bool okk = key <= my_pos;
-                        if (EXT) {
-                            if (p.window > 0) okk = okk && (key > my_pos - p.window || key < p.keep_first);
-                            if (in_sink) okk = okk && key < sink_hi;
-                        } else if (p.window > 0) {
-                            okk = okk && (key > my_pos - p.window);
-                        }
+                        bool okk = key <= my_pos && (key >= my_first || (EXT && key < p.keep_first));
+                        if (EXT && in_sink) okk = okk && key < sink_hi;
                         if (!okk) sv[j] = -INFINITY;
                     }
                 };

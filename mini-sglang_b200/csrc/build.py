@@ -138,6 +138,7 @@ ATTENTION_SOURCES = ["attention.cu"]
 MIXER_SOURCES = ["mixers.cu"]
 GATED_MIXER_SOURCES = ["mixers_gated.cu"]
 DELTA_MIXER_SOURCES = ["mixers_delta.cu"]
+STREAM_MIXER_SOURCES = ["mixers_streams.cu"]
 MMA_HEAD_DIMS = tuple(range(16, 257, 16))   # head sizes the tensor-core attention kernel is built for
 
 
@@ -165,6 +166,12 @@ def delta_mixers_library() -> ctypes.CDLL:
     """The kernels of csrc/mixers_delta.cu (attention with a sink, the gated delta rule, scaled sums, the per-layer token
     input); built only for models that have such parts."""
     return load_library("mixers_delta", DELTA_MIXER_SOURCES)
+
+
+def stream_mixers_library() -> ctypes.CDLL:
+    """The kernels of csrc/mixers_streams.cu (several copies of the residual stream, heads that are the difference of two
+    maps); built only for models with such parts."""
+    return load_library("mixers_streams", STREAM_MIXER_SOURCES)
 
 
 def attention_library(head_dim: int) -> ctypes.CDLL:
@@ -197,7 +204,8 @@ def decode_step_library(head_dim: int) -> ctypes.CDLL:
 def build_all(head_dims: Sequence[int] = (16, 32, 48, 64, 128)) -> List[str]:
     """Compile every library ahead of time (used by the repository's build check)."""
     paths = [compile_library("common", COMMON_SOURCES), compile_library("mixers", MIXER_SOURCES),
-             compile_library("mixers_gated", GATED_MIXER_SOURCES), compile_library("mixers_delta", DELTA_MIXER_SOURCES)]
+             compile_library("mixers_gated", GATED_MIXER_SOURCES), compile_library("mixers_delta", DELTA_MIXER_SOURCES),
+             compile_library("mixers_streams", STREAM_MIXER_SOURCES)]
     for hd in head_dims:
         paths.append(compile_library(f"attention_d{hd}", ATTENTION_SOURCES, {"MSGL_HEAD_DIM": hd}))
     paths.append(compile_library("attention_noalloc_d128", ["attention_noalloc.cu"], {"MSGL_HEAD_DIM": 128}))

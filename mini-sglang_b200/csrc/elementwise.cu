@@ -69,7 +69,7 @@ __global__ void decode_meta_kernel(const int* __restrict__ id, const int* __rest
                                    int page_size, int mp, int common, int* __restrict__ input_ids, int* __restrict__ positions,
                                    int* __restrict__ token_req, int* __restrict__ q_start, int* __restrict__ kv_len,
                                    int* __restrict__ slots, int* __restrict__ out_loc, int* __restrict__ nsplit,
-                                   int* __restrict__ block_table, int window, int* __restrict__ order,
+                                   int* __restrict__ block_table, int window, int chunk_keys, int* __restrict__ order,
                                    const int* __restrict__ even_in, int* __restrict__ even_out, int n_even) {
     const int r = blockIdx.x;
     // the even cut of the step's keys comes ready-made from the host: the blocks copy it between them
@@ -87,6 +87,7 @@ __global__ void decode_meta_kernel(const int* __restrict__ id, const int* __rest
             if (j >= B) return 0;
             int keys = pos[j] + 1;
             if (window > 0) keys = min(keys, window + 1);
+            else if (chunk_keys > 0) keys = pos[j] % chunk_keys + 1;
             return (keys + max(nsplit_in[j], 1) - 1) / max(nsplit_in[j], 1);
         };
         const int mine = load_of(r);
@@ -125,13 +126,13 @@ MSGL_API int msgl_table_delta(const int* deltas, int n_records, int* table, int 
 MSGL_API int msgl_decode_meta(const int* id, const int* slot, const int* pos, const int* nsplit_in, int B, int b, const int* table,
                               int row_stride, int page_size, int mp, int common, int* input_ids, int* positions, int* token_req,
                               int* q_start, int* kv_len, int* slots, int* out_loc, int* nsplit, int* block_table,
-                              int window, int* order, const int* even_in, int* even_out, int n_even, cudaStream_t stream) {
+                              int window, int chunk_keys, int* order, const int* even_in, int* even_out, int n_even, cudaStream_t stream) {
     if (b <= 0) return MSGL_OK;
     if (B < 0 || B > b || page_size < 1 || mp < 1 || row_stride < 1 || order == nullptr) return MSGL_ERR_SIZE;
     if (n_even < 0 || (n_even > 0 && (even_in == nullptr || even_out == nullptr))) return MSGL_ERR_SIZE;
     decode_meta_kernel<<<b, 128, 0, stream>>>(id, slot, pos, nsplit_in, B, b, table, row_stride, page_size, mp, common, input_ids,
                                              positions, token_req, q_start, kv_len, slots, out_loc, nsplit, block_table,
-                                             window, order, even_in, even_out, n_even);
+                                             window, chunk_keys, order, even_in, even_out, n_even);
     return msgl_check_launch();
 }
 
@@ -153,13 +154,14 @@ MSGL_API int msgl_embedding(const int* ids, const void* table, float* out, int T
 //   v      = (res_in ? res_in[src] : 0) + (x ? float(x[src]) : 0)        src = row_idx ? row_idx[r] : r
 //   res_out[r] = v                                                        (if res_out)
 //   y[r]   = T(v * rsqrt(mean(v^2) + eps) * w)                            RMS
-//   y[r]   = T((v - mean(v)) * rsqrt(mean((v - mean(v))^2) + eps) * w)    CENTER: mean taken off, weight, no bias
+//   y[r]   = T((v - mean(v)) * rsqrt(mean((v - mean(v))^2) + eps) * w)    CENTER: mean taken off
+// With a bias b (float32 or null): y[r] += b, before the rounding to T.
 // One block per row; the row is kept in shared memory between the passes when it fits.  X: the type of x (T or float).
 // ---------------------------------------------------------------------------------------
 template <typename T, typename X, bool CENTER>
 __global__ void rmsnorm_kernel(const X* __restrict__ x, const float* res_in, float* res_out,
                                const int* __restrict__ row_idx, const void* __restrict__ w, int w_is_f32,
-                               float eps, T* __restrict__ y, int H, int cache_row) {
+                               float eps, T* __restrict__ y, int H, int cache_row, const float* __restrict__ b) {
     extern __shared__ float srow[];
     __shared__ float red[32];
     const int r = blockIdx.x;
@@ -191,7 +193,7 @@ __global__ void rmsnorm_kernel(const X* __restrict__ x, const float* res_in, flo
     const float total = block_sum(ss, red);
     const float inv = rsqrtf(total / (float)H + eps);
     for (int i = threadIdx.x; i < H; i += blockDim.x)
-        y[dst + i] = from_f32<T>((value(i) - mean) * inv * load_weight(w, i, w_is_f32));
+        y[dst + i] = from_f32<T>((value(i) - mean) * inv * load_weight(w, i, w_is_f32) + (b ? b[i] : 0.f));
 }
 
 // Vectorised variant: 8 elements per thread and pass, the whole row held in registers between the
@@ -227,7 +229,7 @@ template <> struct Vec8<__nv_bfloat16> {
 template <typename T, typename X, bool CENTER, int VPT>
 __global__ void rmsnorm_vec_kernel(const X* __restrict__ x, const float* res_in, float* res_out,
                                    const int* __restrict__ row_idx, const void* __restrict__ w, int w_is_f32,
-                                   float eps, T* __restrict__ y, int H) {
+                                   float eps, T* __restrict__ y, int H, const float* __restrict__ b) {
     __shared__ float red[32];
     pdl_launch_dependents();
     const int r = blockIdx.x;
@@ -289,6 +291,12 @@ __global__ void rmsnorm_vec_kernel(const X* __restrict__ x, const float* res_in,
             float o[8];
 #pragma unroll
             for (int k = 0; k < 8; ++k) o[k] = v[j][k] * inv * wv[j][k];
+            if (b) {
+                float bv[8];
+                Vec8<float>::load(b + i, bv);
+#pragma unroll
+                for (int k = 0; k < 8; ++k) o[k] += bv[k];
+            }
             Vec8<T>::store(y + dst + i, o);
         }
     }
@@ -296,8 +304,8 @@ __global__ void rmsnorm_vec_kernel(const X* __restrict__ x, const float* res_in,
 
 template <typename T, typename X, bool CENTER>
 static int launch_norm(const void* x, const float* res_in, float* res_out, const int* row_idx, const void* w, int w_is_f32,
-                       float eps, void* y, int rows, int H, cudaStream_t stream) {
-    const uintptr_t all = (uintptr_t)x | (uintptr_t)res_in | (uintptr_t)res_out | (uintptr_t)w | (uintptr_t)y;
+                       float eps, void* y, int rows, int H, const float* b, cudaStream_t stream) {
+    const uintptr_t all = (uintptr_t)b | (uintptr_t)x | (uintptr_t)res_in | (uintptr_t)res_out | (uintptr_t)w | (uintptr_t)y;
     const X* xp = (const X*)x;
     T* yp = (T*)y;
     if (!((H & 7) || (all & 15))) {
@@ -306,28 +314,28 @@ static int launch_norm(const void* x, const float* res_in, float* res_out, const
         int vpt = 1;
         while (threads > 512) { vpt *= 2; threads = (((nvec + vpt - 1) / vpt + 31) / 32) * 32; }
         if (vpt <= 4) {
-            if (vpt == 1) msgl_launch_pdl(rmsnorm_vec_kernel<T, X, CENTER, 1>, dim3(rows), dim3(threads), 0, stream, xp, res_in, res_out, row_idx, w, w_is_f32, eps, yp, H);
-            else if (vpt == 2) msgl_launch_pdl(rmsnorm_vec_kernel<T, X, CENTER, 2>, dim3(rows), dim3(threads), 0, stream, xp, res_in, res_out, row_idx, w, w_is_f32, eps, yp, H);
-            else msgl_launch_pdl(rmsnorm_vec_kernel<T, X, CENTER, 4>, dim3(rows), dim3(threads), 0, stream, xp, res_in, res_out, row_idx, w, w_is_f32, eps, yp, H);
+            if (vpt == 1) msgl_launch_pdl(rmsnorm_vec_kernel<T, X, CENTER, 1>, dim3(rows), dim3(threads), 0, stream, xp, res_in, res_out, row_idx, w, w_is_f32, eps, yp, H, b);
+            else if (vpt == 2) msgl_launch_pdl(rmsnorm_vec_kernel<T, X, CENTER, 2>, dim3(rows), dim3(threads), 0, stream, xp, res_in, res_out, row_idx, w, w_is_f32, eps, yp, H, b);
+            else msgl_launch_pdl(rmsnorm_vec_kernel<T, X, CENTER, 4>, dim3(rows), dim3(threads), 0, stream, xp, res_in, res_out, row_idx, w, w_is_f32, eps, yp, H, b);
             return msgl_check_launch();
         }
     }
     const int threads = H >= 2048 ? 512 : (H >= 512 ? 256 : 128);
     const int cache_row = (size_t)H * 4 <= 40 * 1024;
     const size_t smem = cache_row ? (size_t)H * 4 : 0;
-    rmsnorm_kernel<T, X, CENTER><<<rows, threads, smem, stream>>>(xp, res_in, res_out, row_idx, w, w_is_f32, eps, yp, H, cache_row);
+    rmsnorm_kernel<T, X, CENTER><<<rows, threads, smem, stream>>>(xp, res_in, res_out, row_idx, w, w_is_f32, eps, yp, H, cache_row, b);
     return msgl_check_launch();
 }
 
-// x_is_f32: x is float32 whatever the output type; center: LayerNorm (mean taken off), else RMSNorm
+// x_is_f32: x is float32 whatever the output type; center: LayerNorm (mean taken off), else RMSNorm; b: float32 bias or null
 MSGL_API int msgl_rmsnorm(const void* x, int x_is_f32, const float* res_in, float* res_out, const int* row_idx,
                           const void* w, int w_is_f32, float eps, int center, void* y, int rows, int H,
-                          int dtype, cudaStream_t stream) {
+                          int dtype, const float* b, cudaStream_t stream) {
     if (rows <= 0) return MSGL_OK;
     if (H <= 0) return MSGL_ERR_SIZE;
 #define NORM(T, X)                                                                                                          \
-    (center ? launch_norm<T, X, true>(x, res_in, res_out, row_idx, w, w_is_f32, eps, y, rows, H, stream)                     \
-            : launch_norm<T, X, false>(x, res_in, res_out, row_idx, w, w_is_f32, eps, y, rows, H, stream))
+    (center ? launch_norm<T, X, true>(x, res_in, res_out, row_idx, w, w_is_f32, eps, y, rows, H, b, stream)                     \
+            : launch_norm<T, X, false>(x, res_in, res_out, row_idx, w, w_is_f32, eps, y, rows, H, b, stream))
     if (dtype == MSGL_F32) return NORM(float, float);
     if (dtype == MSGL_BF16) return x_is_f32 ? NORM(__nv_bfloat16, float) : NORM(__nv_bfloat16, __nv_bfloat16);
 #undef NORM

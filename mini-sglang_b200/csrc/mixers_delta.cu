@@ -4,10 +4,12 @@
 //
 //   scaled_add_norm_kernel     res += x * s (s a float32 vector of the width), then y = rms(res) * w or y = res (or no y)
 //   rotary_angles_kernel       cos | sin of position * frequency for the tokens of a step, in double precision
-//   sink_qkv_prep_kernel       q and k heads RMS-normed, rotated in halves from the step's angles, values blended with another
-//                              layer's or brought to unit root mean square (each where asked), K and V rows (of head sizes of
-//                              their own) into the paged cache; a 16-byte form where nothing is rotated or blended
-//   sink_attention_kernel      causal softmax attention within a window over the paged cache, scores capped by a tanh
+//   sink_qkv_prep_kernel       q and k heads RMS-normed, rotated in halves or in neighbouring pairs from the step's angles and
+//                              brought to unit root mean square, heads of several maps laid out for one kv head, values
+//                              blended with another layer's or brought to unit root mean square (each where asked), K and V
+//                              rows (of head sizes of their own) into the paged cache; a 16-byte form where nothing is
+//                              blended or rotated in halves
+//   sink_attention_kernel      causal softmax attention within a window or a chunk over the paged cache, scores capped by a tanh
 //                              where asked, with exp(sink_h) in the denominator and the output times a sigmoid gate per
 //                              element where given; float32 arithmetic, any head size to 512
 //   sink_attention_mma_kernel  the same for bfloat16 with both products on mma.sync tiles (64 rows a block, float32 scores,
@@ -161,10 +163,14 @@ MSGL_API int msgl_rotary_angles(const int* positions, const double* freq, double
 // ---------------------------------------------------------------------------------------
 // q, k, v of a packed projection row [q: n_q * d | k: n_kv * d | v: n_kv * dv]:
 //   q and k heads: where weights are given (wq, wk [d], for all heads), x / sqrt(mean(x^2) + eps) * w first; then the first
-//   `rot` elements turn in halves by the token's angles (cs [T][rot] = cos | sin), the rest pass
+//   `rot` elements turn by the token's angles (cs [T][rot] = cos | sin), in halves (element i with i + rot / 2) or, with
+//   `interleaved`, in neighbouring pairs (2 i with 2 i + 1), the rest pass; with qk_unit then x / sqrt(mean(x^2) + eps)
 //   v heads: v <- (1 - lam) v + lam v_first where another layer's values are given; with v_unit then v / sqrt(mean(v^2) + eps)
 //   q -> q_out [T, n_q, d]; k, v -> the paged caches at token slot out_loc[t] (where given)
-// One warp per (token, head of q, k or v).
+// With maps = M > 1 every q and kv head has M vectors of d elements side by side, each treated as a head of its own by all of
+// the above: K rows are the M vectors of a kv head [M * d]; q comes out as n_q * M rows of M * d elements of which row
+// (h, m) has its vector in place m and zeros in the others, so that its product with a K row is that of map m alone.
+// One warp per (token, vector of q, k or v).
 // ---------------------------------------------------------------------------------------
 __device__ __forceinline__ void sk_load16(const float* p, float (&v)[4]) {
     const float4 a = *reinterpret_cast<const float4*>(p);
@@ -192,29 +198,33 @@ struct SinkPrepParams {
     const int* out_loc; void* q_out; void* k_cache; void* v_cache;
     int page_size, n_q, n_kv, d, dv, T;
     const float* wq; const float* wk; int v_unit; float eps;
+    int interleaved, qk_unit, maps;
 };
 
 template <typename T>
 __global__ void __launch_bounds__(128) sink_qkv_prep_kernel(const SinkPrepParams p) {
     const int t = blockIdx.x;
     const int slot = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-    const int n_slots = p.n_q + 2 * p.n_kv;
-    if (slot >= n_slots) return;
+    const int M = p.maps, nq = p.n_q * M, nk = p.n_kv * M;
+    if (slot >= nq + nk + p.n_kv) return;
     const T* row = reinterpret_cast<const T*>(p.proj) + (size_t)t * p.stride;
     const int half = p.rot >> 1;
     const float* cs = p.cs ? p.cs + (size_t)t * p.rot : nullptr;
-    if (slot < p.n_q + p.n_kv) {
-        const bool is_q = slot < p.n_q;
-        const int h = is_q ? slot : slot - p.n_q;
-        const T* src = row + (is_q ? 0 : (size_t)p.n_q * p.d) + (size_t)h * p.d;
+    if (slot < nq + nk) {
+        const bool is_q = slot < nq;
+        const int h = is_q ? slot : slot - nq, m = h % M;
+        const T* src = row + (size_t)slot * p.d;
         T* dst;
         if (is_q) {
-            dst = reinterpret_cast<T*>(p.q_out) + ((size_t)t * p.n_q + h) * p.d;
+            dst = reinterpret_cast<T*>(p.q_out) + ((size_t)t * nq + h) * p.d * M;
+            for (int e = lane; e < p.d * M; e += 32)
+                if (e / p.d != m) dst[e] = from_f32<T>(0.f);
         } else {
             if (p.k_cache == nullptr) return;
             const int loc = p.out_loc[t];
-            dst = reinterpret_cast<T*>(p.k_cache) + (((size_t)(loc / p.page_size) * p.n_kv + h) * p.page_size + loc % p.page_size) * p.d;
+            dst = reinterpret_cast<T*>(p.k_cache) + (((size_t)(loc / p.page_size) * p.n_kv + h / M) * p.page_size + loc % p.page_size) * p.d * M;
         }
+        dst += m * p.d;
         const float* w = is_q ? p.wq : p.wk;
         float f = 1.f;
         if (w != nullptr) {
@@ -223,18 +233,26 @@ __global__ void __launch_bounds__(128) sink_qkv_prep_kernel(const SinkPrepParams
             f = 1.f / sqrtf(warp_sum(ss) / (float)p.d + p.eps);
         }
         auto elem = [&](int e) -> float { const float v = to_f32<T>(src[e]); return w != nullptr ? v * f * w[e] : v; };
-        for (int e = lane; e < p.d; e += 32) {
-            float v = elem(e);
-            if (cs != nullptr && e < p.rot) {
-                if (e < half) v = v * cs[e] - elem(e + half) * cs[half + e];
-                else v = v * cs[e - half] + elem(e - half) * cs[e];
+        auto turned = [&](int e) -> float {
+            const float v = elem(e);
+            if (cs == nullptr || e >= p.rot) return v;
+            if (p.interleaved) {
+                const float c = cs[e >> 1], s = cs[half + (e >> 1)], o = elem(e ^ 1);
+                return (e & 1) ? v * c + o * s : v * c - o * s;
             }
-            dst[e] = from_f32<T>(v);
+            return e < half ? v * cs[e] - elem(e + half) * cs[half + e] : v * cs[e - half] + elem(e - half) * cs[e];
+        };
+        float g = 1.f;
+        if (p.qk_unit) {
+            float ss = 0.f;
+            for (int e = lane; e < p.d; e += 32) { const float v = turned(e); ss = fmaf(v, v, ss); }
+            g = 1.f / sqrtf(warp_sum(ss) / (float)p.d + p.eps);
         }
+        for (int e = lane; e < p.d; e += 32) dst[e] = from_f32<T>(turned(e) * g);
     } else {
         if (p.v_cache == nullptr) return;
-        const int h = slot - p.n_q - p.n_kv;
-        const T* src = row + (size_t)(p.n_q + p.n_kv) * p.d + (size_t)h * p.dv;
+        const int h = slot - nq - nk;
+        const T* src = row + (size_t)(nq + nk) * p.d + (size_t)h * p.dv;
         const T* vf = p.v_first ? reinterpret_cast<const T*>(p.v_first) + (size_t)t * p.vf_stride + (size_t)h * p.dv : nullptr;
         const int loc = p.out_loc[t];
         T* dst = reinterpret_cast<T*>(p.v_cache) + (((size_t)(loc / p.page_size) * p.n_kv + h) * p.page_size + loc % p.page_size) * p.dv;
@@ -252,81 +270,119 @@ __global__ void __launch_bounds__(128) sink_qkv_prep_kernel(const SinkPrepParams
     }
 }
 
-// The same without rotation or blending, a lane 16 bytes of a head (head sizes that are multiples of the vector and at most
-// 32 vectors): one read of every element, the norms from registers.
+// The same without blending or a rotation in halves, a lane 16 bytes of a vector (sizes that are multiples of the lane's share and
+// at most 32 of them): one read of every element, norms and turned pairs from registers.  n_slots: the vectors of a token that
+// are made (q alone where nothing is cached).
 template <typename T>
-__global__ void __launch_bounds__(128) sink_qkv_prep_vec_kernel(const SinkPrepParams p) {
+__global__ void __launch_bounds__(128) sink_qkv_prep_vec_kernel(const SinkPrepParams p, int n_slots) {
     constexpr int V = 16 / sizeof(T);
     const long long w_idx = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
-    const int n_slots = p.n_q + 2 * p.n_kv, lane = threadIdx.x & 31;
-    // heads of a size of 16 vectors or less share a warp: `per` heads side by side
+    const int M = p.maps, nq = p.n_q * M, nk = p.n_kv * M, lane = threadIdx.x & 31;
+    // vectors of 16 shares or less share a warp: `per` of them side by side
     const int nd = p.d / V, nv = p.dv / V, widest = nd > nv ? nd : nv;
     const int lanes = widest <= 4 ? 4 : widest <= 8 ? 8 : widest <= 16 ? 16 : 32, per = 32 / lanes;
     const long long job = w_idx * per + lane / lanes;
     const int l = lane % lanes;
     const bool live = job < (long long)p.T * n_slots;
     const int t = live ? (int)(job / n_slots) : 0, slot = live ? (int)(job - (long long)t * n_slots) : 0;
-    const bool is_v = slot >= p.n_q + p.n_kv, is_q = slot < p.n_q;
+    const bool is_v = slot >= nq + nk, is_q = slot < nq;
     const int n = is_v ? p.dv : p.d;
     const T* row = reinterpret_cast<const T*>(p.proj) + (size_t)t * p.stride;
-    const T* src = is_v ? row + (size_t)(p.n_q + p.n_kv) * p.d + (size_t)(slot - p.n_q - p.n_kv) * p.dv : row + (size_t)slot * p.d;
-    const bool mine = live && l * V < n && (is_q || p.k_cache != nullptr);
+    const T* src = is_v ? row + (size_t)(nq + nk) * p.d + (size_t)(slot - nq - nk) * p.dv : row + (size_t)slot * p.d;
+    const bool mine = live && l * V < n;
     float v[V];
 #pragma unroll
     for (int k = 0; k < V; ++k) v[k] = 0.f;
     if (mine) sk_load16(src + l * V, v);
-    float ss = 0.f;
-#pragma unroll
-    for (int k = 0; k < V; ++k) ss = fmaf(v[k], v[k], ss);
-    for (int o = lanes >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
-    if (!mine) return;
     const float* w = is_v ? nullptr : (is_q ? p.wq : p.wk);
-    const float f = (is_v ? p.v_unit != 0 : w != nullptr) ? 1.f / sqrtf(ss / (float)n + p.eps) : 1.f;
-    if (w != nullptr) {
-        const float4* w4 = reinterpret_cast<const float4*>(w + l * V);
+    if (w != nullptr || (is_v && p.v_unit)) {           // (the lanes of one vector take the same branch: the shuffles stay among them)
+        float ss = 0.f;
 #pragma unroll
-        for (int k = 0; k < V / 4; ++k) {
-            const float4 x = w4[k];
-            v[4 * k] *= f * x.x; v[4 * k + 1] *= f * x.y; v[4 * k + 2] *= f * x.z; v[4 * k + 3] *= f * x.w;
+        for (int k = 0; k < V; ++k) ss = fmaf(v[k], v[k], ss);
+        const unsigned mask = lanes == 32 ? 0xffffffffu : ((1u << lanes) - 1u) << (lane / lanes * lanes);
+        for (int o = lanes >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(mask, ss, o);
+        const float f = 1.f / sqrtf(ss / (float)n + p.eps);
+        if (w != nullptr && mine) {
+            const float4* w4 = reinterpret_cast<const float4*>(w + l * V);
+#pragma unroll
+            for (int k = 0; k < V / 4; ++k) {
+                const float4 x = w4[k];
+                v[4 * k] *= f * x.x; v[4 * k + 1] *= f * x.y; v[4 * k + 2] *= f * x.z; v[4 * k + 3] *= f * x.w;
+            }
+        } else {
+#pragma unroll
+            for (int k = 0; k < V; ++k) v[k] *= f;
         }
-    } else {
+    }
+    if (p.cs != nullptr && !is_v && mine) {             // neighbouring pairs lie within a lane
+        const float* cs = p.cs + (size_t)t * p.rot;
+        const int half = p.rot >> 1;
+#pragma unroll
+        for (int k = 0; k < V; k += 2) {
+            const int pr = (l * V + k) >> 1;
+            if (pr < half) {
+                const float c = cs[pr], s = cs[half + pr], a = v[k], b = v[k + 1];
+                v[k] = a * c - b * s;
+                v[k + 1] = b * c + a * s;
+            }
+        }
+    }
+    if (p.qk_unit && !is_v) {
+        float ss = 0.f;
+#pragma unroll
+        for (int k = 0; k < V; ++k) ss = fmaf(v[k], v[k], ss);
+        const unsigned mask = lanes == 32 ? 0xffffffffu : ((1u << lanes) - 1u) << (lane / lanes * lanes);
+        for (int o = lanes >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(mask, ss, o);
+        const float f = 1.f / sqrtf(ss / (float)n + p.eps);
 #pragma unroll
         for (int k = 0; k < V; ++k) v[k] *= f;
     }
+    if (!mine) return;
     T* dst;
     if (is_q) {
-        dst = reinterpret_cast<T*>(p.q_out) + ((size_t)t * p.n_q + slot) * p.d;
+        const int m = slot % M;
+        dst = reinterpret_cast<T*>(p.q_out) + ((size_t)t * nq + slot) * n * M + l * V;
+        float z[V];
+#pragma unroll
+        for (int k = 0; k < V; ++k) z[k] = 0.f;
+        for (int o = 0; o < M; ++o)
+            if (o != m) sk_store16(dst + o * n, z);
+        dst += m * n;
     } else {
-        const int loc = p.out_loc[t], h = is_v ? slot - p.n_q - p.n_kv : slot - p.n_q;
+        const int loc = p.out_loc[t], h = is_v ? slot - nq - nk : slot - nq;
+        const int mm = is_v ? 1 : M;
         dst = reinterpret_cast<T*>(is_v ? p.v_cache : p.k_cache) +
-              (((size_t)(loc / p.page_size) * p.n_kv + h) * p.page_size + loc % p.page_size) * n;
+              (((size_t)(loc / p.page_size) * p.n_kv + h / mm) * p.page_size + loc % p.page_size) * n * mm + h % mm * n + l * V;
     }
-    sk_store16(dst + l * V, v);
+    sk_store16(dst, v);
 }
 
 MSGL_API int msgl_sink_qkv_prep(const void* proj, long long stride, const float* cs, int rot, const void* v_first, long long vf_stride,
                                 float lam, const int* out_loc, void* q_out, void* k_cache, void* v_cache, int page_size, int n_q, int n_kv,
                                 int d, int dv, int T_, int dtype, const float* wq, const float* wk, int v_unit, float eps,
-                                cudaStream_t stream) {
+                                int interleaved, int qk_unit, int maps, cudaStream_t stream) {
     if (T_ <= 0) return MSGL_OK;
     if (dtype != MSGL_F32 && dtype != MSGL_BF16) return MSGL_ERR_DTYPE;
-    if (d <= 0 || dv <= 0 || n_q <= 0 || n_kv <= 0 || rot < 0 || rot > d || (rot & 1) || page_size < 1 || (rot > 0 && cs == nullptr) ||
+    if (d <= 0 || dv <= 0 || n_q <= 0 || n_kv <= 0 || rot < 0 || rot > d || (rot & 1) || page_size < 1 || maps < 1 || (rot > 0 && cs == nullptr) ||
         (k_cache != nullptr && (out_loc == nullptr || v_cache == nullptr)))
         return MSGL_ERR_SIZE;
     SinkPrepParams p;
     p.proj = proj; p.stride = stride; p.cs = rot > 0 ? cs : nullptr; p.rot = rot; p.v_first = v_first; p.vf_stride = vf_stride; p.lam = lam;
     p.out_loc = out_loc; p.q_out = q_out; p.k_cache = k_cache; p.v_cache = v_cache; p.page_size = page_size; p.n_q = n_q; p.n_kv = n_kv;
     p.d = d; p.dv = dv; p.T = T_; p.wq = wq; p.wk = wk; p.v_unit = v_unit; p.eps = eps;
+    p.interleaved = interleaved; p.qk_unit = qk_unit; p.maps = maps;
     const int V = dtype == MSGL_F32 ? 4 : 8;
     const uintptr_t all = (uintptr_t)proj | (uintptr_t)q_out | (uintptr_t)k_cache | (uintptr_t)v_cache | (uintptr_t)wq | (uintptr_t)wk;
-    if (p.cs == nullptr && v_first == nullptr && d % V == 0 && dv % V == 0 && stride % V == 0 && max(d, dv) <= 32 * V && (all & 15) == 0) {
+    // vectors of a token: q, and where they are cached k and v
+    const int n_slots = maps * n_q + (k_cache != nullptr ? (maps + 1) * n_kv : 0);
+    if ((p.cs == nullptr || interleaved) && v_first == nullptr && d % V == 0 && dv % V == 0 && stride % V == 0 && max(d, dv) <= 32 * V && (all & 15) == 0) {
         const int widest = max(d, dv) / V, lanes = widest <= 4 ? 4 : widest <= 8 ? 8 : widest <= 16 ? 16 : 32, per = 4 * (32 / lanes);
-        const unsigned blocks = (unsigned)(((long long)T_ * (n_q + 2 * n_kv) + per - 1) / per);
-        if (dtype == MSGL_F32) sink_qkv_prep_vec_kernel<float><<<blocks, 128, 0, stream>>>(p);
-        else sink_qkv_prep_vec_kernel<__nv_bfloat16><<<blocks, 128, 0, stream>>>(p);
+        const unsigned blocks = (unsigned)(((long long)T_ * n_slots + per - 1) / per);
+        if (dtype == MSGL_F32) sink_qkv_prep_vec_kernel<float><<<blocks, 128, 0, stream>>>(p, n_slots);
+        else sink_qkv_prep_vec_kernel<__nv_bfloat16><<<blocks, 128, 0, stream>>>(p, n_slots);
         return msgl_check_launch();
     }
-    const dim3 grid(T_, (n_q + 2 * n_kv + 3) / 4);
+    const dim3 grid(T_, (n_slots + 3) / 4);
     if (dtype == MSGL_F32) sink_qkv_prep_kernel<float><<<grid, 128, 0, stream>>>(p);
     else if (dtype == MSGL_BF16) sink_qkv_prep_kernel<__nv_bfloat16><<<grid, 128, 0, stream>>>(p);
     else return MSGL_ERR_DTYPE;
@@ -334,10 +390,11 @@ MSGL_API int msgl_sink_qkv_prep(const void* proj, long long stride, const float*
 }
 
 // ---------------------------------------------------------------------------------------
-// Causal softmax attention within a window over the paged cache, with a sink
+// Causal softmax attention within a window or a chunk over the paged cache, with a sink
 //
-//   s(i, j) = q[i, h] . k[j, g] * scale;   s <- cap * tanh(s / cap) (cap > 0);   j <= i and (no window or i - j < window)
-//   o[i, h, :] = sum_j exp(s(i, j)) v[j, g, :] / (sum_j exp(s(i, j)) + exp(sink[h]))
+//   s(i, j) = q[i, h] . k[j, g] * scale;   s <- cap * tanh(s / cap) (cap > 0);   j <= i and (no window or i - j < window) and
+//   (no chunks or j / chunk_keys == i / chunk_keys)
+//   o[i, h, :] = sum_j exp(s(i, j)) v[j, g, :] / (sum_j exp(s(i, j)) + exp(sink[h]))        (sink null: without that term)
 //   o[i, h, e] <- o[i, h, e] * sigmoid(gate[i, h, e])   (where gates are given: rows of the activation type, one per output element)
 //
 // A block owns a tile of QT tokens x GH query heads of one kv head (SK_ROWS rows, one warp each) and walks the keys in
@@ -356,13 +413,20 @@ struct SinkAttnParams {
     const void* k_cache; const void* v_cache;
     const int* q_start; const int* kv_len; const int* block_table; int bt_stride;
     int uniform;
-    const float* sink;                            // [n_q]
+    const float* sink;                            // [n_q] or null
     void* out; long long out_stride;              // [T rows][n_q * dv]
     float* part_o; float* part_ml; int splits, split_keys;      // [splits][T][n_q][dv], [splits][T][n_q][2]
     int T, B, n_q, n_kv, d, dv, page_size, QT, GH, window;
     float scale, softcap;
     const void* gate; long long gate_stride;      // [T rows][n_q * dv] or null
+    int chunk_keys;                               // > 0 (without a window): keys are seen within chunks of the sequence only
 };
+
+// the first key that the query at position `pos` sees
+__device__ __forceinline__ int sk_first_key(const SinkAttnParams& p, int pos) {
+    if (p.window > 0) return max(0, pos - p.window + 1);
+    return p.chunk_keys > 0 ? pos - pos % p.chunk_keys : 0;
+}
 
 template <typename T, int DPL>
 __global__ void __launch_bounds__(SK_ROWS * 32) sink_attention_kernel(const SinkAttnParams p) {
@@ -397,7 +461,7 @@ __global__ void __launch_bounds__(SK_ROWS * 32) sink_attention_kernel(const Sink
     const int n_tok = min(p.QT, q_len - t0);
     if (n_tok <= 0) return;
     const int p_min = kv_len - q_len + t0, p_max = p_min + n_tok - 1;
-    int key_lo = p.window > 0 ? max(0, p_min - p.window + 1) : 0, key_hi = p_max + 1;      // keys this block walks: [key_lo, key_hi)
+    int key_lo = sk_first_key(p, p_min), key_hi = p_max + 1;      // keys this block walks: [key_lo, key_hi)
     if (p.splits > 1) {
         const int piece = key_lo / p.split_keys + blockIdx.z;
         key_lo = max(key_lo, piece * p.split_keys);
@@ -410,7 +474,7 @@ __global__ void __launch_bounds__(SK_ROWS * 32) sink_attention_kernel(const Sink
     const int head = kvh * G + (row_ok ? hg : 0);
     const int tok = q_base + t0 + (row_ok ? tl : 0);
     const int pos = p_min + tl;
-    const int first_seen = p.window > 0 ? pos - p.window + 1 : 0;
+    const int first_seen = sk_first_key(p, pos);
     const T* qg = reinterpret_cast<const T*>(p.q);
     for (int e = lane; e < d; e += 32) qs[warp * d + e] = row_ok ? to_f32<T>(qg[((size_t)tok * p.n_q + head) * d + e]) : 0.f;
     const T* kc = reinterpret_cast<const T*>(p.k_cache);
@@ -489,7 +553,7 @@ __global__ void __launch_bounds__(SK_ROWS * 32) sink_attention_kernel(const Sink
         if (lane == 0) { p.part_ml[2 * r] = m_run; p.part_ml[2 * r + 1] = l_run; }
         return;
     }
-    const float sk = p.sink[head];
+    const float sk = p.sink ? p.sink[head] : -INFINITY;
     const float M = fmaxf(m_run, sk);
     const float f = expf(m_run - M);
     const float inv = f / (l_run * f + expf(sk - M));
@@ -513,9 +577,10 @@ __global__ void __launch_bounds__(128) sink_merge_kernel(const float* __restrict
                                                          long long gate_stride) {
     const int t = blockIdx.x, head = blockIdx.y;
     const size_t r0 = (size_t)t * n_q + head, step = (size_t)T_ * n_q;
-    float M = sink[head];
+    const float sk = sink ? sink[head] : -INFINITY;
+    float M = sk;
     for (int s = 0; s < splits; ++s) M = fmaxf(M, part_ml[2 * (r0 + s * step)]);
-    float den = expf(sink[head] - M);
+    float den = expf(sk - M);
     for (int s = 0; s < splits; ++s) den = fmaf(part_ml[2 * (r0 + s * step) + 1], expf(part_ml[2 * (r0 + s * step)] - M), den);
     const float inv = 1.f / den;
     for (int e = threadIdx.x; e < dv; e += blockDim.x) {
@@ -534,10 +599,10 @@ MSGL_API int msgl_sink_attention(const void* q, const void* k_cache, const void*
                                  const int* block_table, int bt_stride, int uniform, int n_tiles, const float* sink, void* out,
                                  long long out_stride, float* part_o, float* part_ml, int splits, int split_keys, int T_, int B, int n_q,
                                  int n_kv, int d, int dv, int page_size, int QT, int GH, int window, float scale, float softcap, int dtype,
-                                 const void* gate, long long gate_stride, cudaStream_t stream) {
+                                 const void* gate, long long gate_stride, int chunk_keys, cudaStream_t stream) {
     if (n_tiles <= 0) return MSGL_OK;
     if (d <= 0 || dv <= 0 || dv > 32 * SK_MAX_DPL || d > 32 * SK_MAX_DPL || n_kv <= 0 || n_q % n_kv || QT < 1 || GH < 1 ||
-        QT * GH > SK_ROWS || page_size < 1 || sink == nullptr || window < 0 || splits < 1 ||
+        QT * GH > SK_ROWS || page_size < 1 || window < 0 || chunk_keys < 0 || (window > 0 && chunk_keys > 0) || splits < 1 ||
         (splits > 1 && (!uniform || part_o == nullptr || part_ml == nullptr || split_keys < SK_KC || split_keys % SK_KC)))
         return MSGL_ERR_SIZE;
     if (dtype != MSGL_F32 && dtype != MSGL_BF16) return MSGL_ERR_DTYPE;
@@ -546,7 +611,7 @@ MSGL_API int msgl_sink_attention(const void* q, const void* k_cache, const void*
     p.bt_stride = bt_stride; p.uniform = uniform; p.sink = sink; p.out = out; p.out_stride = out_stride; p.part_o = part_o;
     p.part_ml = part_ml; p.splits = splits; p.split_keys = split_keys; p.T = T_; p.B = B; p.n_q = n_q; p.n_kv = n_kv; p.d = d; p.dv = dv;
     p.page_size = page_size; p.QT = QT; p.GH = GH; p.window = window; p.scale = scale; p.softcap = softcap;
-    p.gate = gate; p.gate_stride = gate_stride;
+    p.gate = gate; p.gate_stride = gate_stride; p.chunk_keys = chunk_keys;
     const int G = n_q / n_kv;
     const dim3 grid(n_tiles, n_kv * ((G + GH - 1) / GH), splits);
     const size_t smem = ((size_t)SK_ROWS * d + (size_t)SK_KC * (d + 1) + (size_t)SK_KC * dv) * sizeof(float);
@@ -660,7 +725,7 @@ __global__ void __launch_bounds__(SKM_THREADS) sink_attention_mma_kernel(const S
     const int n_tok = min(QT, q_len - t0);
     if (n_tok <= 0) return;
     const int p_min = kv_len - q_len + t0, p_max = p_min + n_tok - 1;
-    const int key_lo = p.window > 0 ? max(0, p_min - p.window + 1) : 0;      // the first key any row of the block sees
+    const int key_lo = sk_first_key(p, p_min);      // the first key any row of the block sees
     int kt_lo = key_lo / SKM_KT, kt_hi = p_max / SKM_KT + 1;
     if (p.splits > 1) {       // a piece is a whole number of tiles, counted from the piece that holds key_lo
         const int piece = key_lo / p.split_keys + (int)blockIdx.z;
@@ -680,7 +745,7 @@ __global__ void __launch_bounds__(SKM_THREADS) sink_attention_mma_kernel(const S
     const int tl_lo = r_lo / Gc, tl_hi = r_hi / Gc;
     const int hl_lo = r_lo - tl_lo * Gc, hl_hi = r_hi - tl_hi * Gc;
     const int pos_lo = p_min + tl_lo, pos_hi = p_min + tl_hi;
-    const int first_lo = p.window > 0 ? pos_lo - p.window + 1 : 0, first_hi = p.window > 0 ? pos_hi - p.window + 1 : 0;
+    const int first_lo = sk_first_key(p, pos_lo), first_hi = sk_first_key(p, pos_hi);
     float o[NDB][4];
 #pragma unroll
     for (int i = 0; i < NDB; ++i) { o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f; }
@@ -721,6 +786,7 @@ __global__ void __launch_bounds__(SKM_THREADS) sink_attention_mma_kernel(const S
 
         const bool warp_live = row_base / Gc < n_tok;       // else all 16 rows of the warp are empty: it copies, but multiplies nothing
         const int warp_pos_lo = p_min + row_base / Gc, warp_pos_hi = p_min + (row_base + 15) / Gc;
+        const int warp_first_lo = sk_first_key(p, warp_pos_lo), warp_first_hi = sk_first_key(p, warp_pos_hi);
         const unsigned q_a = q_s + (unsigned)((row_base + (lane & 15)) * LDK + (lane >> 4) * 8) * 2u;
         const unsigned k_lane = (unsigned)(((lane & 7) + ((lane >> 4) & 1) * 8) * LDK + ((lane >> 3) & 1) * 8) * 2u;
         const unsigned v_lane = (unsigned)(((lane & 7) + ((lane >> 3) & 1) * 8) * LDV + ((lane >> 4) & 1) * 8) * 2u;
@@ -738,8 +804,8 @@ __global__ void __launch_bounds__(SKM_THREADS) sink_attention_mma_kernel(const S
             }
             __syncthreads();
             const int key0 = kt * SKM_KT;
-            // no row of the warp sees a key of this tile: the tile lies behind its last token or before its first token's window
-            if (!warp_live || key0 > warp_pos_hi || (p.window > 0 && key0 + SKM_KT - 1 < warp_pos_lo - p.window + 1)) {
+            // no row of the warp sees a key of this tile: the tile lies behind its last token or before its first token's first key
+            if (!warp_live || key0 > warp_pos_hi || key0 + SKM_KT - 1 < warp_first_lo) {
                 __syncthreads();
                 continue;
             }
@@ -762,7 +828,7 @@ __global__ void __launch_bounds__(SKM_THREADS) sink_attention_mma_kernel(const S
                 }
             }
             // ---- scores in log2 units, capped, masked; the tile's maximum per row
-            const bool need_mask = key0 + SKM_KT - 1 > warp_pos_lo || (p.window > 0 && key0 < warp_pos_hi - p.window + 1);
+            const bool need_mask = key0 + SKM_KT - 1 > warp_pos_lo || key0 < warp_first_hi;
             float tmax[2] = {-INFINITY, -INFINITY};
 #pragma unroll
             for (int nb = 0; nb < NKB; ++nb) {
@@ -844,7 +910,7 @@ __global__ void __launch_bounds__(SKM_THREADS) sink_attention_mma_kernel(const S
             if ((lane & 3) == 0) { p.part_ml[2 * r] = m_run[half] * LN2_F; p.part_ml[2 * r + 1] = l; }
             continue;
         }
-        const float sk2 = p.sink[head] * LOG2E_F;
+        const float sk2 = p.sink ? p.sink[head] * LOG2E_F : -INFINITY;
         const float M = fmaxf(m_run[half], sk2);
         const float f = ex2_(m_run[half] - M);
         const float inv = __fdividef(f, l * f + ex2_(sk2 - M));
@@ -873,10 +939,10 @@ MSGL_API int msgl_sink_attention_mma(const void* q, const void* k_cache, const v
                                      const int* block_table, int bt_stride, int uniform, int n_tiles, const float* sink, void* out,
                                      long long out_stride, float* part_o, float* part_ml, int splits, int split_keys, int T_, int B, int n_q,
                                      int n_kv, int d, int dv, int page_size, int window, float scale, float softcap, const void* gate,
-                                     long long gate_stride, cudaStream_t stream) {
+                                     long long gate_stride, int chunk_keys, cudaStream_t stream) {
     if (n_tiles <= 0) return MSGL_OK;
-    if (d <= 0 || dv <= 0 || d > 128 || dv > 128 || d % 8 || dv % 8 || n_kv <= 0 || n_q % n_kv || page_size < 1 || sink == nullptr ||
-        window < 0 || (out_stride & 1) || ((size_t)out & 3) || (gate_stride & 1) || ((size_t)gate & 3) || splits < 1 ||
+    if (d <= 0 || dv <= 0 || d > 128 || dv > 128 || d % 8 || dv % 8 || n_kv <= 0 || n_q % n_kv || page_size < 1 ||
+        window < 0 || chunk_keys < 0 || (window > 0 && chunk_keys > 0) || (out_stride & 1) || ((size_t)out & 3) || (gate_stride & 1) || ((size_t)gate & 3) || splits < 1 ||
         (splits > 1 && (!uniform || part_o == nullptr || part_ml == nullptr || split_keys < SKM_KT || split_keys % SKM_KT || ((size_t)part_o & 7))))
         return MSGL_ERR_SIZE;
     SinkAttnParams p;
@@ -884,7 +950,7 @@ MSGL_API int msgl_sink_attention_mma(const void* q, const void* k_cache, const v
     p.bt_stride = bt_stride; p.uniform = uniform; p.sink = sink; p.out = out; p.out_stride = out_stride; p.part_o = part_o;
     p.part_ml = part_ml; p.splits = splits; p.split_keys = split_keys; p.T = T_; p.B = B; p.n_q = n_q; p.n_kv = n_kv; p.d = d; p.dv = dv;
     p.page_size = page_size; p.QT = 0; p.GH = 0; p.window = window; p.scale = scale; p.softcap = softcap;
-    p.gate = gate; p.gate_stride = gate_stride;
+    p.gate = gate; p.gate_stride = gate_stride; p.chunk_keys = chunk_keys;
     const int G = n_q / n_kv;
     const dim3 grid(n_tiles, n_kv * (G <= SKM_R ? 1 : (G + SKM_R - 1) / SKM_R), splits);
 #define SKM_LAUNCH(DK, DV)                                                                                                   \

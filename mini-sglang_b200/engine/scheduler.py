@@ -156,7 +156,7 @@ class Scheduler:
         self.policy = policy
         self.retract_decode_steps = retract_decode_steps
         self.eos_ids = list(eos_ids)
-        can_share = len(self.mgr.groups) == 1 and self.mgr.groups[0].window is None and not self.mgr.state_ids
+        can_share = len(self.mgr.groups) == 1 and self.mgr.groups[0].span is None and not self.mgr.state_ids
         self.tree: Optional[PrefixTree] = PrefixTree(self.P) if (enable_prefix_cache and can_share) else None
         if policy == "lpm" and self.tree is None:
             self.policy = "fcfs"
@@ -206,9 +206,9 @@ class Scheduler:
     # -- accounting ------------------------------------------------------------------------
     def _hold(self, gi: int, n_tokens: float, portion: int = 1) -> float:
         """Tokens' worth of pages of group `gi` that a request of n_tokens holds at most: all of them, or for a
-        group that keeps a window the window plus the largest `portion` it is still fed in one step (pages
+        group that keeps a window (or a chunk) the window plus the largest `portion` it is still fed in one step (pages
         behind the window are given back) plus a page for the ragged ends."""
-        w = self.mgr.groups[gi].window
+        w = self.mgr.groups[gi].span
         if w is None:
             return n_tokens
         kept = self.mgr.groups[gi].keep_pages * self.P      # the first tokens' pages, which the window never gives back

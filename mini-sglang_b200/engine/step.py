@@ -26,7 +26,7 @@ import numpy as np
 import torch
 
 from .. import ops
-from ..cache import CacheManager, OutOfPages, PagedKVNeed, StateNeed
+from ..cache import CacheManager, OutOfPages, PagedKVNeed, StateNeed, keys_seen
 from ..config import ModelSpec, load_config
 from ..parts import BuildEnv, DecoderModel, GroupContext, KVCacheView, StateCacheView, StepContext, Workspace
 from ..weights import CheckpointSource, RandomSource
@@ -154,14 +154,14 @@ def _fewest_splits_as_fast(keys: int, ns: int, warps: int = DECODE_WARPS) -> int
 
 def plan_kv_splits(q_lens: Sequence[int], kv_lens: Sequence[int], *, n_kv: int, group: int, blocks_per_sm: int,
                    tile_tokens: int, window: Optional[int], cap: int, long_cap: Optional[int] = None,
-                   sm_count: int, warps: int = DECODE_WARPS) -> List[int]:
+                   sm_count: int, warps: int = DECODE_WARPS, chunk: Optional[int] = None) -> List[int]:
     """kv splits per request of one attention launch.  Only query runs that fit one tile of the decode kernel
     (`tile_tokens`) are split (the prefill kernels take whole key ranges).  Two reasons to split: the launch
     would otherwise leave most of the SMs idle (few requests: every request is cut alike), or one request is
     much longer than the launch's mean load per resident block, so that its single block would still run when
     all others are done (it is cut into pieces of about that load).  `cap` bounds the first kind of cut,
     `long_cap` (default: the same) the second.  `sm_count`: the device's number of SMs; `warps`: warps
-    of a block of the kernel that will run the launch."""
+    of a block of the kernel that will run the launch; `chunk`: keys are seen within chunks of that many positions."""
     long_cap = cap if long_cap is None else long_cap
     if cap <= 1 and long_cap <= 1:
         return [1] * len(q_lens)
@@ -170,7 +170,7 @@ def plan_kv_splits(q_lens: Sequence[int], kv_lens: Sequence[int], *, n_kv: int, 
     slots = sm_count * blocks_per_sm
     blocks = sum(-(-q // tile_tokens) for q in q_lens) * heads
     want = slots // max(blocks, 1)                    # fill the SMs once, not more
-    keys = [min(kv, window + q) if window else kv for q, kv in zip(q_lens, kv_lens)]
+    keys = [min(kv, window + q) if window else keys_seen(kv - q + 1, None, chunk) + q - 1 for q, kv in zip(q_lens, kv_lens)]
     load = sum(k for q, k in zip(q_lens, keys) if q <= tile_tokens) * heads / slots      # keys per resident block, dealt out evenly
     piece = max(MIN_KEYS_PER_PIECE, int(load * LONG_REQUEST_FACTOR))
     out = []
@@ -198,10 +198,10 @@ def plan_kv_splits(q_lens: Sequence[int], kv_lens: Sequence[int], *, n_kv: int, 
     return out
 
 
-def plan_even_cut(kv_lens: Sequence[int], window: Optional[int], n_blocks: int, max_pieces: int):
+def plan_even_cut(kv_lens: Sequence[int], window: Optional[int], n_blocks: int, max_pieces: int, chunk: Optional[int] = None):
     """The keys of a decode step (one new token a request) dealt out evenly over the blocks of one kv head.
 
-    The requests' units of DECODE_UNIT_KEYS keys (from the first unit a window still reaches to the unit of the newest
+    The requests' units of DECODE_UNIT_KEYS keys (from the first unit a window or a chunk still reaches to the unit of the newest
     key) are laid end to end and cut into at most `n_blocks` runs of equal length; a cut that falls within
     EVEN_SNAP_UNITS of a request's edge moves onto it.  No run is shorter than EVEN_MIN_UNITS unless the whole step is,
     and no request lies in more than `max_pieces` runs (fewer blocks are used if it would).
@@ -209,7 +209,7 @@ def plan_even_cut(kv_lens: Sequence[int], window: Optional[int], n_blocks: int, 
     -> (blocks in use n, start unit of every block [n + 1], first request of every block [n], first unit of every
     request [B + 1], first block of every request [B], pieces of every request [B]); int32 arrays."""
     pos = np.asarray(kv_lens, dtype=np.int64) - 1
-    k_lo = np.maximum(pos - window + 1, 0) if window else np.zeros_like(pos)
+    k_lo = np.maximum(pos - window + 1, 0) if window else (pos - pos % chunk if chunk else np.zeros_like(pos))
     units = pos // DECODE_UNIT_KEYS - k_lo // DECODE_UNIT_KEYS + 1
     B = len(units)
     cum = np.zeros(B + 1, dtype=np.int64)
@@ -254,13 +254,15 @@ def pack_even_cut(cut, B: int, n_blocks: int) -> np.ndarray:
     return out
 
 
-def decode_order(kv_lens, nsplits, window: Optional[int], b: int) -> np.ndarray:
+def decode_order(kv_lens, nsplits, window: Optional[int], b: int, chunk: Optional[int] = None) -> np.ndarray:
     """The rows of a decode batch in the order in which the attention launch takes them: by falling number of keys
     per kv split (blocks go to the SMs in index order, so the longest start first and the shortest fill the end);
     ties keep the rows' order, and the padding rows up to `b` come last."""
     keys = np.asarray(kv_lens, dtype=np.int64)
     if window:
         keys = np.minimum(keys, window + 1)
+    elif chunk:
+        keys = (keys - 1) % chunk + 1
     ns = np.maximum(np.asarray(nsplits, dtype=np.int64), 1)
     load = np.zeros(b, dtype=np.int64)
     load[:len(keys)] = -(-keys // ns)
@@ -439,7 +441,7 @@ class ModelRunner:
             per_sm, warps, qt = max(fused_blocks // self.sm_count, 1), self.FUSED_WARPS, 1
         return plan_kv_splits(q_lens, kv_lens, n_kv=n_kv, group=G, blocks_per_sm=per_sm, tile_tokens=qt,
                               window=self.mgr.groups[self._plan_group[gi]].window, cap=cap, long_cap=long_cap, sm_count=self.sm_count,
-                              warps=warps)
+                              warps=warps, chunk=self.mgr.groups[self._plan_group[gi]].chunk)
 
     def _fill(self, host: np.ndarray, lay: _Layout, entries: Sequence[StepEntry], starts: Sequence[int],
               want_rows: Sequence[int], nsplits: Sequence[Sequence[int]], pad_to: int = 0, even_cuts=None) -> None:
@@ -465,7 +467,7 @@ class ModelRunner:
                 mp = lay.max_pages[gi]
                 host[lay.out_loc[gi]: lay.out_loc[gi] + n_ent] = g.table[slots, pos // P].astype(np.int64) * P + pos % P
                 host[lay.nsplit[gi]: lay.nsplit[gi] + n_ent] = nsplits[gi]
-                host[lay.order[gi]: lay.order[gi] + B] = decode_order(pos + 1, nsplits[gi], g.window, B)
+                host[lay.order[gi]: lay.order[gi] + B] = decode_order(pos + 1, nsplits[gi], g.window, B, g.chunk)
                 if lay.even_nb[gi] and even_cuts is not None:
                     words = pack_even_cut(even_cuts[gi], B, lay.even_nb[gi])
                     host[lay.even[gi]: lay.even[gi] + len(words)] = words
@@ -512,7 +514,7 @@ class ModelRunner:
             groups.append(GroupContext(block_table=v(lay.table[gi], lay.B * mp).view(lay.B, mp),
                                        out_loc=v(lay.out_loc[gi], lay.T),
                                        nsplit=v(lay.nsplit[gi], lay.B) if max_splits[gi] > 1 else None,
-                                       max_split=max_splits[gi], window=g.window,
+                                       max_split=max_splits[gi], window=g.window, chunk=g.chunk,
                                        host_nsplit=nsplits[gi] if nsplits is not None else None,
                                        order=v(lay.order[gi], lay.B) if uniform else None,
                                        even=v(lay.even[gi], ops.even_cut_size(lay.B, lay.even_nb[gi])) if uniform and lay.even_nb[gi] else None,
@@ -660,7 +662,7 @@ class ModelRunner:
         if not fused and self._even_nb and self._wants_even_cut(kv_lens):
             # long contexts: the keys of all requests dealt out evenly over as many blocks as the SMs hold at once
             pieces = [min(EVEN_MAX_PIECES, nb) for nb in self._even_nb]
-            even_cuts = [plan_even_cut(kv_lens, g.window, nb, mx) for (_, g), nb, mx in zip(self._plans(), self._even_nb, pieces)]
+            even_cuts = [plan_even_cut(kv_lens, g.window, nb, mx, g.chunk) for (_, g), nb, mx in zip(self._plans(), self._even_nb, pieces)]
             nsplits = [c[5].tolist() for c in even_cuts]
             key = (b, mp, "even")
             gr = self._graphs.get(key)
@@ -704,7 +706,7 @@ class ModelRunner:
         if os.environ.get("MSGL_EVEN_CUT", "1") == "0":
             return False
         for g in self.mgr.groups:
-            units = [-(-(min(k, g.window + 1) if g.window else k) // DECODE_UNIT_KEYS) for k in kv_lens]
+            units = [-(-(min(k, g.window + 1) if g.window else keys_seen(k, None, getattr(g, "chunk", None))) // DECODE_UNIT_KEYS) for k in kv_lens]
             mean = sum(units) / len(units)
             if mean >= EVEN_FROM_UNITS and max(units) >= EVEN_UNEVEN * mean:
                 return True
@@ -765,6 +767,7 @@ class ModelRunner:
                             q_start=g0[lay.q_start:], kv_len=g0[lay.kv_len:], slots=g0[lay.slots:],
                             out_loc=g0[lay.out_loc[gi]:], nsplit=g0[lay.nsplit[gi]:], block_table=g0[lay.table[gi]:],
                             order=g0[lay.order[gi]:], window=int(self.mgr.groups[self._plan_group[gi]].window or 0),
+                            chunk=int(self.mgr.groups[self._plan_group[gi]].chunk or 0),
                             even_in=dev[e_off[gi]: e_off[gi] + n_even[gi]] if n_even[gi] else None,
                             even_out=g0[lay.even[gi]:] if n_even[gi] else None)
 

@@ -79,10 +79,10 @@ def _lib():
         lib.msgl_embedding.argtypes = [c_void_p, c_void_p, c_void_p, c_int, c_int, c_int, c_int, c_void_p]
         lib.msgl_resolve_ids.argtypes = [c_void_p, c_void_p, c_int, c_int, c_void_p]
         lib.msgl_table_delta.argtypes = [c_void_p, c_int, c_void_p, c_int, c_void_p]
-        lib.msgl_decode_meta.argtypes = [c_void_p] * 4 + [c_int, c_int, c_void_p, c_int, c_int, c_int, c_int] + [c_void_p] * 9 + [c_int, c_void_p, c_void_p, c_void_p, c_int,
+        lib.msgl_decode_meta.argtypes = [c_void_p] * 4 + [c_int, c_int, c_void_p, c_int, c_int, c_int, c_int] + [c_void_p] * 9 + [c_int, c_int, c_void_p, c_void_p, c_void_p, c_int,
                                          c_void_p]
         lib.msgl_rmsnorm.argtypes = [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int, c_float, c_int, c_void_p,
-                                     c_int, c_int, c_int, c_void_p]
+                                     c_int, c_int, c_int, c_void_p, c_void_p]
         lib.msgl_qknorm_rope_kvwrite.argtypes = [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_void_p, c_int,
                                                  c_float, c_void_p, c_int, c_int, c_void_p, c_void_p, c_void_p,
                                                  c_int, c_int, c_int, c_int, c_int, c_int, c_int, c_void_p]
@@ -109,11 +109,11 @@ def _attn_lib(head_dim: int):
     if lib is None:
         lib = _build.attention_library(hd)
         lib.msgl_attention.argtypes = [c_void_p] * 10 + [c_int] * 9 + [c_float] + [c_int] * 6 + [c_void_p, c_void_p, c_int, c_void_p, c_void_p,
-                                       c_ll, c_void_p]
+                                       c_ll, c_int, c_void_p]
         lib.msgl_attention_window.argtypes = [c_void_p] * 10 + [c_int] * 9 + [c_float] + [c_int] * 6 + [c_void_p, c_int, c_void_p, c_int, c_void_p]
         lib.msgl_attention_combine.argtypes = [c_void_p] * 5 + [c_int] * 5 + [c_void_p, c_void_p, c_ll, c_void_p]
         lib.msgl_attention_tc.argtypes = [c_void_p] * 7 + [c_int] * 8 + [c_float] + [c_int] * 5 + [c_void_p, c_int, c_void_p, c_int, c_void_p,
-                                         c_void_p, c_ll, c_void_p]
+                                         c_void_p, c_ll, c_int, c_void_p]
         lib.msgl_attention_head_dim.restype = c_int
         _attn[hd] = lib
     return lib
@@ -156,7 +156,7 @@ def table_delta(deltas: torch.Tensor, n_records: int, table: torch.Tensor) -> No
 
 def decode_meta(ids: torch.Tensor, slots_in: torch.Tensor, pos: torch.Tensor, nsplit_in: torch.Tensor, B: int, b: int,
                 table: torch.Tensor, page_size: int, mp: int, common: bool, *, input_ids, positions, token_req, q_start, kv_len,
-                slots, out_loc, nsplit, block_table, order, window: int = 0, even_in: Optional[torch.Tensor] = None,
+                slots, out_loc, nsplit, block_table, order, window: int = 0, chunk: int = 0, even_in: Optional[torch.Tensor] = None,
                 even_out: Optional[torch.Tensor] = None) -> None:
     """The step fields of a decode batch of B requests (captured size b) written on the device from (token id, slot,
     position) per request and the device copy of the block tables; see csrc/elementwise.cu.  `order` receives the rows
@@ -165,7 +165,7 @@ def decode_meta(ids: torch.Tensor, slots_in: torch.Tensor, pos: torch.Tensor, ns
     _need_cuda(ids, slots_in, pos, nsplit_in, table, input_ids, block_table)
     code = _lib().msgl_decode_meta(_ptr(ids), _ptr(slots_in), _ptr(pos), _ptr(nsplit_in), B, b, _ptr(table), table.shape[1], page_size,
                                    mp, int(common), _ptr(input_ids), _ptr(positions), _ptr(token_req), _ptr(q_start), _ptr(kv_len),
-                                   _ptr(slots), _ptr(out_loc), _ptr(nsplit), _ptr(block_table), int(window), _ptr(order),
+                                   _ptr(slots), _ptr(out_loc), _ptr(nsplit), _ptr(block_table), int(window), int(chunk), _ptr(order),
                                    _ptr(even_in), _ptr(even_out), even_in.numel() if even_in is not None else 0, _stream())
     _check(code, "decode_meta")
 
@@ -173,15 +173,16 @@ def decode_meta(ids: torch.Tensor, slots_in: torch.Tensor, pos: torch.Tensor, ns
 def rmsnorm(weight: torch.Tensor, eps: float, *, x: Optional[torch.Tensor] = None,
             residual: Optional[torch.Tensor] = None, residual_out: Optional[torch.Tensor] = None,
             rows: Optional[torch.Tensor] = None, out_dtype: Optional[torch.dtype] = None,
-            out: Optional[torch.Tensor] = None, center: bool = False) -> torch.Tensor:
+            out: Optional[torch.Tensor] = None, center: bool = False, bias: Optional[torch.Tensor] = None) -> torch.Tensor:
     """y = rmsnorm(residual + x) * weight, the sum and the norm in float32; with `center` the row's mean is taken off first
-    (a layer norm without bias: the variance is the mean of the squared deviations).
+    (a layer norm: the variance is the mean of the squared deviations).  bias (float32 [H] or None) is added last.
 
     x: float32 or activation dtype [N, H] or None; residual: float32 [N, H] or None; residual_out: float32
     buffer that receives the sum (may be `residual` itself when `rows` is None);
     rows: int32 [R] picks input rows (outputs are then [R, H]).  Returns y in `out_dtype`
     (default: x's dtype)."""
-    _need_cuda(weight, x, residual, residual_out, rows)
+    _need_cuda(weight, x, residual, residual_out, rows, bias)
+    assert bias is None or (bias.dtype == torch.float32 and bias.numel() == weight.numel() and bias.is_contiguous())
     src = x if x is not None else residual
     assert src is not None and src.dim() == 2 and src.is_contiguous()
     H = src.shape[1]
@@ -198,7 +199,7 @@ def rmsnorm(weight: torch.Tensor, eps: float, *, x: Optional[torch.Tensor] = Non
     x_f32 = int(x is not None and x.dtype == torch.float32)
     code = _lib().msgl_rmsnorm(_ptr(x), x_f32, _ptr(residual), _ptr(residual_out), _ptr(rows), _ptr(weight),
                                int(weight.dtype == torch.float32), float(eps), int(bool(center)), _ptr(out), n_out, H, _DT[out_dtype],
-                               _stream())
+                               _ptr(bias), _stream())
     _check(code, "layernorm" if center else "rmsnorm")
     return out
 
@@ -373,11 +374,11 @@ def attention_tc(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_ca
                  q_start: torch.Tensor, kv_len: torch.Tensor, block_table: torch.Tensor, n_kv: int, page_size: int,
                  window: int, scale: float, qlen_min: int, qlen_max: int, q_lens: Sequence[int], keep_first: int = 0,
                  bias_log2: Optional[torch.Tensor] = None, null_log2: Optional[torch.Tensor] = None,
-                 gate: Optional[torch.Tensor] = None) -> bool:
+                 gate: Optional[torch.Tensor] = None, chunk: int = 0) -> bool:
     """Prefill attention on tcgen05 tensor cores for the requests with q_len in [qlen_min, qlen_max];
     q_lens: the host's copy of every request's number of query tokens (to size the grid).  keep_first, bias_log2: as in
     `attention`; they are taken by the kernel on pairs of query tiles only (TMA page sizes), and the call returns False,
-    having launched nothing, where that kernel cannot run.  null_log2, gate: as in `attention`, taken by both kernels."""
+    having launched nothing, where that kernel cannot run.  null_log2, gate, chunk: as in `attention`, taken by both kernels."""
     global _tc2_usable
     gate_stride = _attention_extras(q, null_log2, gate)
     _need_cuda(q, out, k_cache, v_cache, q_start, kv_len, block_table)
@@ -406,7 +407,7 @@ def attention_tc(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_ca
             _ptr(q), _ptr(out), _ptr(k_cache), _ptr(v_cache), _ptr(q_start), _ptr(kv_len), _ptr(block_table), B, T, n_q,
             n_kv, d, page_size, block_table.stride(0), window, float(scale), qlen_min, qlen_max, grid_x, pages, version,
             _ptr(status), int(keep_first), _ptr(bias_log2), bias_log2.shape[1] if bias_log2 is not None else 0, _ptr(null_log2), _ptr(gate),
-            gate_stride, _stream())
+            gate_stride, int(chunk), _stream())
         if code == 2 and version == 2:        # no tensor maps here (driver without the encoder, unaligned cache): one-tile kernel
             _tc2_usable = False
             if ext:
@@ -481,7 +482,7 @@ def attention(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_cache
               uniform_decode: bool, variant: int, grid_x: int, order: Optional[torch.Tensor] = None,
               even: Optional[torch.Tensor] = None, even_nb: int = 0, keep_first: int = 0,
               bias_log2: Optional[torch.Tensor] = None, null_log2: Optional[torch.Tensor] = None,
-              gate: Optional[torch.Tensor] = None) -> None:
+              gate: Optional[torch.Tensor] = None, chunk: int = 0) -> None:
     """One launch of the paged attention kernel over the requests whose q_len lies in
     [qlen_min, qlen_max]; see csrc/attention.cu for the meaning of every argument.  keep_first: with a window, the first
     keys of a request that stay visible whatever the window; bias_log2: float32 [heads, L], added to the scaled score in
@@ -490,7 +491,8 @@ def attention(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_cache
     of a decode step's keys over `even_nb` blocks per kv head (engine/step.py: plan_even_cut) in place of `grid_x` blocks.
     null_log2: float32 [heads], the score in log2 units of one more term in every softmax's denominator that has no key and no
     value; gate [T, heads * d] (a view into packed rows): the output times sigmoid(gate), element by element.  Both enter where a
-    row is normalised, so a launch whose requests are cut hands them to `attention_combine` too."""
+    row is normalised, so a launch whose requests are cut hands them to `attention_combine` too.  chunk > 0 (with window 0): a query sees
+    the keys of its own chunk of `chunk` positions only, counted from the start of the sequence."""
     gate_stride = _attention_extras(q, null_log2, gate)
     _need_cuda(q, out, k_cache, v_cache, q_start, kv_len, block_table, nsplit, part_o, part_ml, order, even)
     T, n_q, d = q.shape
@@ -506,7 +508,7 @@ def attention(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_cache
     if keep_first or bias_log2 is not None:
         _need_cuda(bias_log2)
         assert even is None, "the even cut of a decode step knows no kept tokens and no bias"
-        assert null_log2 is None and gate is None, "a launch with kept tokens or a bias takes no further term and no gate"
+        assert null_log2 is None and gate is None and not chunk, "a launch with kept tokens or a bias takes no further term, gate or chunk"
         if bias_log2 is not None:
             assert bias_log2.dtype == torch.float32 and bias_log2.dim() == 2 and bias_log2.shape[0] == n_q and bias_log2.is_contiguous()
         code = _attn_lib(d).msgl_attention_window(
@@ -520,7 +522,7 @@ def attention(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_cache
         _ptr(q), _ptr(out), _ptr(k_cache), _ptr(v_cache), _ptr(q_start), _ptr(kv_len), _ptr(block_table),
         _ptr(nsplit), _ptr(part_o), _ptr(part_ml), B, T, n_q, n_kv, d, page_size, block_table.stride(0), window,
         max_split, float(scale), qlen_min, qlen_max, int(uniform_decode), variant, grid_x, _dt(q), _ptr(order), _ptr(even), int(even_nb),
-        _ptr(null_log2), _ptr(gate), gate_stride, _stream())
+        _ptr(null_log2), _ptr(gate), gate_stride, int(chunk), _stream())
     _check(code, f"attention (head size {d}, variant {variant})")
 
 
@@ -1554,11 +1556,11 @@ def _delta_lib():
         lib.msgl_scaled_add_norm.argtypes = [c_void_p, c_int, c_void_p, c_void_p, c_void_p, c_float, c_void_p, c_int, c_int, c_int, c_void_p]
         lib.msgl_rotary_angles.argtypes = [c_void_p, c_void_p, ctypes.c_double, c_void_p, c_int, c_int, c_void_p]
         lib.msgl_sink_qkv_prep.argtypes = [c_void_p, c_ll, c_void_p, c_int, c_void_p, c_ll, c_float] + [c_void_p] * 4 + [c_int] * 7 + \
-            [c_void_p, c_void_p, c_int, c_float, c_void_p]
+            [c_void_p, c_void_p, c_int, c_float, c_int, c_int, c_int, c_void_p]
         lib.msgl_sink_attention.argtypes = [c_void_p] * 6 + [c_int, c_int, c_int, c_void_p, c_void_p, c_ll, c_void_p, c_void_p] + \
-            [c_int] * 12 + [c_float, c_float, c_int, c_void_p, c_ll, c_void_p]
+            [c_int] * 12 + [c_float, c_float, c_int, c_void_p, c_ll, c_int, c_void_p]
         lib.msgl_sink_attention_mma.argtypes = [c_void_p] * 6 + [c_int, c_int, c_int, c_void_p, c_void_p, c_ll, c_void_p, c_void_p] + \
-            [c_int] * 10 + [c_float, c_float, c_void_p, c_ll, c_void_p]
+            [c_int] * 10 + [c_float, c_float, c_void_p, c_ll, c_int, c_void_p]
         lib.msgl_delta_rule.argtypes = [c_void_p, c_void_p, c_ll, c_int, c_int] + [c_void_p] * 7 + [c_int] * 7 + [c_void_p]
         lib.msgl_delta_rule_scratch.argtypes = [c_int] * 4
         lib.msgl_delta_rule_scratch.restype = c_ll
@@ -1599,15 +1601,20 @@ def rotary_angles(positions: torch.Tensor, freq: torch.Tensor, magnitude: float,
 def sink_qkv_prep(proj: torch.Tensor, *, n_q: int, n_kv: int, d: int, dv: int, angles: Optional[torch.Tensor],
                   v_first: Optional[torch.Tensor], lam: float, out_loc: Optional[torch.Tensor], k_cache: Optional[torch.Tensor],
                   v_cache: Optional[torch.Tensor], page_size: int, q_norm: Optional[torch.Tensor] = None,
-                  k_norm: Optional[torch.Tensor] = None, v_unit: bool = False, eps: float = 0.0) -> torch.Tensor:
+                  k_norm: Optional[torch.Tensor] = None, v_unit: bool = False, eps: float = 0.0, interleaved: bool = False,
+                  qk_unit: bool = False, maps: int = 1) -> torch.Tensor:
     """proj [T, >= n_q * d + n_kv * d + n_kv * dv] packed rows [q | k | v | ...].  Where weights are given (q_norm, k_norm float32
     [d], one for all heads) every q and k head is RMS-normed by itself first; the first angles.shape[1] elements of every q and
-    k head turn in halves (element i against i + rot / 2) by `angles` float32 [T, rot] = cos | sin of the tokens' positions; v
+    k head turn in halves (element i against i + rot / 2), or with `interleaved` in neighbouring pairs, by `angles` float32 [T, rot]
+    = cos | sin of the tokens' positions; with qk_unit every q and k head is then divided by its root mean square; v
     becomes (1 - lam) v + lam v_first where `v_first` [T, n_kv * dv] (a view into packed rows) is given, and with
-    v_unit every v head is then divided by its root mean square (eps inside the root); k goes to `k_cache` [pages, n_kv, page, d] and v to `v_cache` [pages, n_kv, page, dv] at token slots `out_loc`; the q rows come back as [T, n_q, d]."""
+    v_unit every v head is then divided by its root mean square (eps inside the root); k goes to `k_cache` [pages, n_kv, page, d] and v to `v_cache` [pages, n_kv, page, dv] at token slots `out_loc`; the q rows come back as [T, n_q, d].
+    maps = M > 1: every q and kv head has M vectors of d elements (proj [n_q * M * d | n_kv * M * d | n_kv * dv | ...]), each treated
+    as a head of its own; `k_cache` rows are M * d long, and q comes back as [T, n_q * M, M * d], vector (h, m) in place m of its
+    row and zeros in the others.  Without a cache the packed rows need hold q only."""
     _need_cuda(proj, angles, v_first, out_loc, k_cache, v_cache)
     T = proj.shape[0]
-    width = (n_q + n_kv) * d + n_kv * dv
+    width = n_q * maps * d + (n_kv * (maps * d + dv) if k_cache is not None else 0)
     stride = _rows_view(proj, proj.shape[1], "proj")
     assert proj.shape[1] >= width
     rot = 0
@@ -1620,17 +1627,17 @@ def sink_qkv_prep(proj: torch.Tensor, *, n_q: int, n_kv: int, d: int, dv: int, a
         vf_stride = _rows_view(v_first, n_kv * dv, "v_first")
     if k_cache is not None:
         assert k_cache.dtype == proj.dtype and v_cache.dtype == proj.dtype and k_cache.is_contiguous() and v_cache.is_contiguous()
-        assert tuple(k_cache.shape[1:]) == (n_kv, page_size, d) and tuple(v_cache.shape[1:]) == (n_kv, page_size, dv)
+        assert tuple(k_cache.shape[1:]) == (n_kv, page_size, maps * d) and tuple(v_cache.shape[1:]) == (n_kv, page_size, dv)
         assert out_loc is not None and out_loc.dtype == torch.int32 and out_loc.numel() >= T
     assert (q_norm is None) == (k_norm is None)
     if q_norm is not None:
         assert q_norm.dtype == k_norm.dtype == torch.float32 and q_norm.numel() == k_norm.numel() == d
         assert q_norm.is_contiguous() and k_norm.is_contiguous()
         _need_cuda(q_norm, k_norm)
-    q_out = torch.empty((T, n_q, d), dtype=proj.dtype, device=proj.device)
+    q_out = torch.empty((T, n_q * maps, maps * d), dtype=proj.dtype, device=proj.device)
     code = _delta_lib().msgl_sink_qkv_prep(_ptr(proj), stride, _ptr(angles), rot, _ptr(v_first), vf_stride, float(lam), _ptr(out_loc),
                                            _ptr(q_out), _ptr(k_cache), _ptr(v_cache), page_size, n_q, n_kv, d, dv, T, _dt(proj), _ptr(q_norm), _ptr(k_norm),
-                                           int(bool(v_unit)), float(eps), _stream())
+                                           int(bool(v_unit)), float(eps), int(bool(interleaved)), int(bool(qk_unit)), int(maps), _stream())
     _check(code, "sink_qkv_prep")
     return q_out
 
@@ -1651,21 +1658,22 @@ def sink_attention_on_tensor_cores(dtype: torch.dtype, d: int, dv: int) -> bool:
     return dtype == torch.bfloat16 and d % 8 == 0 and dv % 8 == 0 and max(d, dv) <= SINK_ATTENTION_MMA_MAX_HEAD_DIM
 
 
-def sink_attention_splits(table_width: int, page_size: int, window: int) -> int:
-    """Pieces a one-token step cuts a request's keys into: as many as the block table's width asks for, or as a window touches."""
+def sink_attention_splits(table_width: int, page_size: int, window: int, chunk: int = 0) -> int:
+    """Pieces a one-token step cuts a request's keys into: as many as the block table's width asks for, or as a window or a chunk
+    touches."""
     splits = max(1, -(-(table_width * page_size) // SINK_ATTENTION_SPLIT_KEYS))
-    if window > 0:
-        splits = min(splits, (window - 1) // SINK_ATTENTION_SPLIT_KEYS + 2)
+    if window > 0 or chunk > 0:
+        splits = min(splits, ((window or chunk) - 1) // SINK_ATTENTION_SPLIT_KEYS + 2)
     return splits
 
 
 def sink_attention(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_cache: torch.Tensor, *, q_start: torch.Tensor,
                    kv_len: torch.Tensor, block_table: torch.Tensor, n_kv: int, page_size: int, scale: float, softcap: float,
-                   window: int, sink: torch.Tensor, q_lens: Optional[Sequence[int]], workspace=None,
-                   tensor_cores: Optional[bool] = None, gate: Optional[torch.Tensor] = None) -> None:
+                   window: int, sink: Optional[torch.Tensor], q_lens: Optional[Sequence[int]], workspace=None,
+                   tensor_cores: Optional[bool] = None, gate: Optional[torch.Tensor] = None, chunk: int = 0) -> None:
     """Causal softmax attention over the paged cache: the query at position i sees the keys j <= i with i - j < window (window 0:
-    all), score = q . k * scale, capped as softcap * tanh(score / softcap) where softcap > 0, and every softmax's denominator
-    holds exp(sink[head]) besides the seen keys' terms.  q [T, heads, d]; K cache [pages, n_kv, page, d], V cache [pages, n_kv,
+    all; or, with chunk > 0 and window 0, the keys j <= i of its own chunk, j // chunk == i // chunk), score = q . k * scale, capped as softcap * tanh(score / softcap) where softcap > 0, and every softmax's denominator
+    holds exp(sink[head]) besides the seen keys' terms (sink None: it does not).  q [T, heads, d]; K cache [pages, n_kv, page, d], V cache [pages, n_kv,
     page, dv]; sink float32 [heads]; out [T, heads * dv].  q_lens: the requests' numbers of tokens as the host knows them (they
     size the launch), or None when every request brings one token: the keys are then cut into pieces of
     SINK_ATTENTION_SPLIT_KEYS for blocks of their own, joined in order by a second kernel (workspace: a parts.Workspace for
@@ -1676,7 +1684,7 @@ def sink_attention(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_
     T, n_q, d = q.shape
     dv = v_cache.shape[3]
     assert q.is_contiguous() and k_cache.dtype == q.dtype and v_cache.dtype == q.dtype and out.dtype == q.dtype
-    assert sink.dtype == torch.float32 and sink.numel() == n_q
+    assert sink is None or (sink.dtype == torch.float32 and sink.numel() == n_q)
     out_stride = _rows_view(out, n_q * dv, "out")
     gate_stride = 0
     if gate is not None:
@@ -1691,7 +1699,7 @@ def sink_attention(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_
     n_tiles = B if uniform else sum(-(-n // QT) for n in q_lens)
     splits, part_o, part_ml = 1, None, None
     if uniform:
-        splits = sink_attention_splits(block_table.shape[1], page_size, int(window))
+        splits = sink_attention_splits(block_table.shape[1], page_size, int(window), int(chunk))
         if splits > 1:
             rows = splits * T * n_q
             if workspace is not None:
@@ -1703,12 +1711,12 @@ def sink_attention(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_
         code = _delta_lib().msgl_sink_attention_mma(
             _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(q_start), _ptr(kv_len), _ptr(block_table), block_table.stride(0), int(uniform),
             n_tiles, _ptr(sink), _ptr(out), out_stride, _ptr(part_o), _ptr(part_ml), splits, SINK_ATTENTION_SPLIT_KEYS, T, B, n_q, n_kv, d,
-            dv, page_size, int(window), float(scale), float(softcap), _ptr(gate), gate_stride, _stream())
+            dv, page_size, int(window), float(scale), float(softcap), _ptr(gate), gate_stride, int(chunk), _stream())
     else:
         code = _delta_lib().msgl_sink_attention(
             _ptr(q), _ptr(k_cache), _ptr(v_cache), _ptr(q_start), _ptr(kv_len), _ptr(block_table), block_table.stride(0), int(uniform),
             n_tiles, _ptr(sink), _ptr(out), out_stride, _ptr(part_o), _ptr(part_ml), splits, SINK_ATTENTION_SPLIT_KEYS, T, B, n_q, n_kv, d,
-            dv, page_size, QT, GH, int(window), float(scale), float(softcap), _dt(q), _ptr(gate), gate_stride, _stream())
+            dv, page_size, QT, GH, int(window), float(scale), float(softcap), _dt(q), _ptr(gate), gate_stride, int(chunk), _stream())
     _check(code, f"sink_attention (head sizes {d}, {dv})")
     if splits > 1:
         global LAUNCHES
@@ -1755,6 +1763,64 @@ def side_gate_mul(gate: torch.Tensor, table: torch.Tensor, ids: torch.Tensor, of
                                            table.shape[0], _ptr(out), dim, T, _dt(gate), _stream())
     _check(code, "side_gate_mul")
     return out
+
+
+# ---------------------------------------------------------------------------------------
+# several copies of the residual stream, heads that are the difference of two maps (csrc/mixers_streams.cu)
+# ---------------------------------------------------------------------------------------
+_streams = None
+MAX_STREAMS = 32
+
+
+def _streams_lib():
+    global _streams
+    if _streams is None:
+        lib = _build.stream_mixers_library()
+        lib.msgl_stream_mix_norm.argtypes = [c_void_p, c_ll, c_ll, c_void_p, c_void_p, c_int] + [c_void_p] * 5 + [c_float, c_int, c_void_p, c_void_p] + \
+            [c_int] * 4 + [c_void_p]
+        lib.msgl_map_difference.argtypes = [c_void_p, c_int, c_void_p, c_ll, c_float, c_float, c_float, c_int, c_int, c_int, c_int, c_void_p]
+        _streams = lib
+    return _streams
+
+
+def stream_mix_norm(x: torch.Tensor, *, streams: int, weight: torch.Tensor, bias: Optional[torch.Tensor], eps: float, center: bool,
+                    w_in: Optional[torch.Tensor], y: Optional[torch.Tensor] = None, mix: Optional[torch.Tensor] = None,
+                    w_out: Optional[torch.Tensor] = None, x_out: Optional[torch.Tensor] = None, rows: Optional[torch.Tensor] = None,
+                    out_dtype: torch.dtype = torch.float32) -> torch.Tensor:
+    """S copies of the stream: x float32 [T, S, H], or [T, H] where all copies are still the same row.  With `y` [T, H] (what a
+    sublayer hands over) every copy becomes sum_s mix[s][t] x_s + w_out[t] y (mix [S, S] from s to t, w_out [S]; float32), all from
+    the old ones, and goes to `x_out` [T, S, H] where it is given (may be x).  -> norm(sum_t w_in[t] x_t) * weight (+ bias) in
+    `out_dtype`, w_in float32 [S] (None: ones); center: a layer norm, else an RMS norm.  rows (int32): the rows that are normed
+    (nothing is written to the copies then)."""
+    _need_cuda(x, weight, bias, w_in, y, mix, w_out, x_out, rows)
+    S, H = streams, x.shape[-1]
+    T = x.shape[0]
+    assert x.dtype == torch.float32 and x.is_contiguous() and (x.dim() == 2 or x.shape[1] == S)
+    assert weight.dtype == torch.float32 and weight.numel() == H and (bias is None or (bias.dtype == torch.float32 and bias.numel() == H))
+    for t, n in ((w_in, S), (mix, S * S), (w_out, S)):
+        assert t is None or (t.dtype == torch.float32 and t.numel() == n and t.is_contiguous())
+    if y is not None:
+        assert y.shape == (T, H) and y.is_contiguous() and y.dtype in (out_dtype, torch.float32)
+    assert x_out is None or (x_out.shape == (T, S, H) and x_out.is_contiguous() and x_out.dtype == torch.float32)
+    n = T if rows is None else rows.numel()
+    out = torch.empty((n, H), dtype=out_dtype, device=x.device)
+    code = _streams_lib().msgl_stream_mix_norm(_ptr(x), H * (S if x.dim() == 3 else 1), H if x.dim() == 3 else 0, _ptr(x_out), _ptr(y),
+                                               int(y is not None and y.dtype == torch.float32), _ptr(mix), _ptr(w_out), _ptr(w_in), _ptr(weight),
+                                               _ptr(bias), float(eps), int(bool(center)), _ptr(rows), _ptr(out), n, S, H, _DT[out_dtype], _stream())
+    _check(code, f"stream_mix_norm ({S} streams, width {H})")
+    return out
+
+
+def map_difference(a: torch.Tensor, out: torch.Tensor, *, heads: int, lam: float, eps: float, scale: float) -> None:
+    """a [T, heads * 2, dv] (a head's two maps side by side), out [T, heads * dv]: with v = a_1 - lam a_2 per head,
+    out = v / sqrt(mean(v^2) + eps) * scale, in float32."""
+    _need_cuda(a, out)
+    T, dv = a.shape[0], a.shape[2]
+    assert a.is_contiguous() and a.shape[1] == 2 * heads and a.dtype in (out.dtype, torch.float32)
+    o_stride = _rows_view(out, heads * dv, "out")
+    code = _streams_lib().msgl_map_difference(_ptr(a), int(a.dtype == torch.float32), _ptr(out), o_stride, float(lam), float(eps), float(scale),
+                                              T, heads, dv, _dt(out), _stream())
+    _check(code, f"map_difference (value size {dv})")
 
 
 # ---------------------------------------------------------------------------------------

@@ -106,17 +106,20 @@ class PagedAttention(Mixer):
 
 def paged_attend(q: torch.Tensor, out: torch.Tensor, ctx: StepContext, cache: KVCacheView, *, n_q: int, n_kv: int, d: int,
                  window: int, scale: float, use_mma: bool, keep_first: int = 0, bias_log2: Optional[torch.Tensor] = None,
-                 null_log2: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None) -> None:
+                 null_log2: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, chunk: int = 0) -> None:
     """The attention launches of one step over a paged cache: requests that bring a few tokens through the decode kernel
     with the step's kv splits, longer runs through the prefill kernels, the merge of the splits.  keep_first and bias_log2
     (kept first tokens under a window, a bias by distance: `ops.attention`) are for mixers that have them; such launches
     run on the tcgen05 prefill kernel on pairs of query tiles where it applies and on the mma kernels otherwise.  null_log2
-    (a term in every softmax's denominator that has no key) and gate (sigmoids on the output): `ops.attention`."""
+    (a term in every softmax's denominator that has no key), gate (sigmoids on the output) and chunk (keys are seen within chunks
+    of the sequence only): `ops.attention`."""
     plain = keep_first == 0 and bias_log2 is None
     if not plain and not use_mma:
         raise ValueError("kept first tokens and a distance bias are taken by the bfloat16 mma kernels only")
     joined = {} if null_log2 is None and gate is None else dict(null_log2=null_log2, gate=gate)
-    extra = dict(joined) if plain else dict(keep_first=keep_first, bias_log2=bias_log2, **joined)
+    if chunk and not plain:
+        raise ValueError("a chunk goes with neither kept first tokens nor a distance bias")
+    extra = dict(joined, chunk=chunk) if plain else dict(keep_first=keep_first, bias_log2=bias_log2, **joined)
     g = cache.group
     G = n_q // n_kv
     max_split = g.max_split if g.nsplit is not None else 1

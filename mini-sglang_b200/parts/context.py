@@ -21,6 +21,7 @@ class GroupContext:
     nsplit: Optional[torch.Tensor]     # [B] int32, kv splits per request (None: 1)
     max_split: int
     window: Optional[int]
+    chunk: Optional[int] = None        # without a window: keys are seen within chunks of this many positions
     host_nsplit: Optional[Sequence[int]] = None     # the host's copy of nsplit (None: not known here)
     order: Optional[torch.Tensor] = None            # [B] int32, uniform decode only: the requests by falling number of keys
     even: Optional[torch.Tensor] = None             # int32, uniform decode only: the keys dealt out evenly over even_nb blocks

@@ -99,7 +99,7 @@ class FusedDecodeStep:
 
     def takes(self, ctx: StepContext) -> bool:
         return (ctx.uniform_decode and ctx.all_rows_wanted and 0 < ctx.B <= ops.FUSED_DECODE_MAX_TOKENS
-                and len(ctx.groups) == 1 and ctx.groups[0].window is None and self.blocks_for(ctx.B) > 0)
+                and len(ctx.groups) == 1 and ctx.groups[0].window is None and ctx.groups[0].chunk is None and self.blocks_for(ctx.B) > 0)
 
     def _layers_on_device(self, caches: Dict[int, object]) -> torch.Tensor:
         runs = self.model.schedule

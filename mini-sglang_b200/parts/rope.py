@@ -45,7 +45,8 @@ class RotaryNeox(PositionEncoding):
 
 @register_position_encoding("rope_yarn")
 class RotaryYarn(PositionEncoding):
-    """Rotary position encoding in halves (element i against i + rotary_dim / 2) with YaRN's frequency scaling.
+    """Rotary position encoding in halves (element i against i + rotary_dim / 2), or with `interleaved` in neighbouring pairs
+    (2 i against 2 i + 1), with YaRN's frequency scaling.
 
     Pair i of n = rotary_dim / 2 turns with frequency f_i = theta^(-i / n).  `scaling` = {factor, original, fast, slow} slows the
     pairs whose wavelength is long against a context of `original` tokens: a pair that makes t turns within `original` tokens
@@ -57,13 +58,14 @@ class RotaryYarn(PositionEncoding):
     The frequencies are made on the host in double precision and kept as float32 (`inv_freq`); kernels that make their angles
     themselves (position * frequency in float32) read them and have no position limit; `rotary_table()` gives the same angles
     as a table of `max_positions` rows for kernels that look them up.
-    params: rotary_dim, theta, scaling (or None), max_positions."""
+    params: rotary_dim, theta, scaling (or None), interleaved, max_positions."""
 
     def __init__(self, spec, prefix, env):
         super().__init__(spec, prefix, env)
         self.rotary_dim = int(spec["rotary_dim"])
         self.theta = float(spec["theta"])
         self.scaling = dict(spec["scaling"]) if spec.get("scaling") else None
+        self.interleaved = bool(spec.get("interleaved", False))
         self.max_positions = int(spec.get("max_positions", 0))
         if self.rotary_dim % 2 or self.rotary_dim < 0:
             raise ValueError("rotary_dim must be even")
