@@ -637,6 +637,35 @@ def pokatar_config(size, layers, vocab):
     return {"architecture": "Pokatar", "width": s["width"], "vocab": vocab, "norm": {"eps": 1e-5}, "layers": [kinds[i % 4] for i in range(layers)]}
 
 
+def rubulix_config(size, layers, vocab, chunk=1024, streams=4):
+    """A Rubulix model with the given layer sizes and four copies of the stream.  The attention within chunks has the heads of the
+    Qwen3 layer (key and value size of the head, chunks of 1,024 tokens); the differential attention as many heads whose two
+    maps have half the key size each, so that keys, values and projections are as large as the Qwen3 layer's; dense
+    feed-forwards of the layer's width.  Kinds of layers in turn: chunked, chunked, differential, differential on the keys and
+    values of the layer before it."""
+    s = COMPARE_SIZES[size]
+    base = {"heads": s["heads"], "kv_heads": s["kv_heads"], "vdim": s["dim"]}
+    chunked = {"type": "attention_2", "mixer": dict(base, dim=s["dim"], scale=s["dim"] ** -0.5, mask={"size": chunk},
+                                                    rot={"base": 500000.0, "dims": s["dim"]})}
+    diff = {"type": "attention", "mixer": dict(base, dim=s["dim"] // 2, scale=(s["dim"] // 2) ** -0.5, diff=0.5,
+                                               rot={"base": 10000.0, "dims": s["dim"] // 2,
+                                                    "scaling": {"factor": 4.0, "original": 4096, "fast": 32.0, "slow": 1.0}})}
+    out = []
+    for i in range(layers):
+        l = chunked if i % 4 < 2 else diff
+        l = dict(l, mixer=dict(l["mixer"]), mlp={"kind": "dense", "ff": s["ff"]})
+        if i % 4 == 3:
+            l["mixer"]["kv_from"] = i - 1
+        out.append(l)
+    return {"architecture": "Rubulix", "width": s["width"], "vocab": vocab, "streams": streams, "norm": {"eps": 1e-5}, "layers": out}
+
+
+def workload_rubulix(args):
+    """As --workload vekurax_compare, with a Rubulix model (`rubulix_config`) beside the Pokatar model (the engine's other design
+    with layer norms and a gated attention on the paged kernels) and the Qwen3 model of equal sizes."""
+    return workload_vekurax(args, name="rubulix", config=rubulix_config, beside=("pokatar", "qwen3"))
+
+
 def workload_pokatar(args):
     """As --workload vekurax_compare, with a Pokatar model (`pokatar_config`) beside the Lifulorn model (the engine's other design
     with an attention with a term in the denominator and routed experts beside a shared one), the Nametar model (its other latent
@@ -689,7 +718,7 @@ def workload_vekurax(args, name="vekurax", config=None, beside="qwen3"):
                     tie_word_embeddings=True, max_position_embeddings=CTX + 4096)
         res = {}
         others = {"qwen3": lambda: qwen, "vekurax": lambda: vekurax_config(size, L, V), "pepevik": lambda: pepevik_config(size, L, V),
-                  "lifulorn": lambda: lifulorn_config(size, L, V), "nametar": lambda: nametar_config(size, L, V)}
+                  "lifulorn": lambda: lifulorn_config(size, L, V), "nametar": lambda: nametar_config(size, L, V), "pokatar": lambda: pokatar_config(size, L, V)}
         archs = [(name, config(size, L, V))]
         if not args.alone:
             archs += [(b, others[b]()) for b in ((beside,) if isinstance(beside, str) else beside)]
@@ -769,9 +798,9 @@ def main():
                     help="cudaProfilerStart/Stop around the timed region (ncu --profile-from-start off)")
     ap.add_argument("--no-graph", action="store_true", help="decode without CUDA graphs")
     ap.add_argument("--workload", default="headline", choices=["headline", "qwen3_0.6b_mixed", "qwen3_32b_long", "sweep", "vekurax_compare", "nametar_compare", "pepevik_compare",
-                                                              "lifulorn_compare", "pokatar_compare"],
+                                                              "lifulorn_compare", "pokatar_compare", "rubulix_compare"],
                     help="headline: the default line; the others: further workloads, one JSON line each")
-    ap.add_argument("--sizes", default=None, help="--workload vekurax_compare / nametar_compare / pepevik_compare / lifulorn_compare / pokatar_compare: layer sizes to run, of " + ",".join(COMPARE_SIZES))
+    ap.add_argument("--sizes", default=None, help="--workload vekurax_compare / nametar_compare / pepevik_compare / lifulorn_compare / pokatar_compare / rubulix_compare: layer sizes to run, of " + ",".join(COMPARE_SIZES))
     ap.add_argument("--alone", action="store_true", help="the compare workloads: run the named design only, not the one beside it")
     ap.add_argument("--skip-sanity", action="store_true", help="no comparison with the plain implementation before timing")
     ap.add_argument("--model", default="8b", choices=["8b", "32b", "0.6b"], help="layer sizes for --only decode / prefill")
@@ -802,6 +831,8 @@ def main():
         return workload_lifulorn(args)
     if args.workload == "pokatar_compare":
         return workload_pokatar(args)
+    if args.workload == "rubulix_compare":
+        return workload_rubulix(args)
 
     import torch
 

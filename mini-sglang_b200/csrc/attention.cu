@@ -28,7 +28,7 @@
 //   attn_decode_kernel<D,...>   the same for head sizes 16 mod 32: heads on the M dimension
 //   attn_simt_kernel<T>         any head size up to 512, float32 arithmetic throughout; this is
 //                               the true 32-bit path and the fallback for odd head sizes
-//   attn_combine_kernel<T>      merge of the kv splits
+//   attn_combine_kernel<T>      merge of the kv splits; attn_combine_diff_kernel<T> for heads that are the difference of two maps
 // Scores, softmax and the accumulation are float32 in all of them.  In a step of single tokens the blocks take the
 // requests in the order the step gives (`order`: longest first), the kv heads of one request in adjacent blocks.
 #include "common.cuh"
@@ -85,6 +85,11 @@ struct AttnParams {
     // sigmoid(gate), element by element (likewise where a row is normalised)
     const void* gate = nullptr;
     long long gate_stride = 0;
+    // heads that are the difference of two maps: query heads 2 h and 2 h + 1 are the maps of output head h, whose row
+    // ([T, n_q / 2, d]) is v / sqrt(mean(v^2) + diff_eps) * diff_scale with v = o_2h - diff_lam o_2h+1.  Kernels of short query
+    // runs always leave partial results then, and the merge takes the difference.
+    int diff = 0;
+    float diff_lam = 0.f, diff_eps = 0.f, diff_scale = 0.f;
 };
 
 // weight of the term without a key against the reference m (log2 units) of a row's exponentials
@@ -98,7 +103,7 @@ __device__ __forceinline__ float gate_factor(const void* gate, long long gate_st
 }
 __device__ __forceinline__ float2 gate_pair(unsigned g) {              // two neighbouring bfloat16 gates -> their sigmoids
     const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&g));
-    return make_float2(1.f / (1.f + __expf(-f.x)), 1.f / (1.f + __expf(-f.y)));
+    return make_float2(__fdividef(1.f, 1.f + __expf(-f.x)), __fdividef(1.f, 1.f + __expf(-f.y)));      // (beyond 2^126: 0)
 }
 
 // position -> (page index within the request, slot within the page)
@@ -512,7 +517,37 @@ __global__ void __launch_bounds__(MMA_THREADS) attn_mma_kernel(const AttnParams 
     __nv_bfloat16* og = reinterpret_cast<__nv_bfloat16*>(p.out);
     const bool direct = ns == 1;
 
-    {
+    if (direct && p.diff) {
+        // the rows of a head's two maps are neighbours (the group size is even): they sit in lanes that differ in bit 2
+#pragma unroll
+        for (int half = 0; half < 2; ++half) {
+            const float l = half ? l_hi : l_lo;
+            const float inv = l > 0.f ? 1.f / l : 0.f;
+            float ss = 0.f;
+#pragma unroll
+            for (int nd = 0; nd < NDB; ++nd) {
+#pragma unroll
+                for (int e = 0; e < 2; ++e) {
+                    const float a = o[nd][half * 2 + e] * inv;
+                    const float v = fmaf(-p.diff_lam, __shfl_xor_sync(0xffffffffu, a, 4), a);
+                    o[nd][half * 2 + e] = v;
+                    ss = fmaf(v, v, ss);
+                }
+            }
+            ss += __shfl_xor_sync(0xffffffffu, ss, 1);
+            ss += __shfl_xor_sync(0xffffffffu, ss, 2);
+            const int r = half ? r_hi : r_lo;
+            const int tl = r / Gc, hl = r - tl * Gc, hg = chunk * R + hl;
+            if (!(tl < ti.n_tok && hg < G && tl < QT) || (r & 1)) continue;
+            const float f = p.diff_scale / sqrtf(ss / (float)D + p.diff_eps);
+            const size_t tok = (size_t)(ti.q_base + ti.t0 + tl);
+            __nv_bfloat16* dst = og + (tok * (p.n_q / 2) + (kvh * G + hg) / 2) * D;
+#pragma unroll
+            for (int nd = 0; nd < NDB; ++nd)
+                *reinterpret_cast<__nv_bfloat162*>(dst + nd * 8 + (lane & 3) * 2) =
+                    __floats2bfloat162_rn(o[nd][half * 2] * f, o[nd][half * 2 + 1] * f);
+        }
+    } else {
 #pragma unroll
         for (int half = 0; half < 2; ++half) {
             const int r = half ? r_hi : r_lo;
@@ -778,7 +813,7 @@ __global__ void __launch_bounds__(NW * 32) attn_decode_kernel(const AttnParams p
         }
         const size_t tok = (size_t)(ti.q_base + ti.t0 + tl);
         const int head = kvh * G + hg;
-        if (ns == 1) {
+        if (ns == 1 && !p.diff) {
             L += null_weight(p.null_log2, head, Mu);
             og[(tok * p.n_q + head) * D + col] =
                 __float2bfloat16_rn((L > 0.f ? acc / L : 0.f) * gate_factor<__nv_bfloat16>(p.gate, p.gate_stride, tok, head * D + col));
@@ -1141,7 +1176,7 @@ __device__ __forceinline__ void decode_t_run(const AttnParams& p, const TileInfo
         }
         const size_t tok = (size_t)(ti.q_base + ti.t0 + tl);
         const int head = kvh * G + hg;
-        if (ns == 1) {
+        if (ns == 1 && !p.diff) {
             L += null_weight(p.null_log2, head, Mu);
             og[(tok * p.n_q + head) * D + col] =
                 __float2bfloat16_rn((L > 0.f ? acc / L : 0.f) * gate_factor<__nv_bfloat16>(p.gate, p.gate_stride, tok, head * D + col));
@@ -1409,6 +1444,62 @@ __global__ void attn_combine_kernel(const float* __restrict__ part_o, const floa
     }
 }
 
+// The same for heads that are the difference of two maps: one block per (token, output head) joins the pieces of query heads 2 h
+// and 2 h + 1 (also where a request has one piece only), takes the difference and norms it.  Requests whose query runs are longer
+// than qlen_max (not taken by the kernels of short query runs) and not cut are done already.
+template <typename T>
+__global__ void attn_combine_diff_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
+                                         const int* __restrict__ token_req, const int* __restrict__ nsplit, const int* __restrict__ q_start,
+                                         int qlen_max, T* __restrict__ out, int T_, int n_q, int d, int max_split, float lam, float eps,
+                                         float scale) {
+    __shared__ float red[32];
+    pdl_launch_dependents();
+    pdl_wait();
+    pdl_after_wait();
+    pdl_small();
+    const int tok = blockIdx.x, h = blockIdx.y;
+    const int req = token_req ? token_req[tok] : tok;
+    const int ns = nsplit ? min(max(nsplit[req], 1), max_split) : 1;
+    if (ns == 1 && q_start[req + 1] - q_start[req] > qlen_max) return;
+    float f[2], M[2];
+#pragma unroll
+    for (int m = 0; m < 2; ++m) {
+        M[m] = -INFINITY;
+        for (int s = 0; s < ns; ++s) M[m] = fmaxf(M[m], part_ml[(((size_t)s * T_ + tok) * n_q + 2 * h + m) * 2]);
+        if (M[m] == -INFINITY) M[m] = 0.f;
+        float L = 0.f;
+        for (int s = 0; s < ns; ++s) {
+            const size_t prow = ((size_t)s * T_ + tok) * n_q + 2 * h + m;
+            L += exp2f(part_ml[prow * 2] - M[m]) * part_ml[prow * 2 + 1];
+        }
+        f[m] = L > 0.f ? 1.f / L : 0.f;
+    }
+    float ss = 0.f;
+    constexpr int MAX_TURNS = 4;                 // 128 threads, head sizes up to 512
+    float v[MAX_TURNS];
+#pragma unroll
+    for (int k = 0; k < MAX_TURNS; ++k) {
+        const int c = threadIdx.x + k * blockDim.x;
+        v[k] = 0.f;
+        if (c < d) {
+            float acc[2] = {0.f, 0.f};
+            for (int s = 0; s < ns; ++s) {
+                const size_t prow = ((size_t)s * T_ + tok) * n_q + 2 * h;
+                acc[0] += exp2f(part_ml[prow * 2] - M[0]) * part_o[prow * d + c];
+                acc[1] += exp2f(part_ml[prow * 2 + 2] - M[1]) * part_o[(prow + 1) * d + c];
+            }
+            v[k] = fmaf(acc[0], f[0], -lam * (acc[1] * f[1]));
+            ss = fmaf(v[k], v[k], ss);
+        }
+    }
+    const float g = scale / sqrtf(block_sum(ss, red) / (float)d + eps);
+#pragma unroll
+    for (int k = 0; k < MAX_TURNS; ++k) {
+        const int c = threadIdx.x + k * blockDim.x;
+        if (c < d) out[((size_t)tok * (n_q / 2) + h) * d + c] = from_f32<T>(v[k] * g);
+    }
+}
+
 #if MSGL_HEAD_DIM == 128
 #include "attention_tc.cuh"
 #include "attention_tc2.cuh"
@@ -1465,17 +1556,22 @@ static int attention_launch(const void* q, void* out, const void* k_cache, const
                             int window, int max_split, float scale, int qlen_min, int qlen_max, int uniform_decode,
                             int variant, int grid_x, int dtype, const int* order, const int* even, int even_nb,
                             int keep_first, const float* bias, int bias_len, const float* null_log2, const void* gate,
-                            long long gate_stride, int chunk_keys, cudaStream_t stream);
+                            long long gate_stride, int chunk_keys, int diff, float diff_lam,
+                            float diff_eps, float diff_scale, cudaStream_t stream);
 
+// diff: the query heads are pairs of maps (AttnParams::diff); out is then [T, n_q / 2, d], variant 1 writes it, variant 2 leaves
+// partial results for msgl_attention_combine_diff (part_o, part_ml are needed even with max_split 1).
 MSGL_API int msgl_attention(const void* q, void* out, const void* k_cache, const void* v_cache, const int* q_start,
                             const int* kv_len, const int* block_table, const int* nsplit, float* part_o,
                             float* part_ml, int B, int T_, int n_q, int n_kv, int d, int page_size, int bt_stride,
                             int window, int max_split, float scale, int qlen_min, int qlen_max, int uniform_decode,
                             int variant, int grid_x, int dtype, const int* order, const int* even, int even_nb,
-                            const float* null_log2, const void* gate, long long gate_stride, int chunk_keys, cudaStream_t stream) {
+                            const float* null_log2, const void* gate, long long gate_stride, int chunk_keys, int diff, float diff_lam,
+                            float diff_eps, float diff_scale, cudaStream_t stream) {
     return attention_launch(q, out, k_cache, v_cache, q_start, kv_len, block_table, nsplit, part_o, part_ml, B, T_, n_q, n_kv, d,
                             page_size, bt_stride, window, max_split, scale, qlen_min, qlen_max, uniform_decode, variant, grid_x,
-                            dtype, order, even, even_nb, 0, nullptr, 0, null_log2, gate, gate_stride, chunk_keys, stream);
+                            dtype, order, even, even_nb, 0, nullptr, 0, null_log2, gate, gate_stride, chunk_keys, diff, diff_lam, diff_eps, diff_scale,
+                            stream);
 }
 
 // The same with a window that keeps the first `keep_first` keys of every request visible and with a bias by distance
@@ -1492,7 +1588,7 @@ MSGL_API int msgl_attention_window(const void* q, void* out, const void* k_cache
     if (!(variant == 1 || (variant == 2 && MSGL_HEAD_DIM % 32 == 0 && G <= 16))) return MSGL_ERR_SIZE;
     return attention_launch(q, out, k_cache, v_cache, q_start, kv_len, block_table, nsplit, part_o, part_ml, B, T_, n_q, n_kv, d,
                             page_size, bt_stride, window, max_split, scale, qlen_min, qlen_max, uniform_decode, variant, grid_x,
-                            dtype, order, nullptr, 0, keep_first, bias, bias_len, nullptr, nullptr, 0, 0, stream);
+                            dtype, order, nullptr, 0, keep_first, bias, bias_len, nullptr, nullptr, 0, 0, 0, 0.f, 0.f, 0.f, stream);
 }
 
 static int attention_launch(const void* q, void* out, const void* k_cache, const void* v_cache, const int* q_start,
@@ -1501,7 +1597,11 @@ static int attention_launch(const void* q, void* out, const void* k_cache, const
                             int window, int max_split, float scale, int qlen_min, int qlen_max, int uniform_decode,
                             int variant, int grid_x, int dtype, const int* order, const int* even, int even_nb,
                             int keep_first, const float* bias, int bias_len, const float* null_log2, const void* gate,
-                            long long gate_stride, int chunk_keys, cudaStream_t stream) {
+                            long long gate_stride, int chunk_keys, int diff, float diff_lam, float diff_eps, float diff_scale,
+                            cudaStream_t stream) {
+    if (diff && ((variant != 1 && variant != 2) || n_kv <= 0 || (n_q / n_kv) % 2 || gate != nullptr || null_log2 != nullptr ||
+                 keep_first > 0 || bias != nullptr || (variant == 2 && (part_o == nullptr || part_ml == nullptr))))
+        return MSGL_ERR_SIZE;
     if (chunk_keys < 0 || (chunk_keys > 0 && window > 0)) return MSGL_ERR_SIZE;
     if (gate != nullptr && dtype == MSGL_BF16 && ((gate_stride & 1) || ((uintptr_t)gate & 3))) return MSGL_ERR_ALIGN;
     if (grid_x <= 0 || B <= 0) return MSGL_OK;
@@ -1518,6 +1618,7 @@ static int attention_launch(const void* q, void* out, const void* k_cache, const
     p.uniform_decode = uniform_decode;
     p.keep_first = window > 0 ? keep_first : 0; p.bias = bias; p.bias_len = bias_len;
     p.null_log2 = null_log2; p.gate = gate; p.gate_stride = gate_stride;
+    p.diff = diff; p.diff_lam = diff_lam; p.diff_eps = diff_eps; p.diff_scale = diff_scale;
     const int G = n_q / n_kv;
     const int R = variant == 1 ? 64 : 16;
     const int n_chunks = G <= R ? 1 : (G + R - 1) / R;
@@ -1621,12 +1722,15 @@ MSGL_API int msgl_attention_tc(const void* q, void* out, const void* k_cache, co
                                int page_size, int bt_stride, int window, float scale, int qlen_min, int qlen_max,
                                int grid_x, int cache_pages, int version, int* status, int keep_first, const float* bias,
                                int bias_len, const float* null_log2, const void* gate, long long gate_stride, int chunk_keys,
-                               cudaStream_t stream) {
+                               int diff, float diff_lam, float diff_eps, float diff_scale, cudaStream_t stream) {
 #if MSGL_HEAD_DIM == 128
     if (gate != nullptr && ((gate_stride & 7) || ((uintptr_t)gate & 15))) return MSGL_ERR_ALIGN;
     // kept first tokens under the window and a bias by distance ([n_q][bias_len] float32, log2 units): version 2 only
     const bool ext = (window > 0 && keep_first > 0) || bias != nullptr;
     if (chunk_keys < 0 || (chunk_keys > 0 && window > 0)) return MSGL_ERR_SIZE;
+    // pairs of maps (AttnParams::diff): version 2 only, out [T, n_q / 2, 128]
+    if (diff && (version != 2 || ext || null_log2 != nullptr || gate != nullptr || n_kv <= 0 || (n_q / n_kv) % 2 || n_q / n_kv > 2 * TC_ROWS))
+        return MSGL_ERR_SIZE;
     if (ext && (version != 2 || keep_first < 0 || (bias != nullptr && bias_len < 1))) return MSGL_ERR_SIZE;
     if (grid_x <= 0 || B <= 0) return MSGL_OK;
     if (d != 128 || n_kv <= 0 || n_q % n_kv != 0 || page_size <= 0 || grid_x > 65535) return MSGL_ERR_SIZE;
@@ -1641,15 +1745,17 @@ MSGL_API int msgl_attention_tc(const void* q, void* out, const void* k_cache, co
     if ((page_size & (page_size - 1)) == 0) { int sh = 0; while ((1 << sh) < page_size) ++sh; p.page_shift = sh; }
     p.scale = scale; p.qlen_min = qlen_min; p.qlen_max = qlen_max; p.uniform_decode = 0;
     p.null_log2 = null_log2; p.gate = gate; p.gate_stride = gate_stride;
+    p.diff = diff; p.diff_lam = diff_lam; p.diff_eps = diff_eps; p.diff_scale = diff_scale;
     p.keep_first = window > 0 ? keep_first : 0; p.bias = bias; p.bias_len = bias_len;
     const int G = n_q / n_kv;
-    const int n_chunks = G <= TC_ROWS ? 1 : (G + TC_ROWS - 1) / TC_ROWS;
+    const int n_chunks = (diff || G <= TC_ROWS) ? 1 : (G + TC_ROWS - 1) / TC_ROWS;
     const size_t smem = (size_t)TC_SMEM_BYTES + 1024;
     static MsglOncePerDevice attr_set;
     if (attr_set.due()) {      // first call on this device, never inside a stream capture
         if (cudaFuncSetAttribute(attn_tc_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess ||
             cudaFuncSetAttribute(attn_tc2_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TC2_SMEM_ALLOC) != cudaSuccess ||
-            cudaFuncSetAttribute(attn_tc2_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TC2_SMEM_ALLOC) != cudaSuccess)
+            cudaFuncSetAttribute(attn_tc2_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TC2_SMEM_ALLOC) != cudaSuccess ||
+            cudaFuncSetAttribute(attn_tc2_kernel<false, true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)TC2_SMEM_ALLOC) != cudaSuccess)
             return msgl_check_launch();
         attr_set.mark();
     }
@@ -1665,7 +1771,8 @@ MSGL_API int msgl_attention_tc(const void* q, void* out, const void* k_cache, co
     }
     if (version == 2) {
         if (tma_box == 0) return MSGL_ERR_SIZE;
-        if (ext) attn_tc2_kernel<true><<<dim3(n_kv * n_chunks, grid_x, 1), TC2_THREADS, TC2_SMEM_ALLOC, stream>>>(p, status, kmap, vmap, tma_box);
+        if (diff) attn_tc2_kernel<false, true><<<dim3(n_kv, grid_x, 1), TC2_THREADS, TC2_SMEM_ALLOC, stream>>>(p, status, kmap, vmap, tma_box);
+        else if (ext) attn_tc2_kernel<true><<<dim3(n_kv * n_chunks, grid_x, 1), TC2_THREADS, TC2_SMEM_ALLOC, stream>>>(p, status, kmap, vmap, tma_box);
         else attn_tc2_kernel<false><<<dim3(n_kv * n_chunks, grid_x, 1), TC2_THREADS, TC2_SMEM_ALLOC, stream>>>(p, status, kmap, vmap, tma_box);
         return msgl_check_launch();
     }
@@ -1688,6 +1795,25 @@ MSGL_API int msgl_attention_combine(const float* part_o, const float* part_ml, c
     else if (dtype == MSGL_BF16)
         msgl_launch_pdl(attn_combine_kernel<__nv_bfloat16>, grid, dim3(threads), 0, stream, part_o, part_ml, token_req, nsplit,
                         (__nv_bfloat16*)out, T_, n_q, d, max_split, null_log2, gate, gate_stride);
+    else
+        return MSGL_ERR_DTYPE;
+    return msgl_check_launch();
+}
+
+// The merge for pairs of maps: out [T, n_q / 2, d]; q_start [B + 1], qlen_max and nsplit tell which requests left partial
+// results.
+MSGL_API int msgl_attention_combine_diff(const float* part_o, const float* part_ml, const int* token_req, const int* nsplit,
+                                         const int* q_start, int qlen_max, void* out, int T_, int n_q, int d, int max_split, int dtype,
+                                         float lam, float eps, float scale, cudaStream_t stream) {
+    if (T_ <= 0) return MSGL_OK;
+    if (n_q < 2 || n_q % 2 || d < 1 || d > 512 || max_split < 1 || (max_split > 1 && nsplit == nullptr)) return MSGL_ERR_SIZE;
+    const dim3 grid(T_, n_q / 2);
+    if (dtype == MSGL_F32)
+        msgl_launch_pdl(attn_combine_diff_kernel<float>, grid, dim3(128), 0, stream, part_o, part_ml, token_req, nsplit, q_start, qlen_max,
+                        (float*)out, T_, n_q, d, max_split, lam, eps, scale);
+    else if (dtype == MSGL_BF16)
+        msgl_launch_pdl(attn_combine_diff_kernel<__nv_bfloat16>, grid, dim3(128), 0, stream, part_o, part_ml, token_req, nsplit, q_start,
+                        qlen_max, (__nv_bfloat16*)out, T_, n_q, d, max_split, lam, eps, scale);
     else
         return MSGL_ERR_DTYPE;
     return msgl_check_launch();

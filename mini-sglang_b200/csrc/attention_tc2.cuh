@@ -18,6 +18,14 @@
 // to do, while group B works on S_B(j) it has P V_A(j) and S_A(j+1).  P_X overwrites S_X, so
 // S_X(j+1) is issued after P V_X(j); the tensor core executes in order.
 //
+// DIFF: heads that are the difference of two maps (AttnParams::diff).  Both tiles then hold the same (token, head) rows, A with
+// the head's first query vector against the first 64 elements of a key row, B with the second against the others (four of the
+// eight steps of a product each), and the epilogue joins the two: a softmax thread of either group reads its half of the
+// columns of O_A and O_B from tensor memory, takes the difference, and the halves' sums of squares meet in shared memory.
+//
+// Results (and gates, fetched while the last tile is worked on) pass through the shared memory of the tile's Q, so that a warp's
+// accesses to global memory cover whole rows.
+//
 // Warps: 0-3 softmax A, 4-7 softmax B, 8 K loader, 9 V loader (TMA, see attention_tc.cuh), 10 issuer,
 // 11 idle after the Q gather.  All waits are bounded as in attention_tc.cuh.
 #pragma once
@@ -50,7 +58,7 @@ constexpr unsigned TC2_SMEM_ALLOC = TC2_SMEM_BYTES + 256u + 1024u;
 // EXT: the launch has kept first tokens under its window or a bias by distance (AttnParams::keep_first, bias): the key tiles
 // that hold kept tokens before the window's first tile are walked ahead of the window's, and every score gets its table entry.
 // Without EXT none of that is compiled in.
-template <bool EXT>
+template <bool EXT, bool DIFF = false>
 __global__ void __launch_bounds__(TC2_THREADS, 1) attn_tc2_kernel(const AttnParams p, int* status,
                                                                   const __grid_constant__ CUtensorMap kmap,
                                                                   const __grid_constant__ CUtensorMap vmap, int tma_box) {
@@ -78,20 +86,21 @@ __global__ void __launch_bounds__(TC2_THREADS, 1) attn_tc2_kernel(const AttnPara
     const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31;
 
     const int G = p.n_q / p.n_kv;
-    const int Gc = G <= TC_ROWS ? G : TC_ROWS;
-    const int n_chunks = G <= TC_ROWS ? 1 : (G + TC_ROWS - 1) / TC_ROWS;
-    const int QH = G <= TC_ROWS ? TC_ROWS / G : 1;             // tokens of one 128-row tile
+    const int Gt = DIFF ? G / 2 : G;                            // rows of one token in a tile
+    const int Gc = Gt <= TC_ROWS ? Gt : TC_ROWS;
+    const int n_chunks = Gt <= TC_ROWS ? 1 : (Gt + TC_ROWS - 1) / TC_ROWS;
+    const int QH = Gt <= TC_ROWS ? TC_ROWS / Gt : 1;            // tokens of one 128-row tile
     // The grid is (kv heads, query tiles): blocks are handed out head-first, so all heads of the heaviest tile
     // start before any lighter tile (with one tile index per blockIdx.x the first heads would take every SM).
     const int kvh = blockIdx.x / n_chunks;
     const int chunk = blockIdx.x - kvh * n_chunks;
 
     TileInfo ti;
-    if (!find_tile(p, 2 * QH, ti, sh_tile, (int)blockIdx.y, (int)gridDim.y)) return;
+    if (!find_tile(p, DIFF ? QH : 2 * QH, ti, sh_tile, (int)blockIdx.y, (int)gridDim.y)) return;
     // positions of the block's tokens and its key tiles (anchored at absolute positions)
     const int p_min = ti.kv_len - ti.q_len + ti.t0;
     const int p_max = p_min + ti.n_tok - 1;
-    const int ntok_a = min(ti.n_tok, QH), ntok_b = ti.n_tok - ntok_a;
+    const int ntok_a = DIFF ? ti.n_tok : min(ti.n_tok, QH), ntok_b = DIFF ? ti.n_tok : ti.n_tok - ntok_a;
     const int pmax_a = p_min + ntok_a - 1;
     const int k_lo = first_key(p, p_min);                        // the first key any row of the block sees
     const int kt_begin = k_lo / TC_KT;
@@ -121,7 +130,17 @@ __global__ void __launch_bounds__(TC2_THREADS, 1) attn_tc2_kernel(const AttnPara
     const unsigned tmem = tmem_base_s;
     int fail = 0;
 
-    {   // Q: 256 rows x 16 chunks of 16 bytes, spread over all threads; rows without a query are zero-filled
+    if (DIFF) {   // Q: 2 x 128 rows x 8 chunks of 16 bytes: tile x has vector x of the rows' heads, in columns 64 x .. 64 x + 63
+        const __nv_bfloat16* qg = reinterpret_cast<const __nv_bfloat16*>(p.q);
+        for (int idx = tid; idx < TC2_ROWS * 8; idx += TC2_THREADS) {
+            const int r = idx >> 3, x = r >> 7, rr = r & 127, c = (idx & 7) + 8 * x;
+            const int tl = rr / Gc, hl = rr % Gc;
+            const bool valid = tl < QH && tl < ti.n_tok;
+            const __nv_bfloat16* src = qg + ((size_t)(ti.q_base + ti.t0 + (valid ? tl : 0)) * p.n_q + (size_t)kvh * G + (valid ? 2 * hl + x : 0)) * TC_D;
+            cp_async16_u32(q_s + (unsigned)x * TC_Q_BYTES + tc_tile_off(rr, c, TC_QHALF_BYTES), src + c * 8, valid);
+        }
+        tc_cp_async_arrive(bar_q);
+    } else {   // Q: 256 rows x 16 chunks of 16 bytes, spread over all threads; rows without a query are zero-filled
         const __nv_bfloat16* qg = reinterpret_cast<const __nv_bfloat16*>(p.q);
         for (int idx = tid; idx < TC2_ROWS * 16; idx += TC2_THREADS) {
             const int r = idx >> 4, c = idx & 15;
@@ -144,8 +163,8 @@ __global__ void __launch_bounds__(TC2_THREADS, 1) attn_tc2_kernel(const AttnPara
         auto box_row = [&](int j) -> int {            // first cache row of this lane's box of tile j, or -1
             int key_b = tile_of(j) * TC_KT + lane * tma_box;
             // boxes before the first key that is seen: their pages may have been given back; the rows of that key's own box stand
-            // in for them (finite, and no row of the block gives them weight)
-            if (!(EXT && j < n_sink)) key_b = max(key_b, k_lo - k_lo % tma_box);
+            // in for them (finite, and no row of the block gives them weight).  Boxes with kept first tokens are always there.
+            if (!(EXT && (j < n_sink || key_b < p.keep_first))) key_b = max(key_b, k_lo - k_lo % tma_box);
             if (j >= n_tiles || lane >= n_box || key_b > p_max) return -1;          // boxes past the last visible key are not fetched
             if (EXT && j < n_sink && key_b >= sink_hi) return -1;                   // nor those past the last kept token
             return (bt[page_index(p, key_b)] * p.n_kv + kvh) * p.page_size + page_slot(p, key_b);
@@ -200,10 +219,13 @@ __global__ void __launch_bounds__(TC2_THREADS, 1) attn_tc2_kernel(const AttnPara
                 tp_[kk] = (unsigned)kk * 8u;
             }
             const unsigned long long stage_step = (unsigned long long)(TC_KV_BYTES >> 4);     // address field counts 16-byte units
-            auto issue_s = [&](int x, int j) {                            // S_X(j) = Q_X K(j)^T: 8 steps of 16 along the head size
+            auto issue_s = [&](int x, int j) {                            // S_X(j) = Q_X K(j)^T: 8 steps of 16 along the head size (DIFF: the 4 of half x)
                 const unsigned long long ks = (j & 1) ? stage_step : 0ull;
 #pragma unroll
-                for (int kk = 0; kk < 8; ++kk) tc_mma(tmem + (unsigned)x * 128u, dq[x][kk], dk[kk] + ks, idesc_s, kk > 0 ? 1u : 0u);
+                for (int kk = 0; kk < 8; ++kk) {
+                    if (DIFF && (kk >> 2) != x) continue;
+                    tc_mma(tmem + (unsigned)x * 128u, dq[x][kk], dk[kk] + ks, idesc_s, (DIFF ? (kk & 3) : kk) > 0 ? 1u : 0u);
+                }
                 tc_commit(bar_s(x));
             };
             auto issue_o = [&](int x, int j) {                            // O_X += P_X V(j): 8 steps of 16 keys, P from tensor memory
@@ -250,15 +272,19 @@ __global__ void __launch_bounds__(TC2_THREADS, 1) attn_tc2_kernel(const AttnPara
         const int n_mine = x ? n_b : n_a;
         const unsigned lane_sel = (unsigned)((warp & 3) * 32) << 16;
         const unsigned ts = tmem + (unsigned)x * 128u + lane_sel, to = tmem + 256u + (unsigned)x * 128u + lane_sel;
-        const int my_tl = x * QH + row / Gc;
+        const int my_tl = (DIFF ? 0 : x * QH) + row / Gc;
         const int my_pos = p_min + my_tl;
-        const bool my_valid = row / Gc < QH && my_tl < ti.n_tok && (chunk * TC_ROWS + row % Gc) < G;
-        const int pmin_x = p_min + x * QH, pmax_x = x ? p_max : pmax_a;
+        const bool my_valid = row / Gc < QH && my_tl < ti.n_tok && (chunk * TC_ROWS + row % Gc) < Gt;
+        const int pmin_x = p_min + (DIFF ? 0 : x * QH), pmax_x = x ? p_max : pmax_a;
         const float sc = p.scale * 1.4426950408889634f;
         const float inv_sc = 1.f / sc;
         const float* my_bias = (EXT && p.bias != nullptr)
             ? p.bias + (size_t)min(kvh * G + chunk * TC_ROWS + row % Gc, p.n_q - 1) * p.bias_len : nullptr;
         float m_run = -INFINITY, l_run = 0.f, o_scale = 1.f;
+        // the rows of this warp in global memory and in shared memory, two rows (16 lanes each) an access
+        const int my_head = DIFF ? kvh * Gt + row % Gc : kvh * G + (my_valid ? chunk * TC_ROWS + row % Gc : 0);      // of the output
+        const size_t my_tok = (size_t)(ti.q_base + ti.t0 + (my_valid ? my_tl : 0));
+        const unsigned stage_s = q_s + (unsigned)x * TC_Q_BYTES;            // Q_X; free once the last S_X has been made
 #ifdef MSGL_TC_PROFILE
         long long tp[8] = {0, 0, 0, 0, 0, 0, 0, 0};
         long long t0 = clock64(), t1;
@@ -270,6 +296,18 @@ __global__ void __launch_bounds__(TC2_THREADS, 1) attn_tc2_kernel(const AttnPara
             if (!tc_mbar_wait(bar_s(x), it & 1)) { fail = 1; break; }
             tc_fence_after();
             TC2_MARK(0)
+            if (!DIFF && p.gate != nullptr && it + 1 == n_mine) {
+                // Q_X has been read for the last time: the rows' gates take its place while the last tile is worked on
+                const unsigned long long mine = reinterpret_cast<unsigned long long>(
+                    reinterpret_cast<const __nv_bfloat16*>(p.gate) + my_tok * p.gate_stride + (size_t)my_head * TC_D);
+#pragma unroll 4
+                for (int i = 0; i < 16; ++i) {
+                    const int r = 2 * i + (lane >> 4), c = lane & 15;
+                    const unsigned long long src = __shfl_sync(0xffffffffu, mine, r);
+                    cp_async16_u32(stage_s + tc_tile_off((warp & 3) * 32 + r, c, TC_QHALF_BYTES), reinterpret_cast<const void*>(src + c * 16), true);
+                }
+                cp_async_commit();
+            }
             const int key0 = tile_of(it) * TC_KT;
             const bool in_sink = EXT && it < n_sink;
             const bool need_mask = in_sink || (key0 + TC_KT - 1 > pmin_x) || key0 < first_key(p, pmax_x);
@@ -399,42 +437,90 @@ __global__ void __launch_bounds__(TC2_THREADS, 1) attn_tc2_kernel(const AttnPara
         }
 #endif
         // epilogue: the last P V product, normalise, write
+        auto st_stage = [&](int c, const uint4& v) {                     // 16-byte chunk c of this thread's row
+            asm volatile("st.shared.v4.u32 [%0], {%1,%2,%3,%4};\n" ::"r"(stage_s + tc_tile_off(row, c, TC_QHALF_BYTES)), "r"(v.x), "r"(v.y), "r"(v.z), "r"(v.w) : "memory");
+        };
+        auto ld_stage = [&](int r, int c) -> uint4 {
+            uint4 v;
+            asm volatile("ld.shared.v4.u32 {%0,%1,%2,%3}, [%4];\n" : "=r"(v.x), "=r"(v.y), "=r"(v.z), "=r"(v.w) : "r"(stage_s + tc_tile_off(r, c, TC_QHALF_BYTES)) : "memory");
+            return v;
+        };
+        __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(p.out) + (my_tok * (DIFF ? p.n_q / 2 : p.n_q) + my_head) * TC_D;
+        const unsigned long long my_dst = my_valid ? reinterpret_cast<unsigned long long>(dst) : 0ull;
         if (!fail && n_mine > 0) {
             if (!tc_mbar_wait(bar_o(x), (n_mine - 1) & 1)) fail = 1;
+            if (DIFF && !fail && !tc_mbar_wait(bar_o(1 - x), (n_mine - 1) & 1)) fail = 1;      // the tiles have the same number of keys
             tc_fence_after();
         }
-        if (!__any_sync(0xffffffffu, fail) && n_mine > 0) {
-            const int my_head = kvh * G + (my_valid ? chunk * TC_ROWS + row % Gc : 0);
-            const size_t my_tok = (size_t)(ti.q_base + ti.t0 + (my_valid ? my_tl : 0));
+        if (DIFF) {
+            // both groups take part in every barrier here, also where one of them has given up
+            float* ex = reinterpret_cast<float*>(tc_smem + (k_s - smem_base));        // [2][128] factors, [2][128] sums of squares (K has been read)
+            ex[x * 128 + row] = l_run > 0.f ? o_scale / l_run : 0.f;
+            asm volatile("bar.sync 1, 256;\n" ::: "memory");
+            const float fa = ex[row], fb = ex[128 + row] * p.diff_lam;
+            const unsigned ta = tmem + 256u + lane_sel + (unsigned)x * 64u;           // this group's half of the columns of O_A; O_B: 128 further
+            float v[2][32], ss = 0.f;
+#pragma unroll
+            for (int cb = 0; cb < 2; ++cb) {
+                float b[32];
+                tc_ld32(ta + cb * 32, v[cb]); tc_ld32(ta + 128u + cb * 32, b);
+                tc_wait_ld(v[cb]); tc_wait_ld(b);
+#pragma unroll
+                for (int j = 0; j < 32; ++j) { v[cb][j] = fmaf(v[cb][j], fa, -b[j] * fb); ss = fmaf(v[cb][j], v[cb][j], ss); }
+            }
+            ex[256 + x * 128 + row] = ss;
+            asm volatile("bar.sync 1, 256;\n" ::: "memory");
+            const float f = p.diff_scale / sqrtf((ex[256 + row] + ex[384 + row]) * (1.f / TC_D) + p.diff_eps);
+#pragma unroll
+            for (int c = 0; c < 8; ++c) {
+                const float* w = &v[c >> 2][(c & 3) * 8];
+                st_stage(c, make_uint4(pack_bf16(w[0] * f, w[1] * f), pack_bf16(w[2] * f, w[3] * f), pack_bf16(w[4] * f, w[5] * f), pack_bf16(w[6] * f, w[7] * f)));
+            }
+            __syncwarp();
+            if (!__any_sync(0xffffffffu, fail)) {
+#pragma unroll 4
+                for (int i = 0; i < 8; ++i) {                            // four rows an access, 8 lanes each: 128 bytes of a row
+                    const int r = 4 * i + (lane >> 3), c = lane & 7;
+                    const unsigned long long d = __shfl_sync(0xffffffffu, my_dst, r);
+                    const uint4 o = ld_stage((warp & 3) * 32 + r, c);
+                    if (d != 0ull) *reinterpret_cast<uint4*>(d + x * 128 + c * 16) = o;
+                }
+            }
+        } else if (!__any_sync(0xffffffffu, fail) && n_mine > 0) {
             const float l_all = l_run + null_weight(p.null_log2, my_head, m_run);
             const float inv = l_all > 0.f ? o_scale / l_all : 0.f;        // o_scale: a move of the reference after the last tile
-            const __nv_bfloat16* gt = p.gate ? reinterpret_cast<const __nv_bfloat16*>(p.gate) + my_tok * p.gate_stride + (size_t)my_head * TC_D : nullptr;
-            __nv_bfloat16* dst = reinterpret_cast<__nv_bfloat16*>(p.out) + (my_tok * p.n_q + my_head) * TC_D;
+            if (p.gate != nullptr) {
+                cp_async_wait<0>();
+                __syncwarp();
+            }
 #pragma unroll 1
             for (int cb = 0; cb < 4; ++cb) {
                 float v[32];
                 tc_ld32(to + cb * 32, v);                                // every thread of the warp takes part
                 tc_wait_ld(v);
-                if (my_valid) {
 #pragma unroll
-                    for (int j = 0; j < 32; j += 8) {
-                        uint4 pk;
-                        if (gt != nullptr) {
-                            const uint4 g = *reinterpret_cast<const uint4*>(gt + cb * 32 + j);
-                            const unsigned gw[4] = {g.x, g.y, g.z, g.w};
+                for (int j = 0; j < 32; j += 8) {
+                    const int c = cb * 4 + j / 8;
+                    if (p.gate != nullptr) {
+                        const uint4 g = ld_stage(row, c);
+                        const unsigned gw[4] = {g.x, g.y, g.z, g.w};
 #pragma unroll
-                            for (int e = 0; e < 4; ++e) {
-                                const float2 f = gate_pair(gw[e]);
-                                v[j + 2 * e] *= f.x; v[j + 2 * e + 1] *= f.y;
-                            }
+                        for (int e = 0; e < 4; ++e) {
+                            const float2 f = gate_pair(gw[e]);
+                            v[j + 2 * e] *= f.x; v[j + 2 * e + 1] *= f.y;
                         }
-                        pk.x = pack_bf16(v[j] * inv, v[j + 1] * inv);
-                        pk.y = pack_bf16(v[j + 2] * inv, v[j + 3] * inv);
-                        pk.z = pack_bf16(v[j + 4] * inv, v[j + 5] * inv);
-                        pk.w = pack_bf16(v[j + 6] * inv, v[j + 7] * inv);
-                        *reinterpret_cast<uint4*>(dst + cb * 32 + j) = pk;
                     }
+                    st_stage(c, make_uint4(pack_bf16(v[j] * inv, v[j + 1] * inv), pack_bf16(v[j + 2] * inv, v[j + 3] * inv),
+                                           pack_bf16(v[j + 4] * inv, v[j + 5] * inv), pack_bf16(v[j + 6] * inv, v[j + 7] * inv)));
                 }
+            }
+            __syncwarp();
+#pragma unroll 4
+            for (int i = 0; i < 16; ++i) {
+                const int r = 2 * i + (lane >> 4), c = lane & 15;
+                const unsigned long long d = __shfl_sync(0xffffffffu, my_dst, r);
+                const uint4 o = ld_stage((warp & 3) * 32 + r, c);
+                if (d != 0ull) *reinterpret_cast<uint4*>(d + c * 16) = o;
             }
         }
     }

@@ -109,11 +109,12 @@ def _attn_lib(head_dim: int):
     if lib is None:
         lib = _build.attention_library(hd)
         lib.msgl_attention.argtypes = [c_void_p] * 10 + [c_int] * 9 + [c_float] + [c_int] * 6 + [c_void_p, c_void_p, c_int, c_void_p, c_void_p,
-                                       c_ll, c_int, c_void_p]
+                                       c_ll, c_int, c_int, c_float, c_float, c_float, c_void_p]
         lib.msgl_attention_window.argtypes = [c_void_p] * 10 + [c_int] * 9 + [c_float] + [c_int] * 6 + [c_void_p, c_int, c_void_p, c_int, c_void_p]
         lib.msgl_attention_combine.argtypes = [c_void_p] * 5 + [c_int] * 5 + [c_void_p, c_void_p, c_ll, c_void_p]
         lib.msgl_attention_tc.argtypes = [c_void_p] * 7 + [c_int] * 8 + [c_float] + [c_int] * 5 + [c_void_p, c_int, c_void_p, c_int, c_void_p,
-                                         c_void_p, c_ll, c_int, c_void_p]
+                                         c_void_p, c_ll, c_int, c_int, c_float, c_float, c_float, c_void_p]
+        lib.msgl_attention_combine_diff.argtypes = [c_void_p] * 5 + [c_int, c_void_p] + [c_int] * 5 + [c_float, c_float, c_float, c_void_p]
         lib.msgl_attention_head_dim.restype = c_int
         _attn[hd] = lib
     return lib
@@ -374,11 +375,12 @@ def attention_tc(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_ca
                  q_start: torch.Tensor, kv_len: torch.Tensor, block_table: torch.Tensor, n_kv: int, page_size: int,
                  window: int, scale: float, qlen_min: int, qlen_max: int, q_lens: Sequence[int], keep_first: int = 0,
                  bias_log2: Optional[torch.Tensor] = None, null_log2: Optional[torch.Tensor] = None,
-                 gate: Optional[torch.Tensor] = None, chunk: int = 0) -> bool:
+                 gate: Optional[torch.Tensor] = None, chunk: int = 0, diff: Optional[Tuple[float, float, float]] = None) -> bool:
     """Prefill attention on tcgen05 tensor cores for the requests with q_len in [qlen_min, qlen_max];
     q_lens: the host's copy of every request's number of query tokens (to size the grid).  keep_first, bias_log2: as in
     `attention`; they are taken by the kernel on pairs of query tiles only (TMA page sizes), and the call returns False,
-    having launched nothing, where that kernel cannot run.  null_log2, gate, chunk: as in `attention`, taken by both kernels."""
+    having launched nothing, where that kernel cannot run.  null_log2, gate, chunk: as in `attention`, taken by both kernels;
+    diff: as there, by the kernel on pairs of query tiles only."""
     global _tc2_usable
     gate_stride = _attention_extras(q, null_log2, gate)
     _need_cuda(q, out, k_cache, v_cache, q_start, kv_len, block_table)
@@ -391,7 +393,7 @@ def attention_tc(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_ca
     pages = k_cache.shape[0] if whole else 0
     tma_pages = whole and page_size >= 8 and (page_size & (page_size - 1)) == 0
     versions = [2, 1] if (TC_VERSION == 2 and _tc2_usable and tma_pages) else [1]
-    ext = bool(keep_first) or bias_log2 is not None
+    ext = bool(keep_first) or bias_log2 is not None or diff is not None
     if ext:
         _need_cuda(bias_log2)
         if versions[0] != 2:
@@ -407,7 +409,7 @@ def attention_tc(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_ca
             _ptr(q), _ptr(out), _ptr(k_cache), _ptr(v_cache), _ptr(q_start), _ptr(kv_len), _ptr(block_table), B, T, n_q,
             n_kv, d, page_size, block_table.stride(0), window, float(scale), qlen_min, qlen_max, grid_x, pages, version,
             _ptr(status), int(keep_first), _ptr(bias_log2), bias_log2.shape[1] if bias_log2 is not None else 0, _ptr(null_log2), _ptr(gate),
-            gate_stride, int(chunk), _stream())
+            gate_stride, int(chunk), int(diff is not None), *(diff or (0.0, 0.0, 0.0)), _stream())
         if code == 2 and version == 2:        # no tensor maps here (driver without the encoder, unaligned cache): one-tile kernel
             _tc2_usable = False
             if ext:
@@ -482,7 +484,7 @@ def attention(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_cache
               uniform_decode: bool, variant: int, grid_x: int, order: Optional[torch.Tensor] = None,
               even: Optional[torch.Tensor] = None, even_nb: int = 0, keep_first: int = 0,
               bias_log2: Optional[torch.Tensor] = None, null_log2: Optional[torch.Tensor] = None,
-              gate: Optional[torch.Tensor] = None, chunk: int = 0) -> None:
+              gate: Optional[torch.Tensor] = None, chunk: int = 0, diff: Optional[Tuple[float, float, float]] = None) -> None:
     """One launch of the paged attention kernel over the requests whose q_len lies in
     [qlen_min, qlen_max]; see csrc/attention.cu for the meaning of every argument.  keep_first: with a window, the first
     keys of a request that stay visible whatever the window; bias_log2: float32 [heads, L], added to the scaled score in
@@ -492,23 +494,25 @@ def attention(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_cache
     null_log2: float32 [heads], the score in log2 units of one more term in every softmax's denominator that has no key and no
     value; gate [T, heads * d] (a view into packed rows): the output times sigmoid(gate), element by element.  Both enter where a
     row is normalised, so a launch whose requests are cut hands them to `attention_combine` too.  chunk > 0 (with window 0): a query sees
-    the keys of its own chunk of `chunk` positions only, counted from the start of the sequence."""
+    the keys of its own chunk of `chunk` positions only, counted from the start of the sequence.  diff = (lambda, eps, scale): query heads 2 h and 2 h + 1 are the two maps of
+    output head h, out [T, n_q / 2, d] = v / sqrt(mean(v^2) + eps) * scale with v = a_2h - lambda a_2h+1; the decode variant leaves
+    partial results for `attention_combine_diff` whatever the splits."""
     gate_stride = _attention_extras(q, null_log2, gate)
     _need_cuda(q, out, k_cache, v_cache, q_start, kv_len, block_table, nsplit, part_o, part_ml, order, even)
     T, n_q, d = q.shape
     B = kv_len.numel()
     assert q.is_contiguous() and out.is_contiguous() and block_table.dim() == 2 and block_table.stride(1) == 1
-    assert q_start.numel() == B + 1 and block_table.shape[0] == B and out.shape == q.shape
+    assert q_start.numel() == B + 1 and block_table.shape[0] == B and tuple(out.shape) == (T, n_q if diff is None else n_q // 2, d)
     assert nsplit is None or nsplit.numel() == B
     assert order is None or (uniform_decode and order.numel() == B and order.dtype == torch.int32)
     assert even is None or (uniform_decode and variant == VARIANT_MMA_DECODE and even.dtype == torch.int32 and
                             even.numel() >= even_cut_size(B, even_nb) and even_nb >= 1)
-    if max_split > 1:
+    if max_split > 1 or (diff is not None and variant == VARIANT_MMA_DECODE):
         assert part_o.numel() >= max_split * T * n_q * d and part_ml.numel() >= max_split * T * n_q * 2
     if keep_first or bias_log2 is not None:
         _need_cuda(bias_log2)
         assert even is None, "the even cut of a decode step knows no kept tokens and no bias"
-        assert null_log2 is None and gate is None and not chunk, "a launch with kept tokens or a bias takes no further term, gate or chunk"
+        assert null_log2 is None and gate is None and not chunk and diff is None, "a launch with kept tokens or a bias takes no further term, gate, chunk or pairs of maps"
         if bias_log2 is not None:
             assert bias_log2.dtype == torch.float32 and bias_log2.dim() == 2 and bias_log2.shape[0] == n_q and bias_log2.is_contiguous()
         code = _attn_lib(d).msgl_attention_window(
@@ -522,7 +526,7 @@ def attention(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_cache
         _ptr(q), _ptr(out), _ptr(k_cache), _ptr(v_cache), _ptr(q_start), _ptr(kv_len), _ptr(block_table),
         _ptr(nsplit), _ptr(part_o), _ptr(part_ml), B, T, n_q, n_kv, d, page_size, block_table.stride(0), window,
         max_split, float(scale), qlen_min, qlen_max, int(uniform_decode), variant, grid_x, _dt(q), _ptr(order), _ptr(even), int(even_nb),
-        _ptr(null_log2), _ptr(gate), gate_stride, int(chunk), _stream())
+        _ptr(null_log2), _ptr(gate), gate_stride, int(chunk), int(diff is not None), *(diff or (0.0, 0.0, 0.0)), _stream())
     _check(code, f"attention (head size {d}, variant {variant})")
 
 
@@ -535,6 +539,18 @@ def attention_combine(part_o: torch.Tensor, part_ml: torch.Tensor, token_req: Op
     code = _attn_lib(d).msgl_attention_combine(_ptr(part_o), _ptr(part_ml), _ptr(token_req), _ptr(nsplit), _ptr(out),
                                                T, n_q, d, max_split, _dt(out), _ptr(null_log2), _ptr(gate), gate_stride, _stream())
     _check(code, "attention_combine")
+
+
+def attention_combine_diff(part_o: torch.Tensor, part_ml: torch.Tensor, token_req: Optional[torch.Tensor], nsplit: Optional[torch.Tensor],
+                           q_start: torch.Tensor, qlen_max: int, out: torch.Tensor, max_split: int, diff: Tuple[float, float, float]) -> None:
+    """The partial results of `attention(diff=...)` launches of the decode variant -> out [T, heads, d], for the tokens of the requests
+    that brought at most qlen_max of them or whose keys are cut."""
+    _need_cuda(part_o, part_ml, token_req, nsplit, q_start, out)
+    T, h, d = out.shape
+    assert out.is_contiguous() and part_o.numel() >= max_split * T * 2 * h * d and part_ml.numel() >= max_split * T * 2 * h * 2
+    code = _attn_lib(d).msgl_attention_combine_diff(_ptr(part_o), _ptr(part_ml), _ptr(token_req), _ptr(nsplit), _ptr(q_start), int(qlen_max),
+                                                    _ptr(out), T, 2 * h, d, max_split, _dt(out), *diff, _stream())
+    _check(code, "attention_combine_diff")
 
 
 # ---------------------------------------------------------------------------------------

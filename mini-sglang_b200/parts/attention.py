@@ -1,6 +1,6 @@
 from __future__ import annotations
 
-from typing import Dict, Optional
+from typing import Dict, Optional, Tuple
 
 import torch
 
@@ -106,25 +106,31 @@ class PagedAttention(Mixer):
 
 def paged_attend(q: torch.Tensor, out: torch.Tensor, ctx: StepContext, cache: KVCacheView, *, n_q: int, n_kv: int, d: int,
                  window: int, scale: float, use_mma: bool, keep_first: int = 0, bias_log2: Optional[torch.Tensor] = None,
-                 null_log2: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, chunk: int = 0) -> None:
+                 null_log2: Optional[torch.Tensor] = None, gate: Optional[torch.Tensor] = None, chunk: int = 0,
+                 diff: Optional[Tuple[float, float, float]] = None) -> None:
     """The attention launches of one step over a paged cache: requests that bring a few tokens through the decode kernel
     with the step's kv splits, longer runs through the prefill kernels, the merge of the splits.  keep_first and bias_log2
     (kept first tokens under a window, a bias by distance: `ops.attention`) are for mixers that have them; such launches
     run on the tcgen05 prefill kernel on pairs of query tiles where it applies and on the mma kernels otherwise.  null_log2
-    (a term in every softmax's denominator that has no key), gate (sigmoids on the output) and chunk (keys are seen within chunks
-    of the sequence only): `ops.attention`."""
+    (a term in every softmax's denominator that has no key), gate (sigmoids on the output), chunk (keys are seen within chunks
+    of the sequence only) and diff (query heads are pairs of maps, `out` holds half as many heads; the mma kernels only):
+    `ops.attention`."""
     plain = keep_first == 0 and bias_log2 is None
     if not plain and not use_mma:
         raise ValueError("kept first tokens and a distance bias are taken by the bfloat16 mma kernels only")
     joined = {} if null_log2 is None and gate is None else dict(null_log2=null_log2, gate=gate)
-    if chunk and not plain:
-        raise ValueError("a chunk goes with neither kept first tokens nor a distance bias")
-    extra = dict(joined, chunk=chunk) if plain else dict(keep_first=keep_first, bias_log2=bias_log2, **joined)
+    if (chunk or diff is not None) and not plain:
+        raise ValueError("chunks and pairs of maps go with neither kept first tokens nor a distance bias")
+    if diff is not None and (joined or not use_mma):
+        raise ValueError("pairs of maps are taken by the bfloat16 mma kernels only, without a further term or a gate")
+    extra = dict(joined, chunk=chunk, diff=diff) if plain else dict(keep_first=keep_first, bias_log2=bias_log2, **joined)
     g = cache.group
     G = n_q // n_kv
     max_split = g.max_split if g.nsplit is not None else 1
     part_o = part_ml = None
-    if max_split > 1:
+    qt_dec = ops.attention_tile_tokens(ops.VARIANT_MMA_DECODE, G, d) if use_mma else 0
+    merged = max_split > 1 or (diff is not None and any(n <= qt_dec for n in ctx.host_q_lens))      # whether partial results are left
+    if merged:
         rows = max_split * ctx.T * n_q
         part_o = ctx.workspace.get("attn_part_o", rows * d, torch.float32)
         part_ml = ctx.workspace.get("attn_part_ml", rows * 2, torch.float32)
@@ -138,7 +144,6 @@ def paged_attend(q: torch.Tensor, out: torch.Tensor, ctx: StepContext, cache: KV
         gx = ctx.B if ctx.uniform_decode else sum(-(-n // qt) for n in ctx.host_q_lens)
         ops.attention(q, out, cache.k, cache.v, qlen_min=1, qlen_max=big, variant=ops.VARIANT_SIMT, grid_x=gx, **common)
     else:
-        qt_dec = ops.attention_tile_tokens(ops.VARIANT_MMA_DECODE, G, d)
         qt_row = ops.attention_tile_tokens(ops.VARIANT_MMA_ROWS, G)
         if ctx.uniform_decode:
             even = dict(even=g.even, even_nb=g.even_nb) if plain else {}
@@ -161,5 +166,8 @@ def paged_attend(q: torch.Tensor, out: torch.Tensor, ctx: StepContext, cache: KV
             if n_row and not on_tc:
                 ops.attention(q, out, cache.k, cache.v, qlen_min=qt_dec + 1, qlen_max=big,
                               variant=ops.VARIANT_MMA_ROWS, grid_x=n_row, **common)
-    if max_split > 1:
+    if merged and diff is not None:
+        ops.attention_combine_diff(part_o, part_ml, None if ctx.uniform_decode else ctx.token_req, g.nsplit if max_split > 1 else None,
+                                   ctx.q_start, qt_dec, out, max_split, diff)
+    elif merged:
         ops.attention_combine(part_o, part_ml, None if ctx.uniform_decode else ctx.token_req, g.nsplit, out, max_split, **joined)

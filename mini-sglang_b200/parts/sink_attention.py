@@ -48,6 +48,7 @@ class SinkAttention(Mixer):
     """
 
     graph_safe = True
+    difference = None     # (lambda, eps, scale) of heads that are the difference of two maps
     maps = 1              # vectors of key_dim elements that a q or kv head has side by side, each with a softmax of its own
 
     def __init__(self, spec, prefix, env, position=None):
@@ -166,26 +167,22 @@ class SinkAttention(Mixer):
                               k_norm=self.k_norm, v_unit=self.value_norm, eps=self.eps, qk_unit=self.qk_unit, maps=self.maps,
                               interleaved=bool(getattr(self.position, "interleaved", False)))
         gate = proj[:, Cq + Ck + Cv:Cq + Ck + Cv + self.n_q * self.dv] if self.gate else None
-        return ops.linear(self.finish(self.attend(q, ctx, cache, gate)), self.w_out)
+        return ops.linear(self.attend(q, ctx, cache, gate), self.w_out)
 
     def attend(self, q: torch.Tensor, ctx: StepContext, cache: KVCacheView, gate) -> torch.Tensor:
-        """The attention launches of the step: q [T, heads, key row] -> [T, heads * value_dim]."""
+        """The attention launches of the step: q [T, heads, key row] -> what the output projection reads, [T, heads * value_dim]."""
         n_q = self.n_q * self.maps
         if self.paged:
-            o = torch.empty_like(q)
+            o = torch.empty((ctx.T, self.n_q, self.dv), dtype=q.dtype, device=q.device)
             paged_attend(q, o, ctx, cache, n_q=n_q, n_kv=self.n_kv, d=self.D, window=int(self.window or 0), scale=self.scale,
-                         use_mma=True, null_log2=self.sink_log2, gate=gate, chunk=int(self.chunk or 0))
-            return o.view(ctx.T, n_q * self.dv)
+                         use_mma=True, null_log2=self.sink_log2, gate=gate, chunk=int(self.chunk or 0), diff=self.difference)
+            return o.view(ctx.T, self.n_q * self.dv)
         out = torch.empty((ctx.T, n_q * self.dv), dtype=q.dtype, device=q.device)
         ops.sink_attention(q, out, cache.k, cache.v, q_start=ctx.q_start, kv_len=ctx.kv_len, block_table=cache.group.block_table,
                            n_kv=self.n_kv, page_size=cache.page_size, scale=self.scale, softcap=self.softcap, window=self.window or 0,
                            sink=self.sink, q_lens=None if ctx.uniform_decode else ctx.host_q_lens, workspace=ctx.workspace, gate=gate,
                            chunk=self.chunk or 0)
-        return out
-
-    def finish(self, heads: torch.Tensor) -> torch.Tensor:
-        """What the output projection reads, from the heads side by side."""
-        return heads
+        return out if self.maps == 1 else self.join_maps(out)
 
 
 @register_mixer("differential_attention")
@@ -202,7 +199,8 @@ class DifferentialAttention(SinkAttention):
     then the output projection.  A kv head's cache row holds both key vectors; a query row holds one query vector in its place
     and zeros in the other, so that the attention kernels see 2 * heads query heads on rows of 2 * key_dim elements.
 
-    lambda is made at load in double precision, the difference and its norm are float32.
+    lambda is made at load in double precision, the difference and its norm are float32.  The paged kernels take the difference
+    where a row is normalised (`ops.attention(diff=...)`); behind the kernels for any pair of head sizes it is a kernel of its own.
     params: as `sink_attention` (without sink, gate and value_mix) and diff; names of the four vectors: lq1, lk1, lq2, lk2."""
 
     maps = 2
@@ -212,7 +210,7 @@ class DifferentialAttention(SinkAttention):
         if self.gate or self.value_mix is not None:
             raise ValueError("a differential attention takes no gate and no blended values")
         self.diff = float(spec["diff"])
-        self.difference = 0.0
+        self.difference = (0.0, self.eps, 1.0 - self.diff)
         self.vec_names = [self.name((spec.get("names") or {}).get(k, k)) for k in ("lq1", "lk1", "lq2", "lk2")]
 
     def tensors(self) -> Dict[str, TensorDecl]:
@@ -221,11 +219,12 @@ class DifferentialAttention(SinkAttention):
     def load(self, src) -> None:
         super().load(src)
         lq1, lk1, lq2, lk2 = (src.fetch(n).double() for n in self.vec_names)
-        self.difference = float(torch.exp((lq1 * lk1).sum()) - torch.exp((lq2 * lk2).sum())) + self.diff
+        lam = float(torch.exp((lq1 * lk1).sum()) - torch.exp((lq2 * lk2).sum())) + self.diff
+        self.difference = (lam, self.eps, 1.0 - self.diff)
 
-    def finish(self, heads: torch.Tensor) -> torch.Tensor:
+    def join_maps(self, heads: torch.Tensor) -> torch.Tensor:
         T = heads.shape[0]
         out = torch.empty((T, self.n_q * self.dv), dtype=self.env.dtype, device=heads.device)
-        ops.map_difference(heads.view(T, 2 * self.n_q, self.dv), out, heads=self.n_q, lam=self.difference, eps=self.eps,
-                           scale=1.0 - self.diff)
+        ops.map_difference(heads.view(T, 2 * self.n_q, self.dv), out, heads=self.n_q, lam=self.difference[0], eps=self.eps,
+                           scale=self.difference[2])
         return out
