@@ -1453,6 +1453,7 @@ __global__ void attn_combine_diff_kernel(const float* __restrict__ part_o, const
                                          int qlen_max, T* __restrict__ out, int T_, int n_q, int d, int max_split, float lam, float eps,
                                          float scale) {
     __shared__ float red[32];
+    __shared__ float w_s[2][64];                 // the pieces' weights (a launch has at most 64)
     pdl_launch_dependents();
     pdl_wait();
     pdl_after_wait();
@@ -1461,19 +1462,25 @@ __global__ void attn_combine_diff_kernel(const float* __restrict__ part_o, const
     const int req = token_req ? token_req[tok] : tok;
     const int ns = nsplit ? min(max(nsplit[req], 1), max_split) : 1;
     if (ns == 1 && q_start[req + 1] - q_start[req] > qlen_max) return;
-    float f[2], M[2];
-#pragma unroll
-    for (int m = 0; m < 2; ++m) {
-        M[m] = -INFINITY;
-        for (int s = 0; s < ns; ++s) M[m] = fmaxf(M[m], part_ml[(((size_t)s * T_ + tok) * n_q + 2 * h + m) * 2]);
-        if (M[m] == -INFINITY) M[m] = 0.f;
+    // warp m weighs the pieces of map m: 2^(m_s - M) / sum
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    if (warp < 2) {
+        float mx = -INFINITY;
+        for (int s = lane; s < ns; s += 32) mx = fmaxf(mx, part_ml[(((size_t)s * T_ + tok) * n_q + 2 * h + warp) * 2]);
+        mx = warp_max(mx);
+        if (mx == -INFINITY) mx = 0.f;
         float L = 0.f;
-        for (int s = 0; s < ns; ++s) {
-            const size_t prow = ((size_t)s * T_ + tok) * n_q + 2 * h + m;
-            L += exp2f(part_ml[prow * 2] - M[m]) * part_ml[prow * 2 + 1];
+        for (int s = lane; s < ns; s += 32) {
+            const float2 ml = *reinterpret_cast<const float2*>(part_ml + (((size_t)s * T_ + tok) * n_q + 2 * h + warp) * 2);
+            const float e = exp2f(ml.x - mx);
+            w_s[warp][s] = e;
+            L = fmaf(e, ml.y, L);
         }
-        f[m] = L > 0.f ? 1.f / L : 0.f;
+        L = warp_sum(L);
+        const float inv = L > 0.f ? 1.f / L : 0.f;
+        for (int s = lane; s < ns; s += 32) w_s[warp][s] *= inv;
     }
+    __syncthreads();
     float ss = 0.f;
     constexpr int MAX_TURNS = 4;                 // 128 threads, head sizes up to 512
     float v[MAX_TURNS];
@@ -1483,12 +1490,13 @@ __global__ void attn_combine_diff_kernel(const float* __restrict__ part_o, const
         v[k] = 0.f;
         if (c < d) {
             float acc[2] = {0.f, 0.f};
+#pragma unroll 4
             for (int s = 0; s < ns; ++s) {
-                const size_t prow = ((size_t)s * T_ + tok) * n_q + 2 * h;
-                acc[0] += exp2f(part_ml[prow * 2] - M[0]) * part_o[prow * d + c];
-                acc[1] += exp2f(part_ml[prow * 2 + 2] - M[1]) * part_o[(prow + 1) * d + c];
+                const float* po = part_o + (((size_t)s * T_ + tok) * n_q + 2 * h) * d + c;
+                acc[0] = fmaf(w_s[0][s], po[0], acc[0]);
+                acc[1] = fmaf(w_s[1][s], po[d], acc[1]);
             }
-            v[k] = fmaf(acc[0], f[0], -lam * (acc[1] * f[1]));
+            v[k] = fmaf(-lam, acc[1], acc[0]);
             ss = fmaf(v[k], v[k], ss);
         }
     }
@@ -1806,7 +1814,7 @@ MSGL_API int msgl_attention_combine_diff(const float* part_o, const float* part_
                                          const int* q_start, int qlen_max, void* out, int T_, int n_q, int d, int max_split, int dtype,
                                          float lam, float eps, float scale, cudaStream_t stream) {
     if (T_ <= 0) return MSGL_OK;
-    if (n_q < 2 || n_q % 2 || d < 1 || d > 512 || max_split < 1 || (max_split > 1 && nsplit == nullptr)) return MSGL_ERR_SIZE;
+    if (n_q < 2 || n_q % 2 || d < 1 || d > 512 || max_split < 1 || max_split > 64 || (max_split > 1 && nsplit == nullptr)) return MSGL_ERR_SIZE;
     const dim3 grid(T_, n_q / 2);
     if (dtype == MSGL_F32)
         msgl_launch_pdl(attn_combine_diff_kernel<float>, grid, dim3(128), 0, stream, part_o, part_ml, token_req, nsplit, q_start, qlen_max,

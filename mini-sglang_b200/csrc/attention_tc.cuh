@@ -152,16 +152,17 @@ __global__ void __launch_bounds__(TC_THREADS, 2) attn_tc_kernel(const AttnParams
             const CUtensorMap* map = is_k ? &kmap : &vmap;
             const int n_box = TC_KT / tma_box;
             unsigned vt_phase = 0;
+            const int k_box = k_lo - k_lo % tma_box;
             for (int j = 0; j < n_tiles; ++j) {
                 const int key0 = (kt_begin + j) * TC_KT;
-                // boxes before the first key that is seen: their pages may have been given back; the rows of that key's own box
-                // stand in for them (finite, and no row of the block gives them weight)
-                const int key_b = max(key0 + lane * tma_box, k_lo - k_lo % tma_box);
-                const bool active = lane < n_box && key_b <= p_max;      // boxes past the last visible key are not fetched
+                const int key_b = key0 + lane * tma_box;
+                // boxes past the last visible key are not fetched, nor those before the first (their pages may have been given back)
+                const bool active = lane < n_box && key_b <= p_max && key_b >= k_box;
                 int y = 0;
                 if (active) y = (bt[page_index(p, key_b)] * p.n_kv + kvh) * p.page_size + page_slot(p, key_b);
                 const unsigned n_act = __popc(__ballot_sync(0xffffffffu, active));
-                const bool ragged = !is_k && p_max < key0 + TC_KT - 1;   // V rows past p_max have to be zero
+                const int n_dead = max(0, k_box - key0);                 // rows of the tile before the first box
+                const bool ragged = !is_k && (p_max < key0 + TC_KT - 1 || n_dead > 0);      // V rows that hold no seen key have to be zero
                 if (j >= 1 && !tc_mbar_wait(bar_free, (j - 1) & 1)) { fail = 1; break; }    // the tensor core has read tile j-1
                 TC_LMARK(0)
                 const unsigned bar = ragged ? bar_vt : bar_full;
@@ -174,8 +175,9 @@ __global__ void __launch_bounds__(TC_THREADS, 2) attn_tc_kernel(const AttnParams
                 if (ragged) {
                     if (!tc_mbar_wait(bar_vt, vt_phase)) { fail = 1; break; }
                     vt_phase ^= 1u;
-                    const int r0 = p_max + 1 - key0;                     // first row without a visible key
-                    for (int idx = r0 * 16 + lane; idx < TC_KT * 16; idx += 32) {
+                    const int r0 = min(p_max + 1 - key0, TC_KT);         // first row without a visible key
+                    for (int i = lane; i < (TC_KT - r0 + n_dead) * 16; i += 32) {
+                        const int idx = i < n_dead * 16 ? i : i + (r0 - n_dead) * 16;
                         const unsigned a = dst_tile + (unsigned)((idx >> 3) & 1) * TC_KHALF_BYTES + (unsigned)(idx >> 4) * 128u + (unsigned)(idx & 7) * 16u;
                         asm volatile("st.shared.v4.u32 [%0], {%1,%1,%1,%1};\n" ::"r"(a), "r"(0u) : "memory");
                     }

@@ -160,11 +160,12 @@ __global__ void __launch_bounds__(TC2_THREADS, 1) attn_tc2_kernel(const AttnPara
         const int* bt = p.block_table + (size_t)ti.req * p.bt_stride;
         const int n_box = TC_KT / tma_box;
         unsigned vt_phase = 0;
+        // boxes before that of the first key that is seen are not fetched: their pages may have been given back.  (Boxes with kept
+        // first tokens are always there.)
+        const int k_box = k_lo - k_lo % tma_box;
         auto box_row = [&](int j) -> int {            // first cache row of this lane's box of tile j, or -1
-            int key_b = tile_of(j) * TC_KT + lane * tma_box;
-            // boxes before the first key that is seen: their pages may have been given back; the rows of that key's own box stand
-            // in for them (finite, and no row of the block gives them weight).  Boxes with kept first tokens are always there.
-            if (!(EXT && (j < n_sink || key_b < p.keep_first))) key_b = max(key_b, k_lo - k_lo % tma_box);
+            const int key_b = tile_of(j) * TC_KT + lane * tma_box;
+            if (!(EXT && (j < n_sink || key_b < p.keep_first)) && key_b < k_box) return -1;
             if (j >= n_tiles || lane >= n_box || key_b > p_max) return -1;          // boxes past the last visible key are not fetched
             if (EXT && j < n_sink && key_b >= sink_hi) return -1;                   // nor those past the last kept token
             return (bt[page_index(p, key_b)] * p.n_kv + kvh) * p.page_size + page_slot(p, key_b);
@@ -177,7 +178,8 @@ __global__ void __launch_bounds__(TC2_THREADS, 1) attn_tc2_kernel(const AttnPara
             const int last_key = (EXT && j < n_sink) ? sink_hi - 1 : p_max;      // the tile's rows behind it hold nothing that may be read
             const unsigned dst_tile = (is_k ? k_s : v_s) + (unsigned)st * TC_KV_BYTES;
             const unsigned n_act = __popc(__ballot_sync(0xffffffffu, y >= 0));
-            const bool ragged = !is_k && last_key < key0 + TC_KT - 1;            // V rows past the last key have to be zero
+            const int n_dead = (EXT && j < n_sink) ? 0 : max(0, k_box - key0);   // rows of the tile before the first box
+            const bool ragged = !is_k && (last_key < key0 + TC_KT - 1 || n_dead > 0);      // V rows that hold no seen key have to be zero
             if (j >= 2 && !tc_mbar_wait(is_k ? bar_kr(st) : bar_vr(st), ((j >> 1) - 1) & 1)) { fail = 1; break; }   // tile j-2 has been read
             const unsigned bar = ragged ? bar_vt : (is_k ? bar_kf(st) : bar_vf(st));
             if (lane == 0) tc_mbar_expect_tx(bar, n_act * 2u * (unsigned)tma_box * 128u);
@@ -189,8 +191,10 @@ __global__ void __launch_bounds__(TC2_THREADS, 1) attn_tc2_kernel(const AttnPara
             if (ragged) {
                 if (!tc_mbar_wait(bar_vt, vt_phase)) { fail = 1; break; }
                 vt_phase ^= 1u;
-                const int r0 = last_key + 1 - key0;                              // first row without a visible key
-                for (int idx = r0 * 16 + lane; idx < TC_KT * 16; idx += 32) {
+                const int r0 = min(last_key + 1 - key0, TC_KT);                  // first row without a visible key
+                for (int i = lane; i < (TC_KT - r0 + n_dead) * 16; i += 32) {
+                    const int idx = i < n_dead * 16 ? i : i + (r0 - n_dead) * 16;
+                    if (EXT && i < n_dead * 16 && key0 + (idx >> 4) - (idx >> 4) % tma_box < p.keep_first) continue;
                     const unsigned a = dst_tile + (unsigned)((idx >> 3) & 1) * TC_KHALF_BYTES + (unsigned)(idx >> 4) * 128u + (unsigned)(idx & 7) * 16u;
                     asm volatile("st.shared.v4.u32 [%0], {%1,%1,%1,%1};\n" ::"r"(a), "r"(0u) : "memory");
                 }

@@ -276,6 +276,7 @@ __global__ void __launch_bounds__(128) sink_qkv_prep_kernel(const SinkPrepParams
 template <typename T>
 __global__ void __launch_bounds__(128) sink_qkv_prep_vec_kernel(const SinkPrepParams p, int n_slots) {
     constexpr int V = 16 / sizeof(T);
+    pdl_launch_dependents();
     const long long w_idx = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
     const int M = p.maps, nq = p.n_q * M, nk = p.n_kv * M, lane = threadIdx.x & 31;
     // vectors of 16 shares or less share a warp: `per` of them side by side
@@ -293,6 +294,9 @@ __global__ void __launch_bounds__(128) sink_qkv_prep_vec_kernel(const SinkPrepPa
     float v[V];
 #pragma unroll
     for (int k = 0; k < V; ++k) v[k] = 0.f;
+    pdl_wait();
+    pdl_after_wait();
+    pdl_small();
     if (mine) sk_load16(src + l * V, v);
     const float* w = is_v ? nullptr : (is_q ? p.wq : p.wk);
     if (w != nullptr || (is_v && p.v_unit)) {           // (the lanes of one vector take the same branch: the shuffles stay among them)
@@ -378,8 +382,8 @@ MSGL_API int msgl_sink_qkv_prep(const void* proj, long long stride, const float*
     if ((p.cs == nullptr || interleaved) && v_first == nullptr && d % V == 0 && dv % V == 0 && stride % V == 0 && max(d, dv) <= 32 * V && (all & 15) == 0) {
         const int widest = max(d, dv) / V, lanes = widest <= 4 ? 4 : widest <= 8 ? 8 : widest <= 16 ? 16 : 32, per = 4 * (32 / lanes);
         const unsigned blocks = (unsigned)(((long long)T_ * n_slots + per - 1) / per);
-        if (dtype == MSGL_F32) sink_qkv_prep_vec_kernel<float><<<blocks, 128, 0, stream>>>(p, n_slots);
-        else sink_qkv_prep_vec_kernel<__nv_bfloat16><<<blocks, 128, 0, stream>>>(p, n_slots);
+        if (dtype == MSGL_F32) msgl_launch_pdl(sink_qkv_prep_vec_kernel<float>, dim3(blocks), dim3(128), 0, stream, p, n_slots);
+        else msgl_launch_pdl(sink_qkv_prep_vec_kernel<__nv_bfloat16>, dim3(blocks), dim3(128), 0, stream, p, n_slots);
         return msgl_check_launch();
     }
     const dim3 grid(T_, (n_slots + 3) / 4);

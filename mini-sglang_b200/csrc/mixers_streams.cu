@@ -51,7 +51,9 @@ struct StreamMixParams {
 template <typename A, typename O, int S, int NV>
 __global__ void __launch_bounds__(512) stream_mix_norm_vec_kernel(const StreamMixParams p) {
     __shared__ float red[32];
+    pdl_launch_dependents();
     const int r = blockIdx.x, H = p.H;
+    // the layer's numbers (and the row index) are nobody's output: fetched while the kernel before this one finishes
     const size_t src = p.rows ? (size_t)p.rows[r] : (size_t)r;
     const float* xi = p.x_in + src * p.row_stride;
     float mix[S][S], w_out[S], w_in[S];
@@ -62,6 +64,9 @@ __global__ void __launch_bounds__(512) stream_mix_norm_vec_kernel(const StreamMi
 #pragma unroll
         for (int t = 0; t < S; ++t) mix[s][t] = p.y ? p.mix[s * S + t] : 0.f;
     }
+    pdl_wait();
+    pdl_after_wait();
+    pdl_small();
     float u[NV][4];
     float sm = 0.f;
 #pragma unroll
@@ -183,7 +188,7 @@ static int stream_mix_norm_launch(const StreamMixParams& p, int n_rows, cudaStre
         int nv = 1;
         while ((n4 + nv - 1) / nv > 512) nv *= 2;
         const int threads = (((n4 + nv - 1) / nv) + 31) / 32 * 32;
-#define SMN(S_, NV_) stream_mix_norm_vec_kernel<A, O, S_, NV_><<<n_rows, threads, 0, stream>>>(p)
+#define SMN(S_, NV_) msgl_launch_pdl(stream_mix_norm_vec_kernel<A, O, S_, NV_>, dim3(n_rows), dim3(threads), 0, stream, p)
 #define SMN_S(S_) do { if (nv == 1) SMN(S_, 1); else if (nv == 2) SMN(S_, 2); else SMN(S_, 4); } while (0)
         if (S == 1) SMN_S(1); else if (S == 2) SMN_S(2); else if (S == 3) SMN_S(3); else SMN_S(4);
 #undef SMN_S

@@ -231,7 +231,7 @@ def test_model_level_bound_tells_faults_apart(monkeypatch):
         "a feed-forward's share": moved(None, zero("l2.hc2.out")),
     }
     for what, by in faults.items():
-        assert by > 0.045, f"{what} moves the rows by {by:.2%} only"
+        assert by > 0.3, f"{what} moves the rows by {by:.2%} only"
 
 
 def _one_after_the_other(X, y, mix, w_out):

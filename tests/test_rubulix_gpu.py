@@ -63,12 +63,12 @@ def runner(name, dtype, num_pages, max_reqs=4, page_size=None, graphs=True, ctx=
 
 # The reference is the plain implementation in double precision.  float32 rows are held to 2e-4 of a row's rms (6 times that for
 # the largest element); bfloat16 rows (projections, cached keys and values and the activations between kernels rounded to 8
-# mantissa bits; scores, softmax, norms and the copies of the stream float32) to 4 %, which every planted fault of
-# tests/test_rubulix_cpu.py exceeds, but for a tenth of a request's rows, which may lie in the noise's tail (a difference of maps
-# that nearly cancels is normed up), none by more than TAIL_FACTOR times.
+# mantissa bits; scores, softmax, norms and the copies of the stream float32) to 8 % (a difference of maps that nearly cancels is
+# normed up, and with it the rounding of what it is made of), but for a tenth of a request's rows, which may lie in the noise's
+# tail, none by more than TAIL_FACTOR times.  The faults of tests/test_rubulix_cpu.py move some row by 30 % or more.
 F32_RMS_FRACTION = 2e-4
-BF16_RMS_FRACTION_R = 0.04
-TAIL_SHARE, TAIL_FACTOR = 0.1, 4.0
+BF16_RMS_FRACTION_R = 0.08
+TAIL_SHARE, TAIL_FACTOR = 0.1, 2.0
 
 
 def row_close(row, want, bound):
@@ -635,7 +635,7 @@ def test_random_configurations(seed):
         steps += [{"entries": [("p", toks[2 + 4 * i:6 + 4 * i], [0, 1, 2, 3]), ("o", [other[9 + i]], [0])]} for i in range(24)]
         steps += [{"entries": [("p", toks[98:100], [0, 1])]}]
         got.update(play(r, steps))
-        compare(f"random {seed}", dtype, got, None, ref=ref, bound=0.06 if dtype == "bfloat16" else None)
+        compare(f"random {seed}", dtype, got, None, ref=ref, bound=0.1 if dtype == "bfloat16" else None)
         r.mgr.check_idle()
 
 
@@ -716,7 +716,7 @@ def _holds(cfg, w, prompt, got, dtype):
     toks = list(prompt)
     for t in got:           # bfloat16 may take another of two nearly equal logits
         row = plain_of(cfg, w, toks)[-1]
-        assert float(row.max() - row[t]) < 0.1 * float(row.std()) + 0.05
+        assert float(row.max() - row[t]) < 0.25 * float(row.std())
         toks.append(t)
 
 
