@@ -272,20 +272,17 @@ __global__ void __launch_bounds__(128) sink_qkv_prep_kernel(const SinkPrepParams
 
 // The same without blending or a rotation in halves, a lane 16 bytes of a vector (sizes that are multiples of the lane's share and
 // at most 32 of them): one read of every element, norms and turned pairs from registers.  n_slots: the vectors of a token that
-// are made (q alone where nothing is cached).
+// are made (q alone where nothing is cached); their number in all fits 32 bits.
 template <typename T>
-__global__ void __launch_bounds__(128) sink_qkv_prep_vec_kernel(const SinkPrepParams p, int n_slots) {
+__global__ void __launch_bounds__(128) sink_qkv_prep_vec_kernel(const SinkPrepParams p, int n_slots, int lg) {
     constexpr int V = 16 / sizeof(T);
     pdl_launch_dependents();
-    const long long w_idx = (long long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
     const int M = p.maps, nq = p.n_q * M, nk = p.n_kv * M, lane = threadIdx.x & 31;
-    // vectors of 16 shares or less share a warp: `per` of them side by side
-    const int nd = p.d / V, nv = p.dv / V, widest = nd > nv ? nd : nv;
-    const int lanes = widest <= 4 ? 4 : widest <= 8 ? 8 : widest <= 16 ? 16 : 32, per = 32 / lanes;
-    const long long job = w_idx * per + lane / lanes;
-    const int l = lane % lanes;
-    const bool live = job < (long long)p.T * n_slots;
-    const int t = live ? (int)(job / n_slots) : 0, slot = live ? (int)(job - (long long)t * n_slots) : 0;
+    // 2^lg lanes take a vector; vectors of 16 shares or less share a warp
+    const int lanes = 1 << lg, l = lane & (lanes - 1);
+    const unsigned job = ((blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5)) << (5 - lg)) + (unsigned)(lane >> lg);
+    const bool live = job < (unsigned)p.T * (unsigned)n_slots;
+    const int t = live ? (int)(job / (unsigned)n_slots) : 0, slot = live ? (int)job - t * n_slots : 0;
     const bool is_v = slot >= nq + nk, is_q = slot < nq;
     const int n = is_v ? p.dv : p.d;
     const T* row = reinterpret_cast<const T*>(p.proj) + (size_t)t * p.stride;
@@ -303,7 +300,7 @@ __global__ void __launch_bounds__(128) sink_qkv_prep_vec_kernel(const SinkPrepPa
         float ss = 0.f;
 #pragma unroll
         for (int k = 0; k < V; ++k) ss = fmaf(v[k], v[k], ss);
-        const unsigned mask = lanes == 32 ? 0xffffffffu : ((1u << lanes) - 1u) << (lane / lanes * lanes);
+        const unsigned mask = lanes == 32 ? 0xffffffffu : ((1u << lanes) - 1u) << (lane - l);
         for (int o = lanes >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(mask, ss, o);
         const float f = 1.f / sqrtf(ss / (float)n + p.eps);
         if (w != nullptr && mine) {
@@ -321,21 +318,32 @@ __global__ void __launch_bounds__(128) sink_qkv_prep_vec_kernel(const SinkPrepPa
     if (p.cs != nullptr && !is_v && mine) {             // neighbouring pairs lie within a lane
         const float* cs = p.cs + (size_t)t * p.rot;
         const int half = p.rot >> 1;
+        float cv[V / 2], sv[V / 2];
+        const int p0 = (l * V) >> 1;
+        if (V == 8 && (half & 3) == 0) {                // a lane's pairs are turned together or not at all: 16 bytes of angles at once
+            if (p0 < half) {
+                const float4 c4 = *reinterpret_cast<const float4*>(cs + p0), s4 = *reinterpret_cast<const float4*>(cs + half + p0);
+                cv[0] = c4.x; cv[1] = c4.y; sv[0] = s4.x; sv[1] = s4.y;
+                if constexpr (V == 8) { cv[2] = c4.z; cv[3] = c4.w; sv[2] = s4.z; sv[3] = s4.w; }
+            } else {
 #pragma unroll
-        for (int k = 0; k < V; k += 2) {
-            const int pr = (l * V + k) >> 1;
-            if (pr < half) {
-                const float c = cs[pr], s = cs[half + pr], a = v[k], b = v[k + 1];
-                v[k] = a * c - b * s;
-                v[k + 1] = b * c + a * s;
+                for (int k = 0; k < V / 2; ++k) { cv[k] = 1.f; sv[k] = 0.f; }
             }
+        } else {
+#pragma unroll
+            for (int k = 0; k < V / 2; ++k) { cv[k] = p0 + k < half ? cs[p0 + k] : 1.f; sv[k] = p0 + k < half ? cs[half + p0 + k] : 0.f; }
+        }
+#pragma unroll
+        for (int k = 0; k < V / 2; ++k) {
+            const float a = v[2 * k], b = v[2 * k + 1];
+            if (p0 + k < half) { v[2 * k] = a * cv[k] - b * sv[k]; v[2 * k + 1] = b * cv[k] + a * sv[k]; }
         }
     }
     if (p.qk_unit && !is_v) {
         float ss = 0.f;
 #pragma unroll
         for (int k = 0; k < V; ++k) ss = fmaf(v[k], v[k], ss);
-        const unsigned mask = lanes == 32 ? 0xffffffffu : ((1u << lanes) - 1u) << (lane / lanes * lanes);
+        const unsigned mask = lanes == 32 ? 0xffffffffu : ((1u << lanes) - 1u) << (lane - l);
         for (int o = lanes >> 1; o > 0; o >>= 1) ss += __shfl_xor_sync(mask, ss, o);
         const float f = 1.f / sqrtf(ss / (float)n + p.eps);
 #pragma unroll
@@ -344,7 +352,7 @@ __global__ void __launch_bounds__(128) sink_qkv_prep_vec_kernel(const SinkPrepPa
     if (!mine) return;
     T* dst;
     if (is_q) {
-        const int m = slot % M;
+        const int m = M == 1 ? 0 : (M == 2 ? slot & 1 : slot % M);
         dst = reinterpret_cast<T*>(p.q_out) + ((size_t)t * nq + slot) * n * M + l * V;
         float z[V];
 #pragma unroll
@@ -354,9 +362,10 @@ __global__ void __launch_bounds__(128) sink_qkv_prep_vec_kernel(const SinkPrepPa
         dst += m * n;
     } else {
         const int loc = p.out_loc[t], h = is_v ? slot - nq - nk : slot - nq;
-        const int mm = is_v ? 1 : M;
-        dst = reinterpret_cast<T*>(is_v ? p.v_cache : p.k_cache) +
-              (((size_t)(loc / p.page_size) * p.n_kv + h / mm) * p.page_size + loc % p.page_size) * n * mm + h % mm * n + l * V;
+        const int mm = is_v ? 1 : M, hh = mm == 1 ? h : (mm == 2 ? h >> 1 : h / mm);
+        const unsigned page = (unsigned)loc / (unsigned)p.page_size, at = (unsigned)loc - page * (unsigned)p.page_size;
+        dst = reinterpret_cast<T*>(is_v ? p.v_cache : p.k_cache) + (((size_t)page * p.n_kv + hh) * p.page_size + at) * (size_t)(n * mm) +
+              (h - hh * mm) * n + l * V;
     }
     sk_store16(dst, v);
 }
@@ -379,11 +388,12 @@ MSGL_API int msgl_sink_qkv_prep(const void* proj, long long stride, const float*
     const uintptr_t all = (uintptr_t)proj | (uintptr_t)q_out | (uintptr_t)k_cache | (uintptr_t)v_cache | (uintptr_t)wq | (uintptr_t)wk;
     // vectors of a token: q, and where they are cached k and v
     const int n_slots = maps * n_q + (k_cache != nullptr ? (maps + 1) * n_kv : 0);
-    if ((p.cs == nullptr || interleaved) && v_first == nullptr && d % V == 0 && dv % V == 0 && stride % V == 0 && max(d, dv) <= 32 * V && (all & 15) == 0) {
-        const int widest = max(d, dv) / V, lanes = widest <= 4 ? 4 : widest <= 8 ? 8 : widest <= 16 ? 16 : 32, per = 4 * (32 / lanes);
+    if ((p.cs == nullptr || interleaved) && v_first == nullptr && d % V == 0 && dv % V == 0 && stride % V == 0 && max(d, dv) <= 32 * V && (all & 15) == 0 &&
+        ((uintptr_t)cs & 15) == 0 && (long long)T_ * n_slots < (1ll << 30)) {
+        const int widest = max(d, dv) / V, lg = widest <= 4 ? 2 : widest <= 8 ? 3 : widest <= 16 ? 4 : 5, per = 4 * (32 >> lg);
         const unsigned blocks = (unsigned)(((long long)T_ * n_slots + per - 1) / per);
-        if (dtype == MSGL_F32) msgl_launch_pdl(sink_qkv_prep_vec_kernel<float>, dim3(blocks), dim3(128), 0, stream, p, n_slots);
-        else msgl_launch_pdl(sink_qkv_prep_vec_kernel<__nv_bfloat16>, dim3(blocks), dim3(128), 0, stream, p, n_slots);
+        if (dtype == MSGL_F32) msgl_launch_pdl(sink_qkv_prep_vec_kernel<float>, dim3(blocks), dim3(128), 0, stream, p, n_slots, lg);
+        else msgl_launch_pdl(sink_qkv_prep_vec_kernel<__nv_bfloat16>, dim3(blocks), dim3(128), 0, stream, p, n_slots, lg);
         return msgl_check_launch();
     }
     const dim3 grid(T_, (n_slots + 3) / 4);

@@ -4,12 +4,13 @@
 //
 //   stream_mix_norm_kernel   x_t <- sum_s mix[s][t] x_s + out[t] y for all copies at once, then u = sum_t in[t] x_t, normed:
 //                            the end of one sublayer and the beginning of the next in one pass; a form with the row in
-//                            registers for 1 to 4 copies, one for any number
+//                            registers for 1 to 4 copies (few rows: a row over a cluster of blocks), one for any number
 //   map_difference_kernel    o = a_1 - lambda a_2 of a head's two maps, o / sqrt(mean(o^2) + eps) * scale
 //
 // All arithmetic is float32; the copies are float32, what a sublayer hands over (y) and takes (the normed u) is in the
 // activation type.
 #include "common.cuh"
+#include <cooperative_groups.h>
 #include <math.h>
 
 namespace {
@@ -48,14 +49,31 @@ struct StreamMixParams {
     int S, H;
 };
 
-template <typename A, typename O, int S, int NV>
+// CL > 1: a row lies over a cluster of CL blocks, a quarter each (few rows would keep few SMs busy); the blocks' sums meet through
+// distributed shared memory.
+template <typename A, typename O, int S, int NV, int CL = 1>
 __global__ void __launch_bounds__(512) stream_mix_norm_vec_kernel(const StreamMixParams p) {
     __shared__ float red[32];
     pdl_launch_dependents();
-    const int r = blockIdx.x, H = p.H;
+    const int r = blockIdx.x / CL, H = p.H / CL, W = p.H;              // H: the columns of this block, from c0
+    const int c0 = CL > 1 ? (int)(blockIdx.x % CL) * H : 0;
     // the layer's numbers (and the row index) are nobody's output: fetched while the kernel before this one finishes
     const size_t src = p.rows ? (size_t)p.rows[r] : (size_t)r;
-    const float* xi = p.x_in + src * p.row_stride;
+    const float* xi = p.x_in + src * p.row_stride + c0;
+    // the sum over the row of what each thread holds of it
+    __shared__ float part[2];
+    auto row_sum = [&](float v, int which) -> float {
+        float t = block_sum(v, red);
+        if constexpr (CL > 1) {
+            auto cluster = cooperative_groups::this_cluster();
+            if (threadIdx.x == 0) part[which] = t;
+            cluster.sync();
+            t = 0.f;
+#pragma unroll
+            for (int i = 0; i < CL; ++i) t += cluster.map_shared_rank(part, i)[which];
+        }
+        return t;
+    };
     float mix[S][S], w_out[S], w_in[S];
 #pragma unroll
     for (int s = 0; s < S; ++s) {
@@ -83,7 +101,7 @@ __global__ void __launch_bounds__(512) stream_mix_norm_vec_kernel(const StreamMi
             }
             if (p.y) {
                 float yv[4];
-                ms_load4(reinterpret_cast<const A*>(p.y) + src * H + i, yv);
+                ms_load4(reinterpret_cast<const A*>(p.y) + src * W + c0 + i, yv);
                 float n[S][4];
 #pragma unroll
                 for (int t = 0; t < S; ++t)
@@ -96,7 +114,7 @@ __global__ void __launch_bounds__(512) stream_mix_norm_vec_kernel(const StreamMi
                     }
 #pragma unroll
                 for (int t = 0; t < S; ++t) {
-                    if (p.x_out) ms_store4(p.x_out + (src * S + t) * H + i, n[t]);
+                    if (p.x_out) ms_store4(p.x_out + (src * S + t) * W + c0 + i, n[t]);
 #pragma unroll
                     for (int e = 0; e < 4; ++e) x[t][e] = n[t][e];
                 }
@@ -109,9 +127,9 @@ __global__ void __launch_bounds__(512) stream_mix_norm_vec_kernel(const StreamMi
             for (int e = 0; e < 4; ++e) sm += p.center ? u[k][e] : u[k][e] * u[k][e];
         }
     }
-    float total = block_sum(sm, red);
+    float total = row_sum(sm, 0);
     if (p.center) {
-        const float mean = total / (float)H;
+        const float mean = total / (float)W;
         float ss = 0.f;
 #pragma unroll
         for (int k = 0; k < NV; ++k) {
@@ -121,21 +139,22 @@ __global__ void __launch_bounds__(512) stream_mix_norm_vec_kernel(const StreamMi
                 for (int e = 0; e < 4; ++e) { u[k][e] -= mean; ss = fmaf(u[k][e], u[k][e], ss); }
             }
         }
-        total = block_sum(ss, red);
+        total = row_sum(ss, 1);
     }
-    const float inv = 1.f / sqrtf(total / (float)H + p.eps);
+    const float inv = 1.f / sqrtf(total / (float)W + p.eps);
 #pragma unroll
     for (int k = 0; k < NV; ++k) {
         const int i = (threadIdx.x + k * blockDim.x) * 4;
         if (i < H) {
             float wv[4], bv[4] = {0.f, 0.f, 0.f, 0.f}, ov[4];
-            ms_load4(p.w + i, wv);
-            if (p.b) ms_load4(p.b + i, bv);
+            ms_load4(p.w + c0 + i, wv);
+            if (p.b) ms_load4(p.b + c0 + i, bv);
 #pragma unroll
             for (int e = 0; e < 4; ++e) ov[e] = fmaf(u[k][e] * inv, wv[e], bv[e]);
-            ms_store4(reinterpret_cast<O*>(p.o) + (size_t)r * H + i, ov);
+            ms_store4(reinterpret_cast<O*>(p.o) + (size_t)r * W + c0 + i, ov);
         }
     }
+    if constexpr (CL > 1) cooperative_groups::this_cluster().sync();        // the others may still read this block's sums
 }
 
 #define MS_MAX_STREAMS 32
@@ -184,6 +203,26 @@ static int stream_mix_norm_launch(const StreamMixParams& p, int n_rows, cudaStre
     const int H = p.H, S = p.S;
     const uintptr_t all = (uintptr_t)p.x_in | (uintptr_t)p.x_out | (uintptr_t)p.y | (uintptr_t)p.w | (uintptr_t)p.b | (uintptr_t)p.o;
     if (S <= 4 && H % 8 == 0 && (all & 15) == 0 && p.row_stride % 4 == 0 && p.copy_stride % 4 == 0 && H <= 4 * 4 * 512) {
+        constexpr int CL = 4;
+        if (n_rows <= 32 && H % (4 * CL) == 0 && H >= 1024 && H / (4 * CL) <= 512) {
+            const int threads = (H / (4 * CL) + 31) / 32 * 32;
+            cudaLaunchConfig_t cfg = {};
+            cfg.gridDim = dim3(n_rows * CL);
+            cfg.blockDim = dim3(threads);
+            cfg.stream = stream;
+            cudaLaunchAttribute attr[2];
+            attr[0].id = cudaLaunchAttributeClusterDimension;
+            attr[0].val.clusterDim.x = CL; attr[0].val.clusterDim.y = 1; attr[0].val.clusterDim.z = 1;
+            attr[1].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+            attr[1].val.programmaticStreamSerializationAllowed = 1;
+            cfg.attrs = attr;
+            cfg.numAttrs = msgl_pdl_enabled() ? 2 : 1;
+            if (S == 1) cudaLaunchKernelEx(&cfg, stream_mix_norm_vec_kernel<A, O, 1, 1, CL>, p);
+            else if (S == 2) cudaLaunchKernelEx(&cfg, stream_mix_norm_vec_kernel<A, O, 2, 1, CL>, p);
+            else if (S == 3) cudaLaunchKernelEx(&cfg, stream_mix_norm_vec_kernel<A, O, 3, 1, CL>, p);
+            else cudaLaunchKernelEx(&cfg, stream_mix_norm_vec_kernel<A, O, 4, 1, CL>, p);
+            return msgl_check_launch();
+        }
         const int n4 = H / 4;
         int nv = 1;
         while ((n4 + nv - 1) / nv > 512) nv *= 2;

@@ -125,17 +125,18 @@ def i32(v):
 # kernels alone
 # ---------------------------------------------------------------------------------------------------------------------
 @pytest.mark.parametrize("dtype", BOTH)
-@pytest.mark.parametrize("H", [1, 50, 72, 1000, 2056, 4096, 8200, 12288])
-def test_copies_of_the_stream(dtype, H):
-    """Update, read and norm in one kernel: 1 to 6 copies (the forms with the row in registers and the general one), a layer norm
-    with a bias and an RMS norm without, the copies still one row or apart, updated in place, or only the wanted rows read."""
+@pytest.mark.parametrize("H,T", [(1, 5), (50, 5), (72, 5), (1000, 5), (1024, 32), (2056, 5), (4096, 5), (4096, 33), (8192, 3), (8200, 5), (12288, 5)])
+def test_copies_of_the_stream(dtype, H, T):
+    """Update, read and norm in one kernel: 1 to 6 copies (the forms with the row in registers, in one block or over a cluster where
+    the rows are few, and the general one), a layer norm with a bias and an RMS norm without, the copies still one row or apart,
+    updated in place, or only the wanted rows read."""
     from mini_sglang_b200 import ops
     torch.manual_seed(H)
-    T = 5
     w, b = (1 + 0.1 * torch.randn(H)).cuda(), (0.3 * torch.randn(H)).cuda()
-    rows = i32([4, 0, 3])
+    rows = i32([T - 1, 0, 2])
     for S in (1, 2, 3, 4, 6):
-        X = torch.randn(T, S, H) + torch.tensor([0.0, 3.0, -40.0, 0.0, 1.0])[:, None, None]          # rows far from a mean of zero
+        X = torch.randn(T, S, H)
+        X[1:3] += torch.tensor([3.0, -40.0])[:, None, None]          # rows far from a mean of zero
         y = torch.randn(T, H).to(DT[dtype])
         c_in, mix, c_out = torch.randn(S), torch.randn(S, S), torch.randn(S)
 
