@@ -392,11 +392,11 @@ def test_attention_of_any_pair_of_sizes_within_chunks_in_pieces(dtype, how):
             _chunk_case(dtype, how, H=6, G=2, d=40, dv=24, P=16, ctx=1100, n_new=1, chunk=chunk, spike=spike, seed=spike, splits=2)
 
 
-# (dtype, how, vector size, value size, kv heads, heads): cache rows of 128 (tcgen05), 96, 64, 32, 48, more maps a kv head than a
+# (dtype, how, vector size, value size, kv heads, heads): cache rows of 128 (tcgen05), 256 ... 16, more maps a kv head than a
 # decode block's columns and than a tile's rows; the kernels for any pair
 DIFF = [("bfloat16", "paged", 64, 128, 2, 4), ("bfloat16", "paged", 64, 128, 1, 5), ("bfloat16", "paged", 48, 96, 2, 2), ("bfloat16", "paged", 32, 64, 1, 3),
         ("bfloat16", "paged", 16, 32, 1, 24), ("bfloat16", "paged", 24, 48, 2, 4), ("bfloat16", "paged", 8, 16, 1, 80), ("bfloat16", "paged", 64, 128, 1, 40),
-        ("bfloat16", "pair", 32, 40, 2, 4), ("bfloat16", "f32", 20, 24, 1, 3), ("float32", "pair", 24, 48, 2, 4)]
+        ("bfloat16", "paged", 128, 256, 1, 2), ("bfloat16", "paged", 40, 80, 2, 6), ("bfloat16", "pair", 32, 40, 2, 4), ("bfloat16", "f32", 20, 24, 1, 3), ("float32", "pair", 24, 48, 2, 4)]
 
 
 @pytest.mark.parametrize("dtype,how,d,dv,G,H", DIFF)
