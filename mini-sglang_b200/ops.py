@@ -387,6 +387,7 @@ def attention_tc(q: torch.Tensor, out: torch.Tensor, k_cache: torch.Tensor, v_ca
     T, n_q, d = q.shape
     B = kv_len.numel()
     assert q.is_contiguous() and out.is_contiguous() and block_table.stride(1) == 1 and q.dtype == torch.bfloat16
+    assert tuple(out.shape) == (T, n_q if diff is None else n_q // 2, d) and q_start.numel() == B + 1 and block_table.shape[0] == B
     status = _status_tensor(q.device)
     group = n_q // n_kv
     whole = k_cache.is_contiguous() and v_cache.is_contiguous() and k_cache.shape == v_cache.shape
